@@ -237,11 +237,17 @@ MIXER_KEYS = {
 #              the input) | "gated_silu" (down (silu(gate x) * up x), the score weighs the output) | "clamped" (gate and
 #              up clamped by the entry's ``limit``, g sigmoid(1.702 g) (u + 1)); a ``shared`` always-on expert is read
 #              from the layer's mlp entry; shared_gate: the shared expert's output is weighed by one sigmoid per token
-#   dense_act: activation of a dense feed-forward, "gelu" (erf) | "relu2"
+#   dense_act: activation of a dense feed-forward, "gelu" (erf) | "relu2" | "polynorm" (a learned mix of the first three
+#              powers, each divided by its root mean square over the feed-forward's width)
+#   latent:    rot, the pairing of the rotated entries, "halves" (i with i + dims/2) | "pairs" (2i with 2i+1); gate (a
+#              sigmoid per output channel); p32 as for attention.  A mixer entry may name ``mask.size`` (a sliding window)
+#              and ``kv_from``
+#   depth_average: what a layer passes on is a learned mix of the embedding output and every layer's result so far
 # Per layer, an attention mixer may also name ``softcap`` (scores pass through cap * tanh(score / cap)) and
 # ``kv_from: j`` (no key/value projections: it reads the keys and values layer j cached); a mixture of experts may name
 # ``router.identity`` (that many extra router outputs whose "expert" returns its input).
 _ATTENTION_DEFAULT = {"mask": "window", "sink": False, "qk_norm": "unit", "bias": False, "gate": "head", "p32": False}
+_LATENT_DEFAULT = {"rot": "halves", "gate": True, "p32": False}
 _MOE_DEFAULT = {"router": "sigmoid", "router_bias": False, "expert": "relu2", "shared_gate": False}
 ARCHITECTURE_TRAITS = {
     "Badapel": {"block": "sandwich", "norm": "layer", "tied_head": True},
@@ -253,6 +259,8 @@ ARCHITECTURE_TRAITS = {
     "Zudovik": {"block": "postnorm", "norm": "rms", "tied_head": False, "dense_act": "relu2",
                 "attention": {"mask": "window", "sink": "learned", "qk_norm": "full", "bias": True, "gate": "head", "p32": True},
                 "moe": {"router": "softmax_all", "expert": "clamped", "shared_gate": True}},
+    "Ratesun": {"block": "sandwich", "norm": "layer", "tied_head": True, "dense_act": "polynorm", "depth_average": True,
+                "latent": {"rot": "pairs", "gate": False, "p32": True}},
 }
 FF_KINDS = ("dense", "moe")
 
@@ -274,6 +282,9 @@ class HybridConfig:
     ``attention`` / ``moe`` come from :data:`ARCHITECTURE_TRAITS` unless given.  ``max_positions`` is the length of the
     learned position table (``positions = "learned"``).  A mixture of experts may name a ``shared`` expert
     (``{"ff": n}``) that every token uses.  ``embed_scale`` (``embedding.scale``) multiplies the token embedding.
+    ``bigram`` (``embedding.bigram = {"buckets", "mul_prev", "mul_cur"}``) adds a row of a second table chosen by the
+    previous and the current token.  ``canon_taps`` (``canon.taps``; 0: none) puts a short causal convolution over time,
+    with a residual, between a sandwich block's input norms and its sublayers.  ``logit_scale`` multiplies the logits.
     """
 
     architecture: str = "Badapel"
@@ -297,6 +308,11 @@ class HybridConfig:
     moe: Optional[dict] = None
     embed_scale: float = 1.0
     dense_act: str = ""
+    bigram: Optional[dict] = None
+    canon_taps: int = 0
+    logit_scale: float = 1.0
+    depth_average: Optional[bool] = None
+    latent: Optional[dict] = None
 
     def __post_init__(self) -> None:
         traits = ARCHITECTURE_TRAITS.get(self.architecture, ARCHITECTURE_TRAITS["Badapel"])
@@ -312,7 +328,21 @@ class HybridConfig:
         self.attention = {**_ATTENTION_DEFAULT, **traits.get("attention", {}), **(self.attention or {})}
         self.moe = {**_MOE_DEFAULT, **traits.get("moe", {}), **(self.moe or {})}
         self.dense_act = self.dense_act or traits.get("dense_act", "gelu")
-        if self.dense_act not in ("gelu", "relu2"):
+        self.latent = {**_LATENT_DEFAULT, **traits.get("latent", {}), **(self.latent or {})}
+        if self.depth_average is None:
+            self.depth_average = bool(traits.get("depth_average", False))
+        if self.latent["rot"] not in ("halves", "pairs"):
+            raise ValueError(f"unknown latent attention variant: {self.latent}")
+        if self.bigram is not None:
+            if any(k not in self.bigram for k in ("buckets", "mul_prev", "mul_cur")) or int(self.bigram["buckets"]) < 1:
+                raise ValueError("embedding.bigram needs buckets >= 1, mul_prev and mul_cur")
+            if self.positions == "learned":
+                raise ValueError("a bigram embedding together with learned positions is not implemented")
+        if self.canon_taps < 0 or ((self.canon_taps or self.depth_average) and self.block != "sandwich"):
+            raise ValueError("input convolutions and the average over depth are implemented for sandwich blocks")
+        if self.depth_average and self.loop is not None:
+            raise ValueError("the average over depth counts layers once: it does not combine with a loop")
+        if self.dense_act not in ("gelu", "relu2", "polynorm"):
             raise ValueError(f"unknown dense feed-forward activation {self.dense_act!r}")
         if self.block not in ("sandwich", "prenorm", "parallel", "postnorm") or self.norm not in ("layer", "rms"):
             raise ValueError(f"unknown block {self.block!r} or norm {self.norm!r}")
@@ -353,13 +383,14 @@ class HybridConfig:
                 raise ValueError(f"layer {i}: heads must be a multiple of kv_heads")
             if kind == "lightning" and len(m["decay"]) != int(m["heads"]):
                 raise ValueError(f"layer {i}: one decay per head")
-            if kind == "attention" and m.get("kv_from") is not None:
+            if kind in ("attention", "latent_attention") and m.get("kv_from") is not None:
                 j = int(m["kv_from"])
                 src = self.layers[j] if 0 <= j < i else None
-                if src is None or src.get("type") != "attention" or src["mixer"].get("kv_from") is not None:
-                    raise ValueError(f"layer {i}: kv_from names an earlier attention layer with projections of its own")
-                if any(src["mixer"][k] != m[k] for k in ("kv_heads", "dim", "vdim")) or src["mixer"].get("rot") != m.get("rot"):
-                    raise ValueError(f"layer {i}: kv_from needs the source layer's kv_heads, dim, vdim and rotation")
+                if src is None or src.get("type") != kind or src["mixer"].get("kv_from") is not None:
+                    raise ValueError(f"layer {i}: kv_from names an earlier {kind} layer with projections of its own")
+                same = ("kv_heads", "dim", "vdim") if kind == "attention" else ("kv_rank", "rot_dim")  # what a cache row is made of
+                if any(src["mixer"][k] != m[k] for k in same) or src["mixer"].get("rot") != m.get("rot"):
+                    raise ValueError(f"layer {i}: kv_from needs the source layer's {', '.join(same)} and rotation")
         if self.loop is not None:
             a, b, t = self.loop["start"], self.loop["stop"], self.loop["times"]
             if not (0 <= a < b <= len(self.layers)) or t < 1:
@@ -399,7 +430,9 @@ class HybridConfig:
                    residual_mult=float(d.get("residual_mult", 1.0)),
                    token_side=dict(d["token_side"]) if d.get("token_side") else None,
                    max_positions=int(d.get("max_positions") or 0),
-                   embed_scale=float((d.get("embedding") or {}).get("scale", 1.0)))
+                   embed_scale=float((d.get("embedding") or {}).get("scale", 1.0)),
+                   bigram=dict(d["embedding"]["bigram"]) if (d.get("embedding") or {}).get("bigram") else None,
+                   canon_taps=int((d.get("canon") or {}).get("taps", 0)), logit_scale=float(d.get("logit_scale", 1.0)))
 
     @classmethod
     def from_file(cls, path: Union[str, Path]) -> "HybridConfig":
@@ -423,6 +456,12 @@ class HybridConfig:
             out["max_positions"] = self.max_positions
         if self.embed_scale != 1.0:
             out["embedding"] = {"scale": self.embed_scale}
+        if self.bigram is not None:
+            out.setdefault("embedding", {})["bigram"] = self.bigram
+        if self.canon_taps:
+            out["canon"] = {"taps": self.canon_taps}
+        if self.logit_scale != 1.0:
+            out["logit_scale"] = self.logit_scale
         return out
 
     def save(self, checkpoint_dir: Union[str, Path]) -> Path:

@@ -3,9 +3,9 @@
 Mixers (all written against the packed-batch operations of :mod:`mdi_llm_b200.ops.hybrid`):
 
 * :class:`LatentAttention` — softmax attention whose keys and values are expansions of one cached latent row per
-  token plus a rotated key part shared by the heads.  Only that row is cached; the query is carried into the latent
-  space (``q W_uk``) so that the attention kernel reads the cache directly, and the attended latent is expanded
-  by ``W_uv`` afterwards.
+  token plus a rotated key part shared by the heads.  Only that row is cached; on one-token steps the query is carried
+  into the latent space (``q W_uk``) so that the attention kernel reads the cache directly, and the attended latent is
+  expanded by ``W_uv`` afterwards.  Optional: a sliding window, another layer's cache instead of an own one.
 * :class:`GatedLinearAttention` — ``S_t = diag(a_t) S_(t-1) + k_t v_t^T`` with a data-dependent decay per key
   channel.
 * :class:`ChannelDelta` — the gated delta rule with a decay per key channel, short causal convolutions on q, k, v
@@ -19,7 +19,8 @@ Mixers (all written against the packed-batch operations of :mod:`mdi_llm_b200.op
 
 Feed-forwards: :class:`DenseFF` and :class:`MoEFF` (sigmoid router, top-k, the score scales the expert's *input*).
 
-A layer is a *sandwich* block (``x += norm_b(f(norm_a(x)))`` for the mixer and again for the feed-forward), a
+A layer is a *sandwich* block (``x += m norm_b(f(norm_a(x)))`` for the mixer and again for the feed-forward, optionally
+with a short convolution behind ``norm_a``, a gated per-layer token embedding and an average over depth), a
 *pre-norm* block (``x += m f(norm(x))``, optionally followed by a gated per-layer token embedding), a *parallel* block
 or a *post-norm* block (``x += norm(f(x))``: the sublayer reads the residual stream itself), chosen by the
 architecture (``config.block``), with the residual stream kept in fp32.  A span of layers may be looped; each pass owns its own state and starts by
@@ -90,6 +91,8 @@ class StatePool:
     of a recurrent layer owns ``state [slots, heads, dim, vdim]`` in fp32 and, with a short convolution,
     ``conv [slots, taps - 1, channels]``.  ``alloc`` hands out a slot with zeroed recurrent and convolution state
     (attention rows need no clearing: a row is written before any query can see it); ``free`` returns it.
+    An input convolution's runs own ``canon1`` / ``canon2 [slots, taps - 1, width]`` in fp32 (rows before a sequence's start are
+    never read), and a model with a bigram embedding keeps every slot's last token in ``prev [slots]``.
     The pool grows (doubling, contents kept) when more slots are asked for than it has.  A run of an attention layer
     that names ``kv_from`` owns nothing: its ``cache`` entry IS the cache of the latest earlier run of the layer it
     names (the same tensor), which that run has already extended by the step's tokens when this one reads it.
@@ -101,14 +104,24 @@ class StatePool:
         self.runs: List[Dict[str, torch.Tensor]] = [{} for _ in config.layer_runs()]
         self.free_slots: List[int] = []
         self.length: Dict[int, int] = {}
+        self.prev: Optional[torch.Tensor] = None
         self._grow(max(1, n_slots))
 
     def _shapes(self, spec: Dict[str, Any]) -> Dict[str, Tuple[Tuple[int, ...], torch.dtype]]:
+        out = self._mixer_shapes(spec)
+        if self.config.canon_taps > 1:
+            row = ((self.config.canon_taps - 1, self.config.width), torch.float32)
+            out["canon1"] = row
+            if spec.get("mlp"):
+                out["canon2"] = row
+        return out
+
+    def _mixer_shapes(self, spec: Dict[str, Any]) -> Dict[str, Tuple[Tuple[int, ...], torch.dtype]]:
         m = spec["mixer"]
+        if spec["type"] in ("attention", "latent_attention") and m.get("kv_from") is not None:
+            return {}
         if spec["type"] == "latent_attention":
             return {"cache": ((self.max_seq_length, m["kv_rank"] + m["rot_dim"]), self.dtype)}
-        if spec["type"] == "attention" and m.get("kv_from") is not None:
-            return {}
         if spec["type"] == "attention":  # one row per position: the kv_heads keys, then the kv_heads values
             return {"cache": ((self.max_seq_length, m["kv_heads"] * (m["dim"] + m["vdim"])), self.dtype)}
         out = {"state": ((m["heads"], m["dim"], m["vdim"]), torch.float32)}
@@ -124,9 +137,14 @@ class StatePool:
                 if key in run:
                     new[: self.n_slots] = run[key]
                 run[key] = new
+        if self.config.bigram is not None:
+            new = torch.zeros(n_slots, device=self.device, dtype=torch.int32)
+            if self.prev is not None:
+                new[: self.n_slots] = self.prev
+            self.prev = new
         order = self.config.layer_runs()
         for r, (li, _) in enumerate(order):
-            src = self.config.layers[li]["mixer"].get("kv_from") if self.config.layers[li]["type"] == "attention" else None
+            src = self.config.layers[li]["mixer"].get("kv_from")
             if src is not None:
                 owner = max(j for j in range(r) if order[j][0] == int(src))
                 self.runs[r]["cache"] = self.runs[owner]["cache"]
@@ -191,68 +209,107 @@ class _Fused:
 
 
 class LatentAttention(nn.Module, _Fused):
-    tensor_names = {"dq": "dq", "dq.norm": "dq_norm", "uq": "uq", "dkv": "dkv", "dkv.norm": "dkv_norm", "uk": "uk",
-                    "uv": "uv", "g": "g", "o": "o"}
+    """``traits`` (see ``models/config.py``) pick the pairing of the rotated entries, the sigmoid gate per output channel and
+    whether the prompt form keeps its softmax weights beyond the activation type's mantissa.  A mixer entry may name
+    ``mask.size`` (position ``i`` sees the last ``size`` positions up to its own) and ``kv_from``: the layer then has no ``dkv``,
+    it reads the latent and the rotated key part that layer cached, through its own ``uk`` and ``uv``."""
 
-    def __init__(self, width: int, m: Dict[str, Any], eps: float) -> None:
+    expand_from = 64   # prompts: sequences that bring at least this many tokens, or all of theirs, take the expanded form
+    query_block = 1024  # most rows of the score matrix alive at a time
+
+    def __init__(self, width: int, m: Dict[str, Any], eps: float, traits: Optional[Dict[str, Any]] = None) -> None:
         super().__init__()
+        t = {"rot": "halves", "gate": True, "p32": False, **(traits or {})}
         self.H, self.D, self.R, self.V = m["heads"], m["dim"], m["rot_dim"], m["vdim"]
         self.L, self.QR, self.scale, self.eps = m["kv_rank"], m["q_rank"], float(m["scale"]), eps
         self.nrot, self.rot_base = int(m["rot"]["dims"]), float(m["rot"]["base"])
         if self.nrot > self.R or self.nrot % 2:
             raise ValueError("rot.dims must be even and at most rot_dim")
+        self.window = int((m.get("mask") or {}).get("size", 0) or 0)
+        self.pairing, self.p32, self.borrows = str(t["rot"]), bool(t["p32"]), m.get("kv_from") is not None
         H_, D, R, V, L = self.H, self.D, self.R, self.V, self.L
         self.dq, self.dq_norm, self.uq = _param(self.QR, width), _param(self.QR), _param(H_ * (D + R), self.QR)
-        self.dkv, self.dkv_norm = _param(L + R, width), _param(L)
-        self.uk, self.uv = _param(H_ * D, L), _param(H_ * V, L)
-        self.g, self.o = _param(H_ * V, width), _param(width, H_ * V)
+        self.uk, self.uv, self.o = _param(H_ * D, L), _param(H_ * V, L), _param(width, H_ * V)
+        self.tensor_names = {"dq": "dq", "dq.norm": "dq_norm", "uq": "uq", "uk": "uk", "uv": "uv", "o": "o"}
+        self.dkv = self.dkv_norm = self.g = None
+        if not self.borrows:
+            self.dkv, self.dkv_norm = _param(L + R, width), _param(L)
+            self.tensor_names.update({"dkv": "dkv", "dkv.norm": "dkv_norm"})
+        if t["gate"]:
+            self.g = _param(H_ * V, width)
+            self.tensor_names["g"] = "g"
         self.inv_freq: Optional[torch.Tensor] = None
 
     def finalize(self) -> None:
-        self.fuse(("dq", "dkv", "g"))
+        self.fuse(("dq",) + (() if self.borrows else ("dkv",)) + (() if self.g is None else ("g",)))
         self.inv_freq = H.rotary_inv_freq(self.nrot, self.rot_base, self.dq.device)
+        # prompts expand a cached row [latent | rotated key part] into every head's whole key and value with ONE matrix
+        # product: the rotated part rides along through an identity block (a product with one is exact)
+        Hh, D, R, V, L = self.H, self.D, self.R, self.V, self.L
+        k = self.uk.data.new_zeros(Hh, D + R, L + R)
+        k[:, :D, :L] = self.uk.data.view(Hh, D, L)
+        k[:, D:, L:] = torch.eye(R, device=k.device, dtype=k.dtype)
+        v = self.uv.data.new_zeros(Hh * V, L + R)
+        v[:, :L] = self.uv.data
+        self.w_kv = torch.cat((k.view(Hh * (D + R), L + R), v), 0).contiguous()
+
+    def prompt_form(self, plan: H.BatchPlan) -> bool:
+        """Whether the step runs as matrix products over expanded keys and values: it brings a prompt or a long portion, and
+        no sequence that continues a long context with a few tokens."""
+        return max(n for _, n, _, _ in plan.seqs) >= self.expand_from and all(n >= self.expand_from or p0 == 0 for _, n, _, p0 in plan.seqs)
 
     def forward(self, h: torch.Tensor, plan: H.BatchPlan, st: Dict[str, torch.Tensor]) -> torch.Tensor:
         N = h.size(0)
         Hh, D, R, V, L = self.H, self.D, self.R, self.V, self.L
         p = H.linear(h, self.w_in)
-        cq = H.norm_rows(self.col(p, "dq"), self.dq_norm, None, self.eps, "rms", h.dtype)
+        cq = H.latent_prepare(self.col(p, "dq"), self.dq_norm, None if self.borrows else self.col(p, "dkv"), self.dkv_norm,
+                              self.inv_freq, st["cache"], plan, R, L, self.nrot, self.eps, self.pairing)
         q = H.linear(cq, self.uq)
-        H.latent_append(self.col(p, "dkv"), q, self.dkv_norm, self.inv_freq, st["cache"], plan, Hh, D, R, L, self.nrot, self.eps)
-        if min(n for _, n, _, _ in plan.seqs) >= self.expand_from:
+        if self.prompt_form(plan):
+            H.rotate_heads(q, self.inv_freq, plan, Hh, D, R, self.nrot, self.pairing)
             o = self._expanded(q, st["cache"], plan)
         else:
-            qlat = torch.bmm(q.view(N, Hh, D + R)[:, :, :D].transpose(0, 1), self.uk.view(Hh, D, L)).contiguous()
-            olat = H.latent_attn(qlat, q, st["cache"], plan, Hh, D, R, L, self.scale)
-            o = torch.bmm(olat, self.uv.view(Hh, V, L).transpose(1, 2)).contiguous()
-        return H.linear(H.headmajor_gate(o, self.col(p, "g")), self.o)
-
-    expand_from = 64   # a step whose every sequence brings at least this many tokens takes the expanded form
-    query_block = 1024  # rows of the score matrix alive at a time
+            qlat = H.matmul_f32(q.view(N, Hh, D + R)[:, :, :D].transpose(0, 1), self.uk.view(Hh, D, L))
+            olat = H.latent_attn(qlat, q, st["cache"], plan, Hh, D, R, L, self.scale, window=self.window, inv_freq=self.inv_freq,
+                                 nrot=self.nrot, pairing=self.pairing)
+            o = torch.empty(N, Hh, V, device=h.device, dtype=h.dtype)
+            torch.bmm(olat, self.uv.view(Hh, V, L).transpose(1, 2), out=o.transpose(0, 1))
+        o = o.view(N, Hh * V)
+        if self.g is not None:
+            o = H.headmajor_gate(o.unsqueeze(0), self.col(p, "g"))
+        return H.linear(o, self.o)
 
     def _expanded(self, q: torch.Tensor, cache: torch.Tensor, plan: H.BatchPlan) -> torch.Tensor:
-        """Prompt form: keys and values are expanded from the cached latents once per step (two matrix products),
-        scores and the weighted sum are batched matrix products over heads, the causal softmax runs on fp32 scores.
-        Decoding instead carries the query into the latent space and reads the cache directly (``H.latent_attn``):
-        per query that costs ``kv_rank`` instead of ``dim`` multiplies per key and head, which only pays when
-        there is a single query.  Returns ``[heads, N, vdim]``."""
-        Hh, D, R, V, L = self.H, self.D, self.R, self.V, self.L
-        out = torch.empty(Hh, q.size(0), V, device=q.device, dtype=q.dtype)
+        """Prompt form: keys and values are expanded from the cached rows once per step (one matrix product), scores and
+        the weighted sum are batched matrix products over heads, the masked softmax runs on fp32 scores in between, per
+        band of query rows against the keys the band can see.  Decoding instead carries the query into the latent space
+        and reads the cache directly (``H.latent_attn``): per query that costs ``kv_rank`` instead of ``dim`` multiplies per key
+        and head, which only pays when there is a single query.  Returns ``[N, heads, vdim]``."""
+        Hh, D, R, V, W = self.H, self.D, self.R, self.V, self.window
+        DK = D + R
+        out = torch.empty(q.size(0), Hh, V, device=q.device, dtype=q.dtype)
+        band = min(self.query_block, max(256, (W // 2 + 127) // 128 * 128)) if W > 0 else self.query_block
+        split = self.p32 and q.dtype != torch.float32  # weights as two 16-bit halves: the sum stays on the tensor cores
         for r0, n, slot, p0 in plan.seqs:
-            keys = p0 + n
-            rows = cache[slot, :keys]
-            lat = rows[:, :L]
-            k = torch.empty(Hh, D + R, keys, device=q.device, dtype=q.dtype)  # K^T per head: [unrotated | shared rotated]
-            k[:, :D] = H.linear(lat, self.uk).view(keys, Hh, D).permute(1, 2, 0)
-            k[:, D:] = rows[:, L:].t()
-            v = H.linear(lat, self.uv).view(keys, Hh, V).transpose(0, 1)  # [H, keys, V]
-            qh = q[r0:r0 + n].view(n, Hh, D + R).transpose(0, 1)  # [H, n, D+R]
-            for a in range(0, n, self.query_block):
-                b = min(n, a + self.query_block)
-                vis = p0 + b  # keys any row of this block can see
-                s = H.matmul_f32(qh[:, a:b], k[:, :, :vis]).contiguous()
-                pr = H.causal_softmax(s, p0 + a, self.scale, q.dtype)
-                out[:, r0 + a:r0 + b] = torch.bmm(pr, v[:, :vis])
+            first = max(0, p0 - W + 1) if W > 0 else 0
+            kv = H.linear(cache[slot, first:p0 + n], self.w_kv)
+            keys = kv.size(0)
+            kt = kv[:, :Hh * DK].view(keys, Hh, DK).permute(1, 2, 0)   # [H, D+R, keys]
+            v = kv[:, Hh * DK:].view(keys, Hh, V).transpose(0, 1)      # [H, keys, V]
+            qh = q[r0:r0 + n].view(n, Hh, DK).transpose(0, 1)          # [H, n, D+R]
+            for a in range(0, n, band):
+                b = min(n, a + band)
+                k1 = p0 + b - first
+                k0 = max(0, p0 + a - W + 1 - first) if W > 0 else 0
+                k0 = max(0, k0 - (k0 - k1) % 8)  # a few hidden keys in front: rows of whole 16-byte groups
+                s = H.matmul_f32(qh[:, a:b], kt[:, :, k0:k1]).contiguous()
+                pr = H.causal_softmax(s, p0 + a, self.scale, q.dtype, window=W, key0=first + k0, split=split)
+                vv = v[:, k0:k1]
+                dst = out[r0 + a:r0 + b].transpose(0, 1)
+                if split:
+                    dst.copy_(H.matmul_f32(pr, torch.cat((vv, vv), 1)))
+                else:
+                    torch.bmm(pr, vv, out=dst)
         return out
 
 
@@ -633,15 +690,27 @@ class MoEFF(nn.Module):
 
 
 class DenseFF(nn.Module):
-    tensor_names = {"up": "up", "down": "down"}
+    """``down act(up h)``.  ``act="polynorm"`` has four learned numbers (tensor ``act``) and norms over the ``ff`` values with
+    ``eps``, see :func:`mdi_llm_b200.ops.hybrid.poly_norm`."""
 
-    def __init__(self, width: int, ff: int, act: str = "gelu") -> None:
+    def __init__(self, width: int, ff: int, act: str = "gelu", eps: float = 1e-6) -> None:
         super().__init__()
-        self.act = act
+        self.act, self.eps = act, eps
         self.up, self.down = _param(ff, width), _param(width, ff)
+        self.tensor_names = {"up": "up", "down": "down"}
+        self.coef = self.coef32 = None
+        if act == "polynorm":
+            self.coef = _param(4)
+            self.tensor_names["act"] = "coef"
+
+    def finalize(self) -> None:
+        if self.coef is not None:
+            self.coef32 = self.coef.data.float().contiguous()
 
     def forward(self, h: torch.Tensor) -> torch.Tensor:
         a = H.linear(h, self.up)
+        if self.coef32 is not None:
+            return H.linear(H.poly_norm(a, self.coef32, self.eps), self.down)
         return H.linear(H.relu2_(a) if self.act == "relu2" else H.gelu_(a), self.down)
 
 
@@ -652,27 +721,74 @@ class _LN(nn.Module):
 
 
 class SandwichBlock(nn.Module):
-    """``x += norm1b(mixer(norm1(x)))``, then ``x += norm2b(ff(norm2(x)))`` when the layer has a feed-forward."""
+    """``x += m norm1b(mixer(norm1(x)))``, then ``x += m norm2b(ff(norm2(x)))`` when the layer has a feed-forward, then the
+    gated per-layer token embedding when the model has one (``side``).
 
-    def __init__(self, width: int, mixer: nn.Module, ff: Optional[nn.Module], eps: float) -> None:
+    ``taps`` > 0: what a sublayer reads is ``h + conv(h)`` with ``h`` the normed rows and ``conv`` a causal convolution over time
+    per channel (tensors ``canon1`` / ``canon2 [width, taps]``), whose last inputs are part of a slot's state.  ``index`` (the
+    layer's number, with an average over depth): ``x`` is row ``index + 1`` of the step's ``depth`` rows, and what the layer passes
+    on, ``sum_j dwa[j] depth[j]`` over the embedding output and every result up to its own, is written to the next row.
+
+    Every update of the stream is one kernel that adds the normed output, keeps the rounded copy the token embedding's
+    gate reads, takes the average over depth and, on steps of one token per sequence, goes on to the norm and the
+    convolution of the next sublayer (the next block's, when ``follower`` names it)."""
+
+    def __init__(self, width: int, mixer: nn.Module, ff: Optional[nn.Module], eps: float, mult: float = 1.0,
+                 side: Optional["TokenSide"] = None, taps: int = 0, index: Optional[int] = None) -> None:
         super().__init__()
-        self.mix, self.mlp, self.eps = mixer, ff, eps
+        self.mix, self.mlp, self.eps, self.mult, self.side, self.index = mixer, ff, eps, float(mult), side, index
         self.norm1, self.norm1b = _LN(width), _LN(width)
+        self.canon1 = _param(width, taps) if taps else None
+        self.canon2 = _param(width, taps) if taps and ff is not None else None
         if ff is not None:
             self.norm2, self.norm2b = _LN(width), _LN(width)
-
-    side = None
+        self.dwa = _param(index + 2) if index is not None else None
+        self.conv1 = self.conv2 = self.depth_w = None  # fp32 forms, made by finalize
+        self.follower: Tuple["SandwichBlock", ...] = ()  # a tuple: the next block is not a submodule of this one
 
     def norm_names(self) -> List[str]:
         return ["norm1", "norm1b"] + (["norm2", "norm2b"] if self.mlp is not None else [])
 
+    def extra_tensors(self) -> Dict[str, nn.Parameter]:
+        return {k: getattr(self, k) for k in ("canon1", "canon2", "dwa") if getattr(self, k) is not None}
+
+    def finalize(self) -> None:
+        if self.canon1 is not None:
+            self.conv1 = self.canon1.data.float().t().contiguous()
+        if self.canon2 is not None:
+            self.conv2 = self.canon2.data.float().t().contiguous()
+        if self.dwa is not None:
+            self.depth_w = self.dwa.data.float().contiguous()
+
+    def _input1(self, st: Dict[str, torch.Tensor]) -> H.NextInput:
+        return H.NextInput(self.norm1.w, self.norm1.b, self.eps, "layer", self.conv1, st.get("canon1"))
+
+    def _input2(self, st: Dict[str, torch.Tensor]) -> H.NextInput:
+        return H.NextInput(self.norm2.w, self.norm2.b, self.eps, "layer", self.conv2, st.get("canon2"))
+
     def forward(self, x: torch.Tensor, plan: H.BatchPlan, st: Dict[str, torch.Tensor], dtype: torch.dtype,
-                tokens: Optional[torch.Tensor] = None, side_table: Optional[torch.Tensor] = None) -> None:
-        h = H.norm_rows(x, self.norm1.w, self.norm1.b, self.eps, "layer", dtype)
-        H.norm_accumulate(x, self.mix(h, plan, st), self.norm1b.w, self.norm1b.b, self.eps)
+                tokens: Optional[torch.Tensor] = None, side_table: Optional[torch.Tensor] = None,
+                next_st: Optional[Dict[str, torch.Tensor]] = None) -> None:
+        """``next_st``: the state of the layer run that follows, for the input of its first sublayer."""
+        one, depth = plan.one_token, plan.shared.get("depth")
+        h = plan.shared.pop("sublayer_input", None)  # left by the previous block's last update
+        if h is None:
+            h = H.norm_conv(x, self._input1(st), plan, dtype)
+        y, w, b = self.mix(h, plan, st), self.norm1b.w, self.norm1b.b
         if self.mlp is not None:
-            h = H.norm_rows(x, self.norm2.w, self.norm2.b, self.eps, "layer", dtype)
-            H.norm_accumulate(x, self.mlp(h), self.norm2b.w, self.norm2b.b, self.eps)
+            nxt = self._input2(st)
+            h = H.row_update(x, y, w, b, self.eps, "layer", self.mult, nxt=nxt if one else None, plan=plan, out_dtype=dtype)
+            y, w, b = self.mlp(H.norm_conv(x, nxt, plan, dtype) if h is None else h), self.norm2b.w, self.norm2b.b
+        kind = "layer"
+        if self.side is not None:
+            xa = x if dtype == torch.float32 else torch.empty(x.shape, device=x.device, dtype=dtype)
+            H.row_update(x, y, w, b, self.eps, "layer", self.mult, copy=None if xa is x else xa)
+            y, w, b, kind = self.side.output(xa, tokens, side_table), self.side.norm, None, "rms"
+        nxt = self.follower[0]._input1(next_st) if one and self.follower and next_st is not None else None
+        h = H.row_update(x, y, w, b, self.eps, kind, self.mult, depth=depth, index=0 if self.index is None else self.index + 1,
+                         depth_w=self.depth_w, nxt=nxt, plan=plan, out_dtype=dtype)
+        if h is not None:
+            plan.shared["sublayer_input"] = h
 
 
 class _RMS(nn.Module):
@@ -690,12 +806,15 @@ class TokenSide(nn.Module):
         self.dim, self.col0 = dim, col0
         self.gate, self.proj, self.norm = _param(dim, width), _param(width, dim), _param(width)
 
+    def output(self, xa: torch.Tensor, tokens: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
+        """``y`` from the stream in the activation type, before its norm."""
+        return H.linear(H.token_side_gate(H.linear(xa, self.gate), table, tokens, self.col0), self.proj)
+
     def forward(self, x: torch.Tensor, tokens: torch.Tensor, table: torch.Tensor, eps: float, m: float, dtype: torch.dtype) -> None:
         xa = x if dtype == torch.float32 else torch.empty(x.shape, device=x.device, dtype=dtype)
         if xa is not x:
             H.cast_into(x, xa)
-        g = H.token_side_gate(H.linear(xa, self.gate), table, tokens, self.col0)
-        H.norm_accumulate(x, H.linear(g, self.proj), self.norm, None, eps, "rms", m)
+        H.norm_accumulate(x, self.output(xa, tokens, table), self.norm, None, eps, "rms", m)
 
 
 class PreNormBlock(nn.Module):
@@ -888,7 +1007,7 @@ class HybridLM(nn.Module):
         for i, spec in enumerate(config.layers):
             m, kind = spec["mixer"], spec["type"]
             if kind == "latent_attention":
-                mixer: nn.Module = LatentAttention(C, m, eps)
+                mixer: nn.Module = LatentAttention(C, m, eps, config.latent)
             elif kind == "attention":
                 mixer = WindowAttention(C, m, eps, config.attention)
             elif kind == "lightning":
@@ -907,18 +1026,23 @@ class HybridLM(nn.Module):
                            int(mlp["router"].get("identity", 0) or 0), float(mlp["expert"].get("limit", 0.0)),
                            float(sh.get("limit", 0.0)), bool(config.moe["shared_gate"]))
             else:
-                ff = DenseFF(C, mlp["ff"], config.dense_act)
+                ff = DenseFF(C, mlp["ff"], config.dense_act, eps)
+            sd = int(config.token_side["dim"]) if config.token_side else 0
+            side = TokenSide(C, sd, i * sd) if sd and config.block in ("sandwich", "prenorm") else None
             if config.block == "sandwich":
-                blocks.append(SandwichBlock(C, mixer, ff, eps))
+                blocks.append(SandwichBlock(C, mixer, ff, eps, config.residual_mult, side, config.canon_taps,
+                                            i if config.depth_average else None))
             elif config.block == "parallel":
                 blocks.append(ParallelBlock(C, mixer, ff, eps, config.norm, config.norm_offset, config.layer_scale))
             elif config.block == "postnorm":
                 blocks.append(PostNormBlock(C, mixer, ff, eps, config.norm))
             else:
-                sd = int(config.token_side["dim"]) if config.token_side else 0
-                side = TokenSide(C, sd, i * sd) if sd else None
                 blocks.append(PreNormBlock(C, mixer, ff, eps, config.norm, config.residual_mult, side))
         self.blocks = nn.ModuleList(blocks)
+        if config.block == "sandwich" and config.loop is None:
+            for blk, nxt in zip(blocks, blocks[1:]):
+                blk.follower = (nxt,)
+        self.bigram = _param(int(config.bigram["buckets"]) + 1, C) if config.bigram is not None else None
         self.final_norm = _LN(C) if config.norm == "layer" else _RMS(C)
         self.side_embed = _param(config.vocab, len(config.layers) * int(config.token_side["dim"])) if config.token_side else None
         self.head_w = None if config.tied_head else _param(config.vocab, C)
@@ -934,6 +1058,8 @@ class HybridLM(nn.Module):
             out["loop.in"] = self.loop_in
         if self.pos is not None:
             out["pos"] = self.pos
+        if self.bigram is not None:
+            out["bigram"] = self.bigram
         if self.side_embed is not None:
             out["side.embed"] = self.side_embed
         if self.head_w is not None:
@@ -960,9 +1086,9 @@ class HybridLM(nn.Module):
 
     def load_tensors(self, tensors: Dict[str, torch.Tensor], device: Union[str, torch.device], dtype: torch.dtype) -> "HybridLM":
         tm = self.tensor_map()
-        # a checkpoint may carry tensors a layer has no use for (a mixing factor where nothing is mixed, the scale of
-        # a feed-forward the layer does not have)
-        unused = (".mix.vmix", ".ls2")
+        # a checkpoint may carry tensors a layer has no use for (a mixing factor where nothing is mixed; the scale, norms or
+        # convolution of a feed-forward the layer does not have)
+        unused = (".mix.vmix", ".ls2", ".norm2", ".norm2.b", ".norm2b", ".norm2b.b", ".canon2")
         missing = sorted(set(tm) - set(tensors))
         extra = sorted(n for n in set(tensors) - set(tm) if not n.endswith(unused))
         if missing or extra:
@@ -1004,9 +1130,9 @@ class HybridLM(nn.Module):
     def finalize(self) -> "HybridLM":
         for blk in self.blocks:
             blk.mix.finalize()
-            if isinstance(blk.mlp, (MoEFF, GatedFF)):
+            if isinstance(blk.mlp, (MoEFF, GatedFF, DenseFF)):
                 blk.mlp.finalize()
-            if isinstance(blk, ParallelBlock):
+            if isinstance(blk, (ParallelBlock, SandwichBlock)):
                 blk.finalize()
         self.dtype, self.device = self.embed.dtype, self.embed.device
         return self
@@ -1029,7 +1155,20 @@ class HybridLM(nn.Module):
             if self.pos is not None and p0 + n > self.pos.size(0):
                 raise ValueError(f"sequence of {p0 + n} tokens exceeds the model's {self.pos.size(0)} learned positions")
         plan.shared.clear()
-        x0 = H.embed_rows(self.embed, tokens, self.pos, plan, self.config.embed_scale)
+        cfg, n_runs = self.config, len(self.runs)
+        depth = None
+        if cfg.depth_average:  # row 0: the embedding output; row i + 1: layer i's stream; the last row: what goes to the output
+            depth = torch.empty(n_runs + 2, tokens.numel(), C, device=self.device, dtype=torch.float32)
+            plan.shared["depth"] = depth
+        if self.bigram is not None:
+            g = cfg.bigram
+            x0 = H.embed_pairs(self.embed, self.bigram, tokens, plan, pool.prev, g["buckets"], g["mul_prev"], g["mul_cur"],
+                               cfg.embed_scale, None if depth is None else depth[0], None if depth is None else depth[1])
+        else:
+            x0 = H.embed_rows(self.embed, tokens, self.pos, plan, cfg.embed_scale)
+            if depth is not None:
+                depth[0].copy_(x0)
+                depth[1].copy_(x0)
         x = x0.clone() if self.loop_in is not None else x0
         for run, (li, first) in enumerate(self.runs):
             if first:
@@ -1042,17 +1181,26 @@ class HybridLM(nn.Module):
                     x = y
                 else:
                     H.cast_into(y, x)
-            self.blocks[li](x, plan, pool.runs[run], dt, tokens, self.side_embed)
+            if depth is not None:
+                x = depth[run + 1]
+            blk = self.blocks[li]
+            if isinstance(blk, SandwichBlock):
+                blk(x, plan, pool.runs[run], dt, tokens, self.side_embed, pool.runs[run + 1] if run + 1 < n_runs else None)
+            else:
+                blk(x, plan, pool.runs[run], dt, tokens, self.side_embed)
+            if depth is not None:
+                x = depth[run + 2]
             if trace is not None:
                 trace.append(x.clone())
         return x
 
     @torch.inference_mode()
     def head(self, x: torch.Tensor) -> torch.Tensor:
-        """fp32 logits of residual rows ``x [n, width]``: final norm, output head (tied or its own), soft cap."""
+        """fp32 logits of residual rows ``x [n, width]``: final norm, output head (tied or its own), scale, soft cap."""
         h = H.norm_rows(x, self.final_norm.w, self.final_norm.b, self.config.norm_eps, self.config.norm, self.dtype,
                         self.config.norm_offset)
-        return H.softcap(H.linear(h, self.embed if self.head_w is None else self.head_w), self.config.logit_softcap)
+        return H.softcap(H.linear(h, self.embed if self.head_w is None else self.head_w), self.config.logit_softcap,
+                         self.config.logit_scale)
 
     def forward(self, tokens: torch.Tensor, plan: H.BatchPlan, pool: StatePool, rows: Optional[Sequence[int]] = None,
                 trace: Optional[List[torch.Tensor]] = None) -> torch.Tensor:

@@ -30,10 +30,11 @@ def nvcc_path() -> Optional[str]:
 
 
 # The hybrid model family's kernels are a library of their own (``_mdi_hybrid.so``): a checkout that only serves
-# such a model compiles one file, and that file is built with IEEE math (no ``--use_fast_math``) because its
+# such a model compiles these files only, and they are built with IEEE math (no ``--use_fast_math``) because its
 # 32-bit mode is held to 32-bit rounding.
 HYBRID_LIB = HERE / "_mdi_hybrid.so"
-HYBRID_SOURCES = ("hybrid_mixers.cu",)
+HYBRID_SOURCES = ("hybrid_mixers.cu", "hybrid_rows.cu")
+HYBRID_HEADERS = ("hybrid_common.cuh",)
 
 
 def sources() -> List[Path]:
@@ -43,7 +44,8 @@ def sources() -> List[Path]:
 def _digest() -> str:
     h = hashlib.sha256()
     files = [p for p in CSRC.glob("*.cu") if p.name not in HYBRID_SOURCES]
-    for p in sorted(files + list(CSRC.glob("*.cuh")) + [Path(__file__)]):
+    headers = [p for p in CSRC.glob("*.cuh") if p.name not in HYBRID_HEADERS]
+    for p in sorted(files + headers + [Path(__file__)]):
         h.update(p.name.encode())
         h.update(p.read_bytes())
     return h.hexdigest()
@@ -51,7 +53,7 @@ def _digest() -> str:
 
 def _hybrid_digest() -> str:
     h = hashlib.sha256()
-    for name in HYBRID_SOURCES:
+    for name in HYBRID_SOURCES + HYBRID_HEADERS:
         h.update(name.encode())
         h.update((CSRC / name).read_bytes())
     return h.hexdigest()
@@ -70,7 +72,7 @@ def build_hybrid(force: bool = False, ptxas_info: bool = False) -> Path:
         raise RuntimeError("nvcc not found: cannot build the sm_100a kernels")
     digest = _hybrid_digest()
     tmp = HYBRID_LIB.with_suffix(f".{os.getpid()}.tmp.so")
-    cmd = [nvcc, "-O3", "-std=c++17", "-lineinfo", *ARCH_FLAGS, "-Xcompiler", "-fPIC", "-shared",
+    cmd = [nvcc, "-O3", "-std=c++17", "-lineinfo", *ARCH_FLAGS, "-Xcompiler", "-fPIC", "-shared", "-t", str(len(HYBRID_SOURCES)),
            f'-DMDI_BUILD_DIGEST_STR="{digest}"', *(["-Xptxas", "-v"] if ptxas_info else []),
            *[str(CSRC / n) for n in HYBRID_SOURCES], "-o", str(tmp), "-lcudart"]
     r = subprocess.run(cmd, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)

@@ -6,78 +6,9 @@
 // the meta table.  Every kernel is templated on the activation type (bf16 or fp32); sums, norms, softmax, decays
 // and recurrent state are fp32 in both.  This file is compiled WITHOUT fast-math: its exponentials, divisions and
 // square roots are the IEEE ones.
-#include <cuda_bf16.h>
-#include <cuda_runtime.h>
-#include <math.h>
-#include <stdint.h>
+#include "hybrid_common.cuh"
 
 namespace hyb {
-
-typedef __nv_bfloat16 bf16;
-
-__device__ __forceinline__ float to_f(float v) { return v; }
-__device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
-template <typename T> __device__ __forceinline__ T from_f(float v);
-template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
-template <> __device__ __forceinline__ bf16 from_f<bf16>(float v) { return __float2bfloat16_rn(v); }
-
-__device__ __forceinline__ void load8(const float* p, float* f) {
-  float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
-}
-__device__ __forceinline__ void load8(const bf16* p, float* f) {
-  uint4 u = *reinterpret_cast<const uint4*>(p);
-  const uint32_t w[4] = {u.x, u.y, u.z, u.w};
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    f[2 * i] = __uint_as_float(w[i] << 16);
-    f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
-  }
-}
-
-__device__ __forceinline__ void store8(float* p, const float* f) {
-  *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
-  *reinterpret_cast<float4*>(p + 4) = make_float4(f[4], f[5], f[6], f[7]);
-}
-__device__ __forceinline__ void store8(bf16* p, const float* f) {
-  uint32_t w[4];
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    __nv_bfloat162 h = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]);
-    w[i] = *reinterpret_cast<uint32_t*>(&h);
-  }
-  *reinterpret_cast<uint4*>(p) = make_uint4(w[0], w[1], w[2], w[3]);
-}
-
-__device__ __forceinline__ float warp_sum(float v) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-  return v;
-}
-__device__ __forceinline__ float warp_max(float v) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
-  return v;
-}
-// Sum over the block; every thread gets the result.  `red` holds 33 floats.  Safe to call back to back.
-__device__ __forceinline__ float block_sum(float v, float* red) {
-  int lane = threadIdx.x & 31, w = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
-  v = warp_sum(v);
-  __syncthreads();
-  if (lane == 0) red[w] = v;
-  __syncthreads();
-  if (w == 0) {
-    float t = lane < nw ? red[lane] : 0.f;
-    t = warp_sum(t);
-    if (lane == 0) red[32] = t;
-  }
-  __syncthreads();
-  return red[32];
-}
-__device__ __forceinline__ float sigmoidf_(float x) { return 1.f / (1.f + expf(-x)); }
-__device__ __forceinline__ float softplusf_(float x) { return x > 20.f ? x : log1pf(expf(x)); }
-__device__ __forceinline__ float siluf_(float x) { return x / (1.f + expf(-x)); }
-__device__ __forceinline__ float gelu_erff_(float x) { return 0.5f * x * (1.f + erff(x * 0.70710678118654752f)); }
 
 // ---------------------------------------------------------------------------------------------------------
 // rows: embedding gather, casts, norms, element-wise epilogues
@@ -176,10 +107,10 @@ __global__ void headmajor_gate_kernel(const T* __restrict__ a, const T* __restri
   }
 }
 template <typename T>
-__global__ void softcap_kernel(const T* __restrict__ in, float* __restrict__ out, long long total, float cap) {
+__global__ void softcap_kernel(const T* __restrict__ in, float* __restrict__ out, long long total, float cap, float scale) {
   long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (i < total) {
-    float v = to_f(in[i]);
+    float v = to_f(in[i]) * scale;
     out[i] = cap > 0.f ? cap * tanhf(v / cap) : v;
   }
 }
@@ -187,77 +118,154 @@ __global__ void softcap_kernel(const T* __restrict__ in, float* __restrict__ out
 // ---------------------------------------------------------------------------------------------------------
 // latent attention: cache append (norm + rotary) and attention over the shared latent rows
 // ---------------------------------------------------------------------------------------------------------
-// One block per token.  The row `ckv` holds [L latent | R rotary key]: the latent is RMS-normed with `w`, the key
-// part is rotated for the token's position; both go to cache[slot, pos].  The rotary part of each query head
-// (last R of its D + R values) is rotated in place.  Pair (i, i + nrot/2), angle = pos * inv_freq[i].
+// Rotation of entry r of a vector's first nrot entries by ang(pair) = pos * inv_freq[pair]: pairs (i, i + nrot/2)
+// (halves), or neighbours (2i, 2i+1) (interleaved).
+__device__ __forceinline__ void rot_pair(int i, int nrot, int interleaved, int& a, int& b) {
+  a = interleaved ? 2 * i : i;
+  b = interleaved ? 2 * i + 1 : i + nrot / 2;
+}
+
+// What both sides of latent attention need of a token's input projection, one block per token: cq = RMS norm of the
+// query latent dq [Q] with weight qw, and (ckv != null) the cache row [L latent, RMS-normed with w | R shared key part,
+// rotated for the token's position].  A layer that reads another layer's cache has no ckv.
 template <typename T>
-__global__ void latent_append_kernel(const T* __restrict__ ckv, long long ckv_stride, T* __restrict__ q,
-                                     long long q_stride, const T* __restrict__ w, const float* __restrict__ inv_freq,
-                                     T* __restrict__ cache, long long slot_stride, const int* __restrict__ meta,
-                                     const int* __restrict__ tok_seq, int H, int D, int R, int L, int nrot, float eps) {
-  __shared__ float red[33];
+__global__ void __launch_bounds__(256) latent_prepare_kernel(const T* __restrict__ dq, long long dq_stride, const T* __restrict__ qw,
+                                                             T* __restrict__ cq, int Q, const T* __restrict__ ckv,
+                                                             long long ckv_stride, const T* __restrict__ w,
+                                                             const float* __restrict__ inv_freq, T* __restrict__ cache,
+                                                             long long slot_stride, const int* __restrict__ meta,
+                                                             const int* __restrict__ tok_seq, int R, int L, int nrot,
+                                                             int interleaved, float eps, int vec) {
+  __shared__ float red[2][8];
   int tok = blockIdx.x;
+  const T* qs = dq + (size_t)tok * dq_stride;
+  const T* src = ckv ? ckv + (size_t)tok * ckv_stride : nullptr;
+  float s1 = 0.f, s2 = 0.f;
+  if (vec) {
+    float f[8];
+    for (int i = threadIdx.x * 8; i < Q; i += blockDim.x * 8) {
+      load8(qs + i, f);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) s1 += f[e] * f[e];
+    }
+    if (src)
+      for (int i = threadIdx.x * 8; i < L; i += blockDim.x * 8) {
+        load8(src + i, f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) s2 += f[e] * f[e];
+      }
+  } else {
+    for (int i = threadIdx.x; i < Q; i += blockDim.x) { float v = to_f(qs[i]); s1 += v * v; }
+    if (src)
+      for (int i = threadIdx.x; i < L; i += blockDim.x) { float v = to_f(src[i]); s2 += v * v; }
+  }
+  s1 = warp_sum(s1);
+  s2 = warp_sum(s2);
+  if ((threadIdx.x & 31) == 0) { red[0][threadIdx.x >> 5] = s1; red[1][threadIdx.x >> 5] = s2; }
+  __syncthreads();
+  s1 = s2 = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) { s1 += red[0][i]; s2 += red[1][i]; }
+  const float i1 = 1.f / sqrtf(s1 / Q + eps);
+  T* co = cq + (size_t)tok * Q;
+  auto apply = [&](const T* in, const T* wt, T* o, int n, float inv) {
+    if (vec) {
+      float f[8], g[8];
+      for (int i = threadIdx.x * 8; i < n; i += blockDim.x * 8) {
+        load8(in + i, f);
+        load8(wt + i, g);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] = f[e] * inv * g[e];
+        store8(o + i, f);
+      }
+    } else {
+      for (int i = threadIdx.x; i < n; i += blockDim.x) o[i] = from_f<T>(to_f(in[i]) * inv * to_f(wt[i]));
+    }
+  };
+  apply(qs, qw, co, Q, i1);
+  if (!src) return;
   const int* m = meta + 4 * tok_seq[tok];
   int pos = m[3] + tok - m[0];
-  const T* src = ckv + (size_t)tok * ckv_stride;
   T* dst = cache + (size_t)m[2] * slot_stride + (size_t)pos * (L + R);
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < L; i += blockDim.x) {
-    float v = to_f(src[i]);
-    ss += v * v;
+  apply(src, w, dst, L, 1.f / sqrtf(s2 / L + eps));
+  for (int i = threadIdx.x; i < nrot / 2; i += blockDim.x) {
+    int a, b;
+    rot_pair(i, nrot, interleaved, a, b);
+    float sn, cs;
+    sincosf((float)pos * inv_freq[i], &sn, &cs);
+    float u = to_f(src[L + a]), v = to_f(src[L + b]);
+    dst[L + a] = from_f<T>(u * cs - v * sn);
+    dst[L + b] = from_f<T>(v * cs + u * sn);
   }
-  float inv = 1.f / sqrtf(block_sum(ss, red) / L + eps);
-  for (int i = threadIdx.x; i < L; i += blockDim.x) dst[i] = from_f<T>(to_f(src[i]) * inv * to_f(w[i]));
-  int half = nrot / 2;
-  // work items: (H + 1) vectors (vector H is the shared key part) x (half pairs, then the R - nrot values that pass);
-  // one thread owns both members of a pair, so the in-place rotation of q needs no barrier
-  int per = half + (R - nrot);
-  for (int idx = threadIdx.x; idx < (H + 1) * per; idx += blockDim.x) {
-    int vec = idx / per, i = idx - vec * per;
-    T* qd = q + (size_t)tok * q_stride + (size_t)vec * (D + R) + D;
-    const T* s = vec < H ? qd : src + L;
-    T* d = vec < H ? qd : dst + L;
-    if (i < half) {
-      float sn, cs;
-      sincosf((float)pos * inv_freq[i], &sn, &cs);
-      float u = to_f(s[i]), v = to_f(s[i + half]);
-      d[i] = from_f<T>(u * cs - v * sn);
-      d[i + half] = from_f<T>(v * cs + u * sn);
-    } else if (vec == H) {
-      d[nrot + i - half] = s[nrot + i - half];
-    }
+  for (int i = nrot + threadIdx.x; i < R; i += blockDim.x) dst[L + i] = src[L + i];
+}
+
+// The last R entries of each of the H heads (D + R wide) of every row of q are rotated in place; a thread owns both
+// members of a pair.  The angles of a token are evaluated once and shared by its heads.
+template <typename T>
+__global__ void rotate_heads_kernel(T* __restrict__ q, long long q_stride, const float* __restrict__ inv_freq,
+                                    const int* __restrict__ meta, const int* __restrict__ tok_seq, int H, int D, int R,
+                                    int nrot, int interleaved) {
+  extern __shared__ float cssn[];  // [nrot/2] cosines, [nrot/2] sines
+  int tok = blockIdx.x, half = nrot / 2;
+  const int* m = meta + 4 * tok_seq[tok];
+  float pos = (float)(m[3] + tok - m[0]);
+  for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(pos * inv_freq[i], &cssn[half + i], &cssn[i]);
+  __syncthreads();
+  for (int idx = threadIdx.x; idx < H * half; idx += blockDim.x) {
+    int h = idx / half, i = idx - h * half, a, b;
+    rot_pair(i, nrot, interleaved, a, b);
+    T* d = q + (size_t)tok * q_stride + (size_t)h * (D + R) + D;
+    float u = to_f(d[a]), v = to_f(d[b]), cs = cssn[i], sn = cssn[half + i];
+    d[a] = from_f<T>(u * cs - v * sn);
+    d[b] = from_f<T>(v * cs + u * sn);
   }
 }
 
 // Attention of H query heads over ONE shared key row per position, whose first Dv entries are also the value
 // (queries arrive already multiplied into the latent space).  Block = one token x 8 heads, one warp per head;
 // a tile of 32 cached rows is staged in shared memory once and used by all 8 heads.  Online softmax in fp32.
+// window > 0: a token sees the last `window` positions up to its own.  qlat is fp32.  inv_freq != null: the rotary part
+// of the query (read from q) is rotated for the token's position as it is loaded.
 #define LAT_WARPS 8
 #define LAT_TILE 32
-#define LAT_MAXV 16  // Dv <= 512
-template <typename T>
-__global__ void latent_attn_kernel(const T* __restrict__ qlat, const T* __restrict__ q, long long q_stride,
+template <typename T, int LAT_MAXV>  // Dv <= 32 * LAT_MAXV
+__global__ void latent_attn_kernel(const float* __restrict__ qlat, const T* __restrict__ q, long long q_stride,
                                    const T* __restrict__ cache, long long slot_stride, const int* __restrict__ meta,
                                    const int* __restrict__ tok_seq, T* __restrict__ out, int N, int H, int D, int R,
                                    int L, float scale, int nsplit, float* __restrict__ part_acc,
-                                   float* __restrict__ part_ml) {
+                                   float* __restrict__ part_ml, int window, const float* __restrict__ inv_freq, int nrot,
+                                   int interleaved) {
   extern __shared__ float smem[];
   int Dk = L + R, ldk = Dk + 1;
   float* sq = smem;                       // [LAT_WARPS][Dk]
   float* kt = smem + LAT_WARPS * Dk;      // [LAT_TILE][ldk]
   int tok = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int* m = meta + 4 * tok_seq[tok];
-  int nkeys = m[3] + tok - m[0] + 1;
+  int pos = m[3] + tok - m[0], first = window > 0 ? max(0, pos - window + 1) : 0, nkeys = pos + 1 - first;
   int h = blockIdx.y * LAT_WARPS + warp;
   bool active = h < H;
   if (active) {
     for (int d = lane; d < Dk; d += 32) {
-      float v = d < L ? to_f(qlat[((size_t)h * N + tok) * L + d])
-                      : to_f(q[(size_t)tok * q_stride + (size_t)h * (D + R) + D + (d - L)]);
+      float v;
+      if (d < L) {
+        v = qlat[((size_t)h * N + tok) * L + d];
+      } else {
+        const T* qr = q + (size_t)tok * q_stride + (size_t)h * (D + R) + D;
+        int r = d - L;
+        v = to_f(qr[r]);
+        if (inv_freq && r < nrot) {  // this entry and its partner: (u, v) -> (u cos - v sin, v cos + u sin)
+          int half = nrot / 2, i = interleaved ? r >> 1 : (r < half ? r : r - half), a, b;
+          rot_pair(i, nrot, interleaved, a, b);
+          float sn, cs;
+          sincosf((float)pos * inv_freq[i], &sn, &cs);
+          v = r == a ? v * cs - to_f(qr[b]) * sn : v * cs + to_f(qr[a]) * sn;
+        }
+      }
       sq[warp * Dk + d] = v * scale;
     }
   }
-  const T* rows = cache + (size_t)m[2] * slot_stride;
+  const T* rows = cache + (size_t)m[2] * slot_stride + (size_t)first * Dk;
   float mx = -INFINITY, l = 0.f, acc[LAT_MAXV];
 #pragma unroll
   for (int i = 0; i < LAT_MAXV; ++i) acc[i] = 0.f;
@@ -914,54 +922,66 @@ int hyb_headmajor_gate(const void* a, const void* g, long long g_stride, void* o
   return (int)cudaGetLastError();
 }
 
-int hyb_softcap(const void* in, float* out, long long total, float cap, int dt, cudaStream_t st) {
+int hyb_softcap(const void* in, float* out, long long total, float cap, float scale, int dt, cudaStream_t st) {
   if (total == 0) return 0;
   int blocks = (int)((total + 255) / 256);
-  HYB_DISPATCH(dt, (softcap_kernel<bf16><<<blocks, 256, 0, st>>>((const bf16*)in, out, total, cap)),
-               (softcap_kernel<float><<<blocks, 256, 0, st>>>((const float*)in, out, total, cap)));
+  HYB_DISPATCH(dt, (softcap_kernel<bf16><<<blocks, 256, 0, st>>>((const bf16*)in, out, total, cap, scale)),
+               (softcap_kernel<float><<<blocks, 256, 0, st>>>((const float*)in, out, total, cap, scale)));
   return (int)cudaGetLastError();
 }
 
-int hyb_latent_append(const void* ckv, long long ckv_stride, void* q, long long q_stride, const void* w,
-                      const float* inv_freq, void* cache, long long slot_stride, const int* meta, const int* tok_seq,
-                      int N, int H, int D, int R, int L, int nrot, float eps, int dt, cudaStream_t st) {
+int hyb_latent_prepare(const void* dq, long long dq_stride, const void* qw, void* cq, int Q, const void* ckv, long long ckv_stride,
+                       const void* w, const float* inv_freq, void* cache, long long slot_stride, const int* meta,
+                       const int* tok_seq, int N, int R, int L, int nrot, int interleaved, float eps, int dt, cudaStream_t st) {
   if (N == 0) return 0;
-  if (nrot > R || (nrot & 1)) return -2;
-  int threads = 256;
+  if (nrot > R || (nrot & 1) || Q < 1) return -2;
+  uintptr_t bits = (uintptr_t)dq | (uintptr_t)qw | (uintptr_t)cq | (uintptr_t)ckv | (uintptr_t)w | (uintptr_t)cache;
+  int vec = (bits & 15) == 0 && ((Q | L | R) & 7) == 0 && ((dq_stride | ckv_stride | slot_stride) & 7) == 0;
   HYB_DISPATCH(dt,
-               (latent_append_kernel<bf16><<<N, threads, 0, st>>>((const bf16*)ckv, ckv_stride, (bf16*)q, q_stride,
-                                                                  (const bf16*)w, inv_freq, (bf16*)cache, slot_stride,
-                                                                  meta, tok_seq, H, D, R, L, nrot, eps)),
-               (latent_append_kernel<float><<<N, threads, 0, st>>>((const float*)ckv, ckv_stride, (float*)q, q_stride,
-                                                                   (const float*)w, inv_freq, (float*)cache,
-                                                                   slot_stride, meta, tok_seq, H, D, R, L, nrot, eps)));
+               (latent_prepare_kernel<bf16><<<N, 256, 0, st>>>((const bf16*)dq, dq_stride, (const bf16*)qw, (bf16*)cq, Q,
+                                                               (const bf16*)ckv, ckv_stride, (const bf16*)w, inv_freq,
+                                                               (bf16*)cache, slot_stride, meta, tok_seq, R, L, nrot,
+                                                               interleaved, eps, vec)),
+               (latent_prepare_kernel<float><<<N, 256, 0, st>>>((const float*)dq, dq_stride, (const float*)qw, (float*)cq, Q,
+                                                                (const float*)ckv, ckv_stride, (const float*)w, inv_freq,
+                                                                (float*)cache, slot_stride, meta, tok_seq, R, L, nrot,
+                                                                interleaved, eps, vec)));
   return (int)cudaGetLastError();
 }
 
-int hyb_latent_attn(const void* qlat, const void* q, long long q_stride, const void* cache, long long slot_stride,
+int hyb_rotate_heads(void* q, long long q_stride, const float* inv_freq, const int* meta, const int* tok_seq, int N, int H, int D,
+                     int R, int nrot, int interleaved, int dt, cudaStream_t st) {
+  if (N == 0 || nrot == 0) return 0;
+  if (nrot > R || (nrot & 1) || nrot > 8192) return -2;
+  HYB_DISPATCH(dt,
+               (rotate_heads_kernel<bf16><<<N, 256, nrot * sizeof(float), st>>>((bf16*)q, q_stride, inv_freq, meta, tok_seq, H, D, R, nrot, interleaved)),
+               (rotate_heads_kernel<float><<<N, 256, nrot * sizeof(float), st>>>((float*)q, q_stride, inv_freq, meta, tok_seq, H, D, R, nrot, interleaved)));
+  return (int)cudaGetLastError();
+}
+
+int hyb_latent_attn(const float* qlat, const void* q, long long q_stride, const void* cache, long long slot_stride,
                     const int* meta, const int* tok_seq, void* out, int N, int H, int D, int R, int L, float scale,
-                    int nsplit, float* part_acc, float* part_ml, int dt, cudaStream_t st) {
+                    int nsplit, float* part_acc, float* part_ml, int window, const float* inv_freq, int nrot, int interleaved,
+                    int dt, cudaStream_t st) {
   if (N == 0) return 0;
-  if (L > 32 * LAT_MAXV || nsplit < 1 || (nsplit > 1 && (!part_acc || !part_ml))) return -3;
+  if (L > 1024 || nsplit < 1 || (nsplit > 1 && (!part_acc || !part_ml))) return -3;
+  if (inv_freq && (nrot > R || (nrot & 1))) return -2;
   int Dk = L + R;
   size_t smem = (size_t)(LAT_WARPS * Dk + LAT_TILE * (Dk + 1)) * sizeof(float);
   if (smem > 200 * 1024) return -3;
   dim3 grid(N, (H + LAT_WARPS - 1) / LAT_WARPS, nsplit);
-  if (dt == 0) {
-    cudaFuncSetAttribute(latent_attn_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    latent_attn_kernel<bf16><<<grid, LAT_WARPS * 32, smem, st>>>((const bf16*)qlat, (const bf16*)q, q_stride,
-                                                                 (const bf16*)cache, slot_stride, meta, tok_seq,
-                                                                 (bf16*)out, N, H, D, R, L, scale, nsplit, part_acc,
-                                                                 part_ml);
-    if (nsplit > 1) latent_combine_kernel<bf16><<<dim3(N, H), 128, 0, st>>>(part_acc, part_ml, (bf16*)out, N, H, L, nsplit);
-  } else {
-    cudaFuncSetAttribute(latent_attn_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    latent_attn_kernel<float><<<grid, LAT_WARPS * 32, smem, st>>>((const float*)qlat, (const float*)q, q_stride,
-                                                                  (const float*)cache, slot_stride, meta, tok_seq,
-                                                                  (float*)out, N, H, D, R, L, scale, nsplit, part_acc,
-                                                                  part_ml);
-    if (nsplit > 1) latent_combine_kernel<float><<<dim3(N, H), 128, 0, st>>>(part_acc, part_ml, (float*)out, N, H, L, nsplit);
-  }
+#define LA(T, MV)                                                                                                           \
+  do {                                                                                                                      \
+    cudaFuncSetAttribute(latent_attn_kernel<T, MV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                \
+    latent_attn_kernel<T, MV><<<grid, LAT_WARPS * 32, smem, st>>>(qlat, (const T*)q, q_stride, (const T*)cache, slot_stride, \
+                                                                  meta, tok_seq, (T*)out, N, H, D, R, L, scale, nsplit,     \
+                                                                  part_acc, part_ml, window, inv_freq, nrot, interleaved);  \
+    if (nsplit > 1) latent_combine_kernel<T><<<dim3(N, H), 128, 0, st>>>(part_acc, part_ml, (T*)out, N, H, L, nsplit);      \
+  } while (0)
+#define LAV(T) do { if (L <= 128) LA(T, 4); else if (L <= 512) LA(T, 16); else LA(T, 32); } while (0)
+  if (dt == 0) LAV(bf16); else LAV(float);
+#undef LAV
+#undef LA
   return (int)cudaGetLastError();
 }
 

@@ -1,6 +1,6 @@
 """Operations of the hybrid (attention + recurrent) model family over packed variable-length batches.
 
-Every function has two bodies.  On a CUDA tensor it launches the sm_100a kernel of ``csrc/hybrid_mixers.cu``
+Every function has two bodies.  On a CUDA tensor it launches the sm_100a kernel of ``csrc/hybrid_*.cu``
 (library ``_mdi_hybrid.so``, built on first use; a missing or unbuildable library raises — a CUDA tensor never
 takes the PyTorch body).  On a CPU tensor it runs the same arithmetic with plain PyTorch operations, which is how
 the models are brought up and tested on a machine without a GPU.
@@ -27,10 +27,11 @@ import torch.nn.functional as F
 from . import build as _build
 
 __all__ = ["BatchPlan", "HybridOpsError", "lib", "embed_rows", "cast_into", "norm_rows", "norm_accumulate", "gelu_",
-           "headmajor_gate", "softcap", "glu", "latent_append", "latent_attn", "causal_softmax", "matmul_f32", "conv_silu", "gated_recurrence", "linear",
+           "headmajor_gate", "softcap", "glu", "latent_attn", "causal_softmax", "matmul_f32", "conv_silu", "gated_recurrence", "linear",
            "rotary_inv_freq", "scaled_inv_freq", "linear_f32", "grouped_linear", "window_append", "window_attn", "head_gate", "relu2_",
            "token_side_gate", "router_topk", "moe_gemv", "gather_scale_rows", "combine_rows", "act_mul", "scaled_branches",
-           "full_norm_append", "lightning_recurrence", "norm_gate_rows", "gated_sum_norm_accumulate"]
+           "full_norm_append", "lightning_recurrence", "norm_gate_rows", "gated_sum_norm_accumulate", "embed_pairs",
+           "row_update", "norm_conv", "poly_norm", "latent_prepare", "rotate_heads", "NextInput"]
 
 
 class HybridOpsError(RuntimeError):
@@ -45,6 +46,13 @@ class _RecArgs(ctypes.Structure):
                 + [(n, c_longlong) for n in ("q_stride", "k_stride", "v_stride", "z_stride", "g_stride", "beta_stride",
                                              "out_stride")]
                 + [(n, c_int) for n in ("H", "G", "D", "V", "mode")] + [("tau", c_float), ("eps", c_float)])
+
+
+class _RowUpdateArgs(ctypes.Structure):
+    _fields_ = ([(n, c_void_p) for n in ("y", "w1", "b1", "x", "copy", "hist", "avg_w", "avg_out", "w2", "b2", "conv_w", "conv_state",
+                                         "h", "meta", "tok_seq")]
+                + [("y_stride", c_longlong)] + [(n, c_int) for n in ("N", "C", "kind1", "kind2", "n_avg", "taps")]
+                + [(n, c_float) for n in ("eps1", "eps2", "mult")])
 
 
 def lib() -> ctypes.CDLL:
@@ -76,9 +84,14 @@ def lib() -> ctypes.CDLL:
     h.hyb_act_mul_rows.argtypes = [vp, i64, vp, i64, i32, i32, f32, i32, vp]
     h.hyb_scaled_branches.argtypes = [vp, i64, vp, i64, vp, vp, i64, vp, i64, vp, i32, i32, i32, vp]
     h.hyb_headmajor_gate.argtypes = [vp, vp, i64, vp, i32, i32, i32, i32, vp]
-    h.hyb_softcap.argtypes = [vp, vp, i64, f32, i32, vp]
-    h.hyb_latent_append.argtypes = [vp, i64, vp, i64, vp, vp, vp, i64, vp, vp, i32, i32, i32, i32, i32, i32, f32, i32, vp]
-    h.hyb_latent_attn.argtypes = [vp, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, vp, vp, i32, vp]
+    h.hyb_softcap.argtypes = [vp, vp, i64, f32, f32, i32, vp]
+    h.hyb_latent_prepare.argtypes = [vp, i64, vp, vp, i32, vp, i64, vp, vp, vp, i64, vp, vp, i32, i32, i32, i32, i32, f32, i32, vp]
+    h.hyb_rotate_heads.argtypes = [vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp]
+    h.hyb_latent_attn.argtypes = [vp, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, vp, vp, i32, vp, i32, i32, i32, vp]
+    h.hyb_row_update.argtypes = [ctypes.POINTER(_RowUpdateArgs), i32, vp]
+    h.hyb_norm_conv.argtypes = [vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, i32, vp]
+    h.hyb_poly_norm.argtypes = [vp, i64, vp, i64, vp, i32, i32, f32, i32, vp]
+    h.hyb_embed_pairs.argtypes = [vp, vp, vp, vp, vp, i32, i32, i32, f32, i64, i64, i64, vp, vp, vp, i32, i32, vp]
     h.hyb_causal_softmax.argtypes = [vp, vp, i64, i32, i32, i32, f32, i32, i32, i32, i32, f32, vp, i32, i32, vp]
     h.hyb_full_norm_append.argtypes = [vp, i64, vp, i64, vp, i64, vp, vp, i64, vp, vp, i32, i32, i32, i32, i32, i32, f32, vp, vp, i32, vp]
     h.hyb_lightning.argtypes = [vp, i64, vp, i64, vp, i64, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp, vp, i32, vp, i32, vp]
@@ -139,6 +152,11 @@ class BatchPlan:
         tok_seq = torch.repeat_interleave(torch.arange(len(seqs), dtype=torch.int32), meta[:, 1].long())
         pos = torch.cat([torch.arange(p, p + n) for _, n, _, p in seqs]) if seqs else torch.zeros(0, dtype=torch.long)
         return cls(seqs, row, meta.to(device), tok_seq.to(device), pos.to(device))
+
+    @property
+    def one_token(self) -> bool:
+        """Every sequence brings exactly one token."""
+        return self.n_tokens == len(self.seqs)
 
     @property
     def last_rows(self) -> List[int]:
@@ -344,89 +362,128 @@ def headmajor_gate(a: torch.Tensor, g: torch.Tensor) -> torch.Tensor:
     return out
 
 
-def softcap(logits: torch.Tensor, cap: float) -> torch.Tensor:
-    """fp32 ``cap * tanh(logits / cap)`` (``cap <= 0``: a plain conversion to fp32)."""
+def softcap(logits: torch.Tensor, cap: float, scale: float = 1.0) -> torch.Tensor:
+    """fp32 ``cap * tanh(scale * logits / cap)`` (``cap <= 0``: ``scale * logits`` in fp32)."""
     if not logits.is_cuda:
         lf = logits.float()
+        if scale != 1.0:
+            lf = lf * float(scale)
         return cap * torch.tanh(lf / cap) if cap > 0 else lf
     assert logits.is_contiguous()
     out = torch.empty(logits.shape, device=logits.device, dtype=torch.float32)
-    _check(lib().hyb_softcap(logits.data_ptr(), out.data_ptr(), logits.numel(), float(cap), _dt(logits), _st()), "softcap")
+    _check(lib().hyb_softcap(logits.data_ptr(), out.data_ptr(), logits.numel(), float(cap), float(scale), _dt(logits), _st()), "softcap")
     return out
 
 
 # ---------------------------------------------------------------------------------------------------------
 # latent attention
 # ---------------------------------------------------------------------------------------------------------
-def latent_append(ckv: torch.Tensor, q: torch.Tensor, w: torch.Tensor, inv_freq: torch.Tensor, cache: torch.Tensor,
-                  plan: BatchPlan, H: int, D: int, R: int, L: int, nrot: int, eps: float) -> None:
-    """Per token: RMS-norm the latent (first ``L`` of the ``ckv`` row), rotate the shared key part (last ``R``) and
-    write both to ``cache[slot, pos]``; rotate the last ``R`` values of each of the ``H`` query heads of ``q`` in
-    place.  Rotation pairs entry ``i`` with ``i + nrot/2`` for the first ``nrot`` entries, angle ``pos * inv_freq[i]``."""
-    if not ckv.is_cuda:
-        N = ckv.size(0)
-        pos = plan.positions.float()
-        ang = pos[:, None] * inv_freq[None, :]
-        cs, sn = torch.cos(ang), torch.sin(ang)
-        half = nrot // 2
+def _rotate_torch(x: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor, nrot: int, pairing: str) -> torch.Tensor:
+    """``x [tokens, ..., R]``: the first ``nrot`` entries of the last axis rotated by ``pos * inv_freq``, in fp32."""
+    xf = x.float().clone()
+    if nrot == 0:
+        return xf
+    ang = positions.float()[:, None] * inv_freq[None, :]
+    c, s = torch.cos(ang), torch.sin(ang)
+    while c.dim() < xf.dim():
+        c, s = c.unsqueeze(1), s.unsqueeze(1)
+    i, j = (slice(0, nrot, 2), slice(1, nrot, 2)) if pairing == "pairs" else (slice(0, nrot // 2), slice(nrot // 2, nrot))
+    u, v = xf[..., i].clone(), xf[..., j].clone()
+    xf[..., i] = u * c - v * s
+    xf[..., j] = v * c + u * s
+    return xf
 
-        def rot(x: torch.Tensor) -> torch.Tensor:  # [..., R] with a leading token axis
-            xf = x.float()
-            u, v = xf[..., :half], xf[..., half:nrot]
-            c, s = (cs, sn) if xf.dim() == 2 else (cs[:, None, :], sn[:, None, :])
-            return torch.cat((u * c - v * s, v * c + u * s, xf[..., nrot:]), -1).to(x.dtype)
 
-        lat = _norm_torch(ckv[:, :L], w, None, eps, "rms").to(cache.dtype)
-        kr = rot(ckv[:, L:])
-        qv = q.view(N, H, D + R)
-        qv[..., D:] = rot(qv[..., D:])
-        for r0, n, slot, p0 in plan.seqs:
-            cache[slot, p0:p0 + n, :L] = lat[r0:r0 + n]
-            cache[slot, p0:p0 + n, L:] = kr[r0:r0 + n]
-        return
-    cs_, _ = _rows(ckv)
-    qs, _ = _rows(q)
-    _check(lib().hyb_latent_append(ckv.data_ptr(), cs_, q.data_ptr(), qs, w.data_ptr(), inv_freq.data_ptr(), cache.data_ptr(),
-                                   cache.stride(0), plan.meta.data_ptr(), plan.tok_seq.data_ptr(), ckv.size(0), H, D, R, L,
-                                   nrot, eps, _dt(ckv), _st()), "latent_append")
+def latent_prepare(dq: torch.Tensor, qw: torch.Tensor, ckv: Optional[torch.Tensor], w: Optional[torch.Tensor],
+                   inv_freq: torch.Tensor, cache: Optional[torch.Tensor], plan: BatchPlan, R: int, L: int, nrot: int, eps: float,
+                   pairing: str = "halves") -> torch.Tensor:
+    """Per token: the query latent ``dq`` RMS-normed with ``qw`` (returned), and, with ``ckv``, the token's cache row: the
+    latent (first ``L`` of the ``ckv`` row) RMS-normed with ``w``, the shared key part (last ``R``) rotated, both written
+    to ``cache[slot, pos]``.  ``ckv is None``: a layer that reads another layer's cache.  The rotation pairs entry ``i``
+    with ``i + nrot/2`` (``pairing="halves"``) or ``2i`` with ``2i+1`` (``"pairs"``) of the first ``nrot`` entries, angle
+    ``pos * inv_freq[i]``."""
+    if not dq.is_cuda:
+        if ckv is not None:
+            lat = _norm_torch(ckv[:, :L], w, None, eps, "rms").to(cache.dtype)
+            kr = _rotate_torch(ckv[:, L:], plan.positions, inv_freq, nrot, pairing).to(cache.dtype)
+            for r0, n, slot, p0 in plan.seqs:
+                cache[slot, p0:p0 + n, :L] = lat[r0:r0 + n]
+                cache[slot, p0:p0 + n, L:] = kr[r0:r0 + n]
+        return _norm_torch(dq, qw, None, eps, "rms").to(dq.dtype)
+    ds, Q = _rows(dq)
+    cq = torch.empty(dq.size(0), Q, device=dq.device, dtype=dq.dtype)
+    for t in (qw, w):
+        if t is not None and (t.dtype != dq.dtype or not t.is_contiguous()):
+            raise HybridOpsError("norm weights have the activation type")
+    none = ckv is None
+    _check(lib().hyb_latent_prepare(dq.data_ptr(), ds, qw.data_ptr(), cq.data_ptr(), Q, None if none else ckv.data_ptr(),
+                                    0 if none else _rows(ckv)[0], None if none else w.data_ptr(), inv_freq.data_ptr(),
+                                    None if none else cache.data_ptr(), 0 if none else cache.stride(0), plan.meta.data_ptr(),
+                                    plan.tok_seq.data_ptr(), dq.size(0), R, L, nrot, int(pairing == "pairs"), float(eps), _dt(dq),
+                                    _st()), "latent_prepare")
+    return cq
+
+
+def rotate_heads(q: torch.Tensor, inv_freq: torch.Tensor, plan: BatchPlan, H: int, D: int, R: int, nrot: int,
+                 pairing: str = "halves") -> torch.Tensor:
+    """The last ``R`` values of each of the ``H`` heads of ``q [N, H * (D + R)]`` rotated in place (as in
+    :func:`latent_prepare`)."""
+    if not q.is_cuda:
+        qv = q.view(q.size(0), H, D + R)
+        qv[..., D:] = _rotate_torch(qv[..., D:], plan.positions, inv_freq, nrot, pairing).to(q.dtype)
+        return q
+    _check(lib().hyb_rotate_heads(q.data_ptr(), _rows(q)[0], inv_freq.data_ptr(), plan.meta.data_ptr(), plan.tok_seq.data_ptr(),
+                                  q.size(0), H, D, R, nrot, int(pairing == "pairs"), _dt(q), _st()), "rotate_heads")
+    return q
 
 
 _SM_TARGET = 148  # one block per SM of a B200
 
 
 def latent_attn(qlat: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, plan: BatchPlan, H: int, D: int, R: int, L: int,
-                scale: float, split: int = 0) -> torch.Tensor:
-    """Causal softmax attention of ``H`` heads over the cached rows ``[L latent | R rotated key]`` of each token's slot.
-    The query of head ``h`` is ``[qlat[h, tok] | q[tok, h, D:]]``, the value of a row is its latent part.
-    Returns the attended latents ``[H, N, L]``.  ``split`` (CUDA): key shares per query, 0 = chosen from the batch shape."""
+                scale: float, split: int = 0, window: int = 0, inv_freq: Optional[torch.Tensor] = None, nrot: int = 0,
+                pairing: str = "halves") -> torch.Tensor:
+    """Causal softmax attention of ``H`` heads over the cached rows ``[L latent | R rotated key]`` of each token's slot
+    (``window > 0``: the last ``window`` positions up to the token's own).  The query of head ``h`` is
+    ``[qlat[h, tok] | q[tok, h, D:]]``, the value of a row is its latent part.  ``qlat`` is used in fp32.  With
+    ``inv_freq`` the second part of the query is not rotated yet: that happens as it is loaded (fp32, unrounded).
+    Returns the attended latents ``[H, N, L]``.  ``split`` (CUDA): key shares per query, 0 = chosen from the batch shape
+    and the window."""
     N = q.size(0)
     if not q.is_cuda:
         out = torch.empty(H, N, L, dtype=q.dtype)
-        qr = q.view(N, H, D + R)[..., D:].permute(1, 0, 2)
-        qq = torch.cat((qlat, qr), -1).float() * scale  # [H, N, L+R]
+        qr = q.view(N, H, D + R)[..., D:].float()
+        if inv_freq is not None:
+            qr = _rotate_torch(qr, plan.positions, inv_freq, nrot, pairing)
+        qq = torch.cat((qlat.float(), qr.permute(1, 0, 2)), -1) * scale  # [H, N, L+R]
         for r0, n, slot, p0 in plan.seqs:
             rows = cache[slot, :p0 + n].float()
             s = qq[:, r0:r0 + n] @ rows.T  # [H, n, keys]
-            keys = torch.arange(p0 + n)
-            s = s.masked_fill(keys[None, None, :] > (p0 + torch.arange(n))[None, :, None], float("-inf"))
-            out[:, r0:r0 + n] = (torch.softmax(s, -1) @ rows[:, :L]).to(q.dtype)
+            keys, pos = torch.arange(p0 + n)[None, None, :], (p0 + torch.arange(n))[None, :, None]
+            hidden = keys > pos
+            if window > 0:
+                hidden = hidden | (pos - keys >= window)
+            out[:, r0:r0 + n] = (torch.softmax(s.masked_fill(hidden, float("-inf")), -1) @ rows[:, :L]).to(q.dtype)
         return out
     assert qlat.is_contiguous()
+    qlat = qlat.float()
     qs, _ = _rows(q)
     out = torch.empty(H, N, L, device=q.device, dtype=q.dtype)
     # few query tokens (decoding) cannot fill the GPU with one block per token and 8 heads: split the keys of each
-    # query over several blocks and merge the partial softmaxes.  The split count depends only on the batch shape,
-    # so a captured step stays valid while contexts grow.
+    # query over several blocks and merge the partial softmaxes.  The split count depends only on the batch shape
+    # and the window, so a captured step stays valid while contexts grow.
     blocks = N * ((H + 7) // 8)
-    nsplit = 1 if blocks >= 2 * _SM_TARGET or split == 1 else (split or max(1, min(32, (2 * _SM_TARGET) // blocks)))
+    tiles = (window + 31) // 32 if window > 0 else 32
+    nsplit = 1 if blocks >= 2 * _SM_TARGET or split == 1 else (split or max(1, min(32, tiles, (2 * _SM_TARGET) // blocks)))
     pa = pm = None
     if nsplit > 1:
         pa = torch.empty(nsplit, H, N, L, device=q.device, dtype=torch.float32)
         pm = torch.empty(nsplit, H, N, 2, device=q.device, dtype=torch.float32)
     _check(lib().hyb_latent_attn(qlat.data_ptr(), q.data_ptr(), qs, cache.data_ptr(), cache.stride(0), plan.meta.data_ptr(),
                                  plan.tok_seq.data_ptr(), out.data_ptr(), N, H, D, R, L, float(scale), nsplit,
-                                 None if pa is None else pa.data_ptr(), None if pm is None else pm.data_ptr(), _dt(q), _st()),
-           "latent_attn")
+                                 None if pa is None else pa.data_ptr(), None if pm is None else pm.data_ptr(), int(window),
+                                 None if inv_freq is None else inv_freq.data_ptr(), int(nrot), int(pairing == "pairs"), _dt(q),
+                                 _st()), "latent_attn")
     return out
 
 
@@ -1002,3 +1059,163 @@ def gated_sum_norm_accumulate(resid: torch.Tensor, a: torch.Tensor, b: Optional[
                                     None if sg is None else sg.data_ptr(), 0 if sg is None else sg.stride(0), w.data_ptr(),
                                     resid.data_ptr(), resid.stride(0), a.size(0), a.size(1), float(eps),
                                     _NORM_KINDS[kind], None if copy is None else copy.data_ptr(), _dt(a), _st()), "gated_sum_norm")
+
+
+# ---------------------------------------------------------------------------------------------------------
+# sandwich blocks with input convolutions and an average over depth; the bigram embedding; the polynomial activation
+# ---------------------------------------------------------------------------------------------------------
+def embed_pairs(table: torch.Tensor, pair_table: torch.Tensor, tokens: torch.Tensor, plan: BatchPlan, prev: torch.Tensor,
+                buckets: int, mul_prev: int, mul_cur: int, scale: float = 1.0, out: Optional[torch.Tensor] = None,
+                out2: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """fp32 rows ``scale * table[token] + pair_table[(previous * mul_prev + token * mul_cur) mod buckets]``; a sequence's
+    first token takes row ``buckets`` of ``pair_table [buckets + 1, C]``.  ``prev`` int32 ``[slots]`` holds the last token of
+    each slot between steps and is advanced.  ``out2`` receives a second copy of the rows."""
+    N, C = tokens.numel(), table.size(1)
+    out = torch.empty(N, C, device=table.device, dtype=torch.float32) if out is None else out
+    if not table.is_cuda:
+        row = torch.empty(N, dtype=torch.long)
+        tk = tokens.long()
+        for r0, n, slot, p0 in plan.seqs:
+            before = torch.cat((prev[slot:slot + 1].long(), tk[r0:r0 + n - 1]))
+            row[r0:r0 + n] = (before * int(mul_prev) + tk[r0:r0 + n] * int(mul_cur)) % int(buckets)
+            if p0 == 0:
+                row[r0] = int(buckets)
+            prev[slot] = tokens[r0 + n - 1]
+        out.copy_(table[tk].float() * float(scale) + pair_table[row].float())
+        if out2 is not None:
+            out2.copy_(out)
+        return out
+    if pair_table.dtype != table.dtype or pair_table.size(1) != C or pair_table.size(0) != int(buckets) + 1 \
+            or not (pair_table.is_contiguous() and table.is_contiguous() and out.is_contiguous()):
+        raise HybridOpsError("the pair table has buckets + 1 rows and the embedding table's type and width")
+    _check(lib().hyb_embed_pairs(table.data_ptr(), pair_table.data_ptr(), tokens.data_ptr(), out.data_ptr(),
+                                 None if out2 is None else out2.data_ptr(), N, len(plan.seqs), C, float(scale), int(buckets),
+                                 int(mul_prev), int(mul_cur), prev.data_ptr(), plan.meta.data_ptr(), plan.tok_seq.data_ptr(),
+                                 int(not plan.one_token), _dt(table), _st()), "embed_pairs")
+    return out
+
+
+@dataclass
+class NextInput:
+    """How a sublayer reads the residual stream: a norm (``w``, ``b``, ``eps``, ``kind``), then ``h + conv(h)`` over time with
+    ``conv_w`` fp32 ``[taps, C]`` (last row: the current token; None: no convolution) and ``state`` fp32 ``[slots, taps-1, C]``,
+    the normed rows before a step's first token, oldest first."""
+
+    w: torch.Tensor
+    b: Optional[torch.Tensor]
+    eps: float
+    kind: str
+    conv_w: Optional[torch.Tensor] = None
+    state: Optional[torch.Tensor] = None
+
+
+def norm_conv(x: torch.Tensor, nxt: NextInput, plan: BatchPlan, out_dtype: torch.dtype, tile: int = 0) -> torch.Tensor:
+    """``h = norm(x)``, then ``h + sum_j conv_w[j] * h_(t - taps + 1 + j)`` for every token, in fp32 with one rounding; rows
+    before the sequence's start are zero, rows of earlier steps come from ``nxt.state``, which is advanced.  ``tile``
+    (CUDA): token rows per block, 0 = chosen from the step's size (the result does not depend on it)."""
+    if nxt.conv_w is None:
+        return norm_rows(x, nxt.w, nxt.b, nxt.eps, nxt.kind, out_dtype)
+    taps, C = nxt.conv_w.shape
+    if not x.is_cuda:
+        h = _norm_torch(x, nxt.w, nxt.b, nxt.eps, nxt.kind)
+        out = torch.empty(h.shape, dtype=out_dtype)
+        for r0, n, slot, p0 in plan.seqs:
+            past = nxt.state[slot].clone() if taps > 1 else h.new_zeros(0, C)
+            past[:max(0, taps - 1 - p0)] = 0.0  # positions before the sequence's start, whatever the slot holds
+            full = torch.cat((past, h[r0:r0 + n]), 0)
+            acc = torch.zeros(n, C)
+            for j in range(taps):
+                acc += nxt.conv_w[j] * full[j:j + n]
+            out[r0:r0 + n] = (h[r0:r0 + n] + acc).to(out_dtype)
+            if taps > 1:
+                nxt.state[slot] = full[-(taps - 1):]
+        return out
+    if plan.one_token:
+        return row_update(x, nxt=nxt, plan=plan, out_dtype=out_dtype)
+    N = x.size(0)
+    if not x.is_contiguous() or nxt.w.dtype != out_dtype:
+        raise HybridOpsError("the residual rows are dense; norm weights have the activation type")
+    out = torch.empty(N, C, device=x.device, dtype=out_dtype)
+    tile = tile or max(1, min(16, N // (4 * _SM_TARGET)))
+    _check(lib().hyb_norm_conv(x.data_ptr(), nxt.w.data_ptr(), None if nxt.b is None else nxt.b.data_ptr(), nxt.conv_w.data_ptr(),
+                               None if taps == 1 else nxt.state.data_ptr(), out.data_ptr(), plan.meta.data_ptr(),
+                               plan.tok_seq.data_ptr(), N, len(plan.seqs), C, taps, _NORM_KINDS[nxt.kind], float(nxt.eps), tile,
+                               _dt(out), _st()), "norm_conv")
+    return out
+
+
+def row_update(x: torch.Tensor, y: Optional[torch.Tensor] = None, w: Optional[torch.Tensor] = None, b: Optional[torch.Tensor] = None,
+               eps: float = 0.0, kind: str = "layer", mult: float = 1.0, copy: Optional[torch.Tensor] = None,
+               depth: Optional[torch.Tensor] = None, index: int = 0, depth_w: Optional[torch.Tensor] = None,
+               nxt: Optional[NextInput] = None, plan: Optional[BatchPlan] = None,
+               out_dtype: Optional[torch.dtype] = None) -> Optional[torch.Tensor]:
+    """One pass over the fp32 residual rows ``x [N, C]``:
+
+    * ``x += mult * norm(y)`` (``y`` given; ``kind`` "layer" or "rms" with ``w`` and, for layer, ``b``);
+    * ``copy`` receives ``x`` rounded to its type;
+    * ``depth [rows, N, C]`` (fp32; ``x`` IS ``depth[index]``): ``depth[index + 1] = sum_(j <= index) depth_w[j] depth[j]``, the
+      average over depth with ``depth_w`` fp32 ``[index + 1]``;
+    * ``nxt``: returns what the next sublayer reads of the result (the average if there is one, else ``x``) in
+      ``out_dtype``: its norm and convolution (see :func:`norm_conv`).  On CUDA this needs a step of one token per
+      sequence; other steps call :func:`norm_conv` afterwards."""
+    if x.dtype != torch.float32:
+        raise HybridOpsError("the residual stream is fp32")
+    if depth is not None and depth_w.numel() != index + 1:
+        raise HybridOpsError("the average over depth needs one weight per row so far")
+    if not x.is_cuda:
+        if y is not None:
+            x.add_(_norm_torch(y, w, b, eps, kind), alpha=float(mult))
+        if copy is not None:
+            copy.copy_(x)
+        if depth is not None:
+            acc = torch.zeros_like(x)
+            for j in range(index + 1):
+                acc += depth_w[j] * depth[j]
+            depth[index + 1].copy_(acc)
+            x = depth[index + 1]
+        return None if nxt is None else norm_conv(x, nxt, plan, out_dtype)
+    if nxt is not None and not plan.one_token:
+        raise HybridOpsError("the next sublayer's input is fused only into steps of one token per sequence")
+    if not x.is_contiguous() or (depth is not None and not depth.is_contiguous()) or (copy is not None and not copy.is_contiguous()):
+        raise HybridOpsError("residual rows are dense")
+    N, C = x.shape
+    a = _RowUpdateArgs()
+    dt = None
+    for t in (y, w, b, copy, None if nxt is None else nxt.w, None if nxt is None else nxt.b):
+        if t is not None:
+            if dt is not None and t.dtype != dt:
+                raise HybridOpsError("the sublayer's output, norm weights and copy have one type")
+            dt = t.dtype
+    h = None
+    if y is not None:
+        a.y, a.y_stride, a.w1, a.b1 = y.data_ptr(), _rows(y)[0], w.data_ptr(), None if b is None else b.data_ptr()
+        a.kind1, a.eps1 = _NORM_KINDS[kind], float(eps)
+    a.mult, a.x, a.copy, a.N, a.C = float(mult), x.data_ptr(), None if copy is None else copy.data_ptr(), N, C
+    if depth is not None:
+        a.hist, a.avg_w, a.n_avg, a.avg_out = depth.data_ptr(), depth_w.data_ptr(), index, depth[index + 1].data_ptr()
+    if nxt is not None:
+        h = torch.empty(N, C, device=x.device, dtype=out_dtype)
+        if out_dtype != dt:
+            raise HybridOpsError("norm weights have the activation type")
+        a.w2, a.b2, a.kind2, a.eps2 = nxt.w.data_ptr(), None if nxt.b is None else nxt.b.data_ptr(), _NORM_KINDS[nxt.kind], float(nxt.eps)
+        a.h, a.meta, a.tok_seq = h.data_ptr(), plan.meta.data_ptr(), plan.tok_seq.data_ptr()
+        if nxt.conv_w is not None:
+            a.taps, a.conv_w = nxt.conv_w.size(0), nxt.conv_w.data_ptr()
+            a.conv_state = nxt.state.data_ptr() if a.taps > 1 else None
+    _check(lib().hyb_row_update(ctypes.byref(a), 1 if dt in (None, torch.float32) else 0, _st()), "row_update")
+    return h
+
+
+def poly_norm(z: torch.Tensor, coef: torch.Tensor, eps: float) -> torch.Tensor:
+    """``c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3`` per row of ``z [N, F]``: powers entry by entry, ``N(v) = v / sqrt(mean(v^2) +
+    eps)`` over the row, everything in fp32; ``coef`` fp32 ``[4]``.  Result in the activation type."""
+    if not z.is_cuda:
+        zf = z.float()
+        y = sum(coef[k] * _norm_torch(zf ** (k + 1), None, None, eps, "rms") for k in range(3)) + coef[3]
+        return y.to(z.dtype)
+    if coef.dtype != torch.float32 or coef.numel() != 4 or not coef.is_contiguous():
+        raise HybridOpsError("the activation has four fp32 numbers")
+    out = torch.empty(z.shape, device=z.device, dtype=z.dtype)
+    _check(lib().hyb_poly_norm(z.data_ptr(), _rows(z)[0], out.data_ptr(), out.stride(0), coef.data_ptr(), z.size(0), z.size(1),
+                               float(eps), _dt(z), _st()), "poly_norm")
+    return out
