@@ -22,6 +22,9 @@ of the same width, whose windowed attention and mixture of experts are the close
 timed inside one chunk (the prompt ends short of a chunk edge), so that a step sees about as many keys as the
 windowed design does.
 
+``bench.py --family ratesun`` measures the sandwich design with input convolutions, an average over depth, windowed
+latent attention on shared caches and a polynomial activation beside the plain sandwich design of the same width.
+
 ``bench.py --family zudovik`` measures the post-norm design (causal grouped-query attention with the norm over the
 whole q and k projections, a score cap and learned sinks, a layer on another layer's keys and values, the fixed-decay
 linear recurrence, clamped gated experts with identity experts and a token-gated shared expert) beside the
@@ -36,7 +39,22 @@ from typing import Any, Callable, Dict, List
 
 import torch
 
-__all__ = ["run_family_compare", "hybrid_bench_config", "vudelix_bench_config", "labepel_bench_config", "zudovik_bench_config"]
+__all__ = ["run_family_compare", "hybrid_bench_config", "vudelix_bench_config", "labepel_bench_config", "zudovik_bench_config",
+           "ratesun_bench_config"]
+
+
+def ratesun_bench_config(width: int, window: int = 1024) -> Dict[str, Any]:
+    """4 layers of windowed latent attention + dense (polynomial activation, ``4 * width``), the second and the fourth on the
+    cache of the layer before; attention sizes of the sandwich design's bench model."""
+    h = width // 128
+    lat = {"heads": h, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "q_rank": min(1536, width),
+           "scale": 192 ** -0.5, "rot": {"dims": 64, "base": 10000.0}, "mask": {"size": window}}
+    mlp = {"kind": "dense", "ff": 4 * width}
+    layers = [{"type": "latent_attention", "mixer": dict(lat) if i % 2 == 0 else dict(lat, kv_from=i - 1), "mlp": dict(mlp)}
+              for i in range(4)]
+    return {"architecture": "Ratesun", "vocab": 32000, "width": width, "layers": layers, "norm": {"eps": 1e-6},
+            "embedding": {"bigram": {"buckets": 50021, "mul_prev": 1009, "mul_cur": 31}}, "canon": {"taps": 4},
+            "residual_mult": 0.5, "token_side": {"dim": 64}, "logit_scale": 0.5}
 
 
 def zudovik_bench_config(width: int) -> Dict[str, Any]:
@@ -130,7 +148,7 @@ def _hybrid(width: int, prompt_len: int, batch: int, steps: int, warmup: int, de
 
     dev = torch.device("cuda")
     make = {"hybrid": hybrid_bench_config, "vudelix": vudelix_bench_config, "labepel": labepel_bench_config,
-            "zudovik": zudovik_bench_config}[design]
+            "zudovik": zudovik_bench_config, "ratesun": ratesun_bench_config}[design]
     cfg = HybridConfig.from_dict(make(width))
     model = HybridLM(cfg, {}).init_random(dev, torch.bfloat16, seed=1)
     params = sum(p.numel() for p in model.tensor_map().values())
@@ -164,7 +182,7 @@ def _hybrid(width: int, prompt_len: int, batch: int, steps: int, warmup: int, de
         out[f"decode_ms_b{b}"] = round(ms, 4)
         del r
     kernels = {"hybrid": _hybrid_kernels, "vudelix": _vudelix_kernels, "labepel": _labepel_kernels,
-               "zudovik": _zudovik_kernels}[design]
+               "zudovik": _zudovik_kernels, "ratesun": _ratesun_kernels}[design]
     out["kernels"] = kernels(model, prompt_len, batch)
     return out
 
@@ -333,6 +351,80 @@ def _zudovik_kernels(model: Any, T: int, batch: int) -> List[Dict[str, Any]]:
     return rows
 
 
+def _ratesun_kernels(model: Any, T: int, batch: int) -> List[Dict[str, Any]]:
+    """The kernels of the sandwich design with input convolutions and an average over depth; ``like`` names the row of
+    ``_hybrid_kernels`` (or, for the per-layer token embedding, of ``_vudelix_kernels``) that does the corresponding work."""
+    from ..ops import hybrid as H
+
+    pk = _peaks()
+    dev, dt, cfg = model.device, model.dtype, model.config
+    C = cfg.width
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    rows: List[Dict[str, Any]] = []
+
+    def rec(name: str, like: str, phase: str, fn: Callable[[], Any], nbytes: float, flops: float = 0.0) -> None:
+        ms = _time(fn, 5, 3, flush)
+        rows.append({"kernel": name, "like": like, "phase": phase, "ms": round(ms, 4), "gb_s": round(nbytes / ms / 1e6, 1),
+                     "tflops": round(flops / ms / 1e9, 2),
+                     "frac_of_roofline": round(max(nbytes / ms / 1e6 / pk["hbm_gbs"], flops / ms / 1e9 / pk["bf16_tflops"]), 4),
+                     "peaks": pk["source"]})
+
+    blk = model.blocks[2]
+    mix, side, taps, bg = blk.mix, blk.side, cfg.canon_taps, cfg.bigram
+    Hh, D, R, V, L, W = mix.H, mix.D, mix.R, mix.V, mix.L, mix.window
+    for phase, lengths, starts in (("prefill", [T], [0]), ("decode", [1] * batch, [T] * batch)):
+        n_seq, N = len(lengths), sum(lengths)
+        pool = model.new_pool(n_seq, T + 8)
+        plan = H.BatchPlan.make(lengths, list(range(n_seq)), starts, dev)
+        st = pool.runs[2]
+        st["cache"].normal_()
+        tok = torch.randint(0, cfg.vocab, (N,), device=dev, dtype=torch.int32)
+        depth = torch.randn(6, N, C, device=dev)
+        x, y = depth[3], torch.randn(N, C, device=dev).to(dt)
+        b1 = (blk.norm1b.w, blk.norm1b.b, 1e-6, "layer", 0.5)
+        conv_bytes = 8.0 * n_seq * (taps - 1) * C  # state read and written
+        rec("embed_pairs", "embed_rows", phase,
+            lambda: H.embed_pairs(model.embed, model.bigram, tok, plan, pool.prev, bg["buckets"], bg["mul_prev"], bg["mul_cur"], 1.0,
+                                  depth[0], depth[1]), N * C * 12.0)
+        if phase == "prefill":
+            rec("norm_conv", "layer_norm", phase, lambda: H.norm_conv(x, blk._input1(st), plan, dt), N * C * 6.0 + conv_bytes)
+            rec("row_update", "norm_accumulate", phase, lambda: H.row_update(x, y, *b1), N * C * 10.0)
+            rec("row_update[depth average of 4 rows]", "norm_accumulate", phase,
+                lambda: H.row_update(x, y, side.norm, None, 1e-6, "rms", 0.5, depth=depth, index=3, depth_w=blk.depth_w), N * C * 26.0)
+        else:
+            rec("row_update[+ next norm, convolution]", "norm_accumulate", phase,
+                lambda: H.row_update(x, y, *b1, nxt=blk._input2(st), plan=plan, out_dtype=dt), N * C * 12.0 + conv_bytes)
+            rec("row_update[depth average, next norm, convolution]", "norm_accumulate", phase,
+                lambda: H.row_update(x, y, side.norm, None, 1e-6, "rms", 0.5, depth=depth, index=3, depth_w=blk.depth_w,
+                                     nxt=blk._input1(st), plan=plan, out_dtype=dt), N * C * 28.0 + conv_bytes)
+        h = torch.randn(N, C, device=dev).to(dt)
+        p = H.linear(h, mix.w_in)
+        rec("latent_prepare", "latent_prepare", phase,
+            lambda: H.latent_prepare(mix.col(p, "dq"), mix.dq_norm, mix.col(p, "dkv"), mix.dkv_norm, mix.inv_freq, st["cache"], plan, R, L,
+                                     mix.nrot, 1e-6, mix.pairing), 4.0 * N * (L + R + mix.QR))
+        q = H.linear(h[:, :mix.QR].contiguous(), mix.uq)
+        keys = sum(min(W, s + i + 1) for n, s in zip(lengths, starts) for i in range(n))  # visible (query, key) pairs
+        if phase == "prefill":
+            rec("rotate_heads", "latent_prepare", phase,
+                lambda: H.rotate_heads(q, mix.inv_freq, plan, Hh, D, R, mix.nrot, mix.pairing), 4.0 * N * Hh * R)
+            rec("latent_attn_expanded[window]", "latent_attn_expanded(gemm+softmax)", phase, lambda: mix._expanded(q, st["cache"], plan),
+                2.0 * N * Hh * (D + R + V), 2.0 * T * L * Hh * (D + V) + 2.0 * Hh * keys * (D + R + V))
+        else:
+            qlat = torch.randn(Hh, N, L, device=dev)
+            rec("latent_attn[window, rotation]", "latent_attn", phase,
+                lambda: H.latent_attn(qlat, q, st["cache"], plan, Hh, D, R, L, mix.scale, window=W, inv_freq=mix.inv_freq, nrot=mix.nrot,
+                                      pairing=mix.pairing),
+                6.0 * Hh * N * L + 2.0 * Hh * N * R + 2.0 * (L + R) * sum(min(W, s + 1) for s in starts), 2.0 * Hh * keys * (2 * L + R))
+        a = torch.randn(N, blk.mlp.up.size(0), device=dev).to(dt)
+        rec("poly_norm", "gelu", phase, lambda: H.poly_norm(a, blk.mlp.coef32, 1e-6), 4.0 * a.numel())
+        rec("dense_ff(gemm+poly_norm)", "dense_ff(gemm+gelu)", phase, lambda: blk.mlp(h), 4.0 * C * a.size(1) + 4.0 * N * C,
+            4.0 * N * C * a.size(1))
+        zs = H.linear(h, side.gate)
+        rec("token_side_gate", "token_side_gate", phase, lambda: H.token_side_gate(zs, model.side_embed, tok, 0), 6.0 * N * side.dim)
+        del pool
+    return rows
+
+
 def _labepel_kernels(model: Any, T: int, batch: int) -> List[Dict[str, Any]]:
     """The parallel-block design's own kernels alone, on the prompt shape and on the decode shape; ``like`` names the
     row of ``_vudelix_kernels`` that does the corresponding work in the pre-norm design."""
@@ -454,9 +546,9 @@ def _hybrid_kernels(model: Any, T: int, batch: int) -> List[Dict[str, Any]]:
                     ms = _time(lambda: H.latent_attn(qlat, q, st["cache"], plan, Hh, D, R, L, mix.scale), 5, 3, flush)
                     nbytes = 2.0 * (2 * Hh * N * L + Hh * N * R) + 2.0 * (L + R) * sum(s + n for n, s in zip(lengths, starts))
                     rec("latent_attn", phase, ms, nbytes, 2.0 * Hh * keys * (2 * L + R))
-                ms = _time(lambda: H.latent_append(mix.col(p, "dkv"), q, mix.dkv_norm, mix.inv_freq, st["cache"], plan, Hh, D,
-                                                   R, L, mix.nrot, 1e-6), 5, 3, flush)
-                rec("latent_append", phase, ms, 2.0 * N * (2 * (L + R) + 2 * Hh * R), 0.0)
+                ms = _time(lambda: H.latent_prepare(mix.col(p, "dq"), mix.dq_norm, mix.col(p, "dkv"), mix.dkv_norm, mix.inv_freq,
+                                                    st["cache"], plan, R, L, mix.nrot, 1e-6), 5, 3, flush)
+                rec("latent_prepare", phase, ms, 4.0 * N * (L + R + mix.QR), 0.0)
             else:
                 mode = "delta" if li == 1 else "gla"
                 Hh, D, V = mix.H, mix.D, mix.V
@@ -480,6 +572,18 @@ def _hybrid_kernels(model: Any, T: int, batch: int) -> List[Dict[str, Any]]:
         blk = model.blocks[0]
         ms = _time(lambda: H.norm_rows(x, blk.norm1.w, blk.norm1.b, 1e-6, "layer", dt), 5, 3, flush)
         rec("layer_norm", phase, ms, N * model.config.width * 6.0, 0.0)
+        C = model.config.width
+        y = torch.randn(N, C, device=dev).to(dt)
+        ms = _time(lambda: H.norm_accumulate(x, y, blk.norm1b.w, blk.norm1b.b, 1e-6), 5, 3, flush)
+        rec("norm_accumulate", phase, ms, N * C * 10.0, 0.0)
+        tok = torch.randint(0, model.config.vocab, (N,), device=dev, dtype=torch.int32)
+        ms = _time(lambda: H.embed_rows(model.embed, tok), 5, 3, flush)
+        rec("embed_rows", phase, ms, N * C * 6.0, 0.0)
+        a = torch.randn(N, blk.mlp.up.size(0), device=dev).to(dt)
+        ms = _time(lambda: H.gelu_(a), 5, 3, flush)
+        rec("gelu", phase, ms, 4.0 * a.numel(), 0.0)
+        ms = _time(lambda: blk.mlp(y), 5, 3, flush)
+        rec("dense_ff(gemm+gelu)", phase, ms, 4.0 * C * a.size(1) + 4.0 * N * C, 4.0 * N * C * a.size(1))
         del pool
     return rows
 
@@ -573,6 +677,30 @@ def run_family_compare(widths: List[int], prompt_len: int = 2048, batch: int = 8
                 k["roofline_vs_like"] = round(k["frac_of_roofline"] / other, 3) if other else None
             results.append({"width": w, "zudovik": new, "labepel": old, "sandwich_recurrence": rec_rows})
         return {"metric": "family_compare", "family": "zudovik", "dtype": "bf16", "data": "synthetic", "prompt_len": prompt_len,
+                "decode_batch": batch, "steps": steps, "warmup": warmup, "l2": "flushed between single-kernel timings",
+                "results": results}
+    if family == "ratesun":
+        from ..models.config import HybridConfig
+        from ..models.hybrid import HybridLM
+
+        for w in widths:
+            new = _hybrid(w, prompt_len, batch, steps, warmup, "ratesun")
+            torch.cuda.empty_cache()
+            old = _hybrid(w, prompt_len, batch, steps, warmup, "hybrid")
+            torch.cuda.empty_cache()
+            # the per-layer token embedding's like kernel lives in the pre-norm design: its kernels alone
+            prenorm = HybridLM(HybridConfig.from_dict(vudelix_bench_config(w)), {}).init_random(torch.device("cuda"), torch.bfloat16, seed=1)
+            side_rows = [k for k in _vudelix_kernels(prenorm, prompt_len, batch) if k["kernel"] == "token_side_gate"]
+            del prenorm
+            torch.cuda.empty_cache()
+            theirs = {(k["kernel"], k["phase"]): k for k in old["kernels"] + side_rows}
+            for k in new["kernels"]:  # how far from its roofline, relative to the like kernel (above 1: this one is nearer)
+                other = theirs.get((k["like"], k["phase"]))
+                k["like_ms"] = other["ms"] if other else None
+                k["roofline_vs_like"] = round(k["frac_of_roofline"] / other["frac_of_roofline"], 3) \
+                    if other and other["frac_of_roofline"] else None
+            results.append({"width": w, "ratesun": new, "hybrid": old, "prenorm_side": side_rows})
+        return {"metric": "family_compare", "family": "ratesun", "dtype": "bf16", "data": "synthetic", "prompt_len": prompt_len,
                 "decode_batch": batch, "steps": steps, "warmup": warmup, "l2": "flushed between single-kernel timings",
                 "results": results}
     if family == "labepel":
