@@ -180,105 +180,120 @@ __global__ void __launch_bounds__(HR_THREADS) row_update_kernel(RowUpdateArgs a)
   }
 }
 
-// h = norm(x), out = h + conv(h) for steps that bring several tokens of a sequence.  A block owns `tile` consecutive
-// token rows and slides over them with the last `taps` normed rows in a ring in shared memory; the rows before its first
-// one are normed again (or come from conv_state where they belong to an earlier step), so blocks are independent.  A
-// thread owns the same channels in every row: the ring needs no barrier.  When `tails` is set the kernel only advances
-// conv_state: block s norms the last rows of sequence s (rows whose state was read by the main launch before).
+// h = norm(x), out = h + conv(h) for steps that bring several tokens of a sequence.  A block owns `tile` consecutive token
+// rows.  First its warps take the statistics of those rows and of the taps - 1 rows before them, one row per warp; then
+// every thread walks its channels: a tap reads the earlier row again (it is in the first-level cache) and norms it on the
+// fly, rows of earlier steps come from conv_state.  Blocks are independent.
+// mode 0: outputs only.  mode 1: outputs, and the block that holds a sequence's last token writes its conv_state (allowed
+// when no sequence of the step reads it: they all start at position 0).  mode 2: conv_state only, one block per sequence.
 template <typename T, int VEC>
 __global__ void __launch_bounds__(HR_THREADS) norm_conv_kernel(const float* __restrict__ x, const T* __restrict__ w,
                                                                const T* __restrict__ b, const float* __restrict__ conv_w,
                                                                float* __restrict__ state, T* __restrict__ out,
                                                                const int* __restrict__ meta, const int* __restrict__ tok_seq,
-                                                               int N, int C, int taps, int kind, float eps, int tile, int tails) {
-  extern __shared__ float ring[];  // [taps][C]
-  __shared__ float red[33];
-  auto norm_into = [&](int tok, float* dst) {
-    float s = 0.f, mean, inv;
-    for (int c = threadIdx.x * VEC; c < C; c += HR_THREADS * VEC) {
-      float f[VEC];
-      ldv<VEC>(x + (size_t)tok * C + c, f);
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) { s += f[e]; dst[c + e] = f[e]; }
-    }
-    row_stats<VEC>(dst, C, kind, eps, s, red, mean, inv);
-    for (int c = threadIdx.x * VEC; c < C; c += HR_THREADS * VEC) {
-      float f[VEC], bb[VEC];
-      ldv<VEC>(w + c, f);
-      if (b) ldv<VEC>(b + c, bb);
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) dst[c + e] = (dst[c + e] - mean) * inv * f[e] + (b ? bb[e] : 0.f);
-    }
-  };
-  if (tails) {
+                                                               int N, int C, int taps, int kind, float eps, int tile, int mode) {
+  extern __shared__ float2 stats[];  // (mean, 1 / deviation) of rows r0 .. last - 1
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  int first = blockIdx.x * tile, last = min(N, first + tile);
+  if (mode == 2) {
     const int* m = meta + 4 * blockIdx.x;
-    float* st = state + (size_t)m[2] * (taps - 1) * C;
-    for (int r = 0; r < taps - 1; ++r) {  // new row r: `back` tokens before the last one; ascending, so old rows shift down
-      int src = m[1] - 1 - (taps - 2 - r);
-      if (src >= 0) {
-        norm_into(m[0] + src, ring);
-        for (int c = threadIdx.x * VEC; c < C; c += HR_THREADS * VEC) stv<VEC>(st + (size_t)r * C + c, ring + c);
-      } else {  // an input of an earlier step: it moves down by the tokens of this one
-        for (int c = threadIdx.x * VEC; c < C; c += HR_THREADS * VEC) {
-          float f[VEC];
-          ldv<VEC>(st + (size_t)(r + m[1]) * C + c, f);
-          stv<VEC>(st + (size_t)r * C + c, f);
-        }
-      }
-    }
-    return;
+    last = m[0] + m[1];
+    first = last;
   }
-  int seq = -1, cur = 0;
-  const int first = blockIdx.x * tile, last = min(N, first + tile);
-  for (int tok = first; tok < last; ++tok) {
-    const int* m = meta + 4 * tok_seq[tok];
-    if (tok_seq[tok] != seq) {  // (re)fill the ring with the taps - 1 rows before this one
-      seq = tok_seq[tok];
-      int local = tok - m[0];
-      const float* st = state ? state + (size_t)m[2] * (taps - 1) * C : nullptr;
-      for (int k = taps - 1; k >= 1; --k) {
-        float* dst = ring + (size_t)((cur + 2 * taps - k) % taps) * C;
-        if (local - k >= 0) {
-          norm_into(tok - k, dst);
-        } else {
-          bool before = m[3] + local - k < 0;
-          for (int c = threadIdx.x * VEC; c < C; c += HR_THREADS * VEC) {
-            float f[VEC];
-            if (!before) ldv<VEC>(st + (size_t)(taps - 1 + local - k) * C + c, f);
+  const int r0 = max(0, first - (taps - 1));
+  for (int r = r0 + warp; r < last; r += HR_THREADS / 32) {
+    const float* row = x + (size_t)r * C;
+    float mean = 0.f, s = 0.f, ss = 0.f;
+    if (kind == 0) {
+#pragma unroll 8
+      for (int c = lane * VEC; c < C; c += 32 * VEC) {
+        float f[VEC];
+        ldv<VEC>(row + c, f);
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) dst[c + e] = before ? 0.f : f[e];
-          }
-        }
+        for (int e = 0; e < VEC; ++e) s += f[e];
       }
+      mean = warp_sum(s) / C;
     }
-    float* h = ring + (size_t)cur * C;
-    norm_into(tok, h);
-    for (int c = threadIdx.x * VEC; c < C; c += HR_THREADS * VEC) {
-      float acc[VEC], f[VEC], o[VEC];
+#pragma unroll 8
+    for (int c = lane * VEC; c < C; c += 32 * VEC) {
+      float f[VEC];
+      ldv<VEC>(row + c, f);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss += (f[e] - mean) * (f[e] - mean);
+    }
+    ss = warp_sum(ss);
+    if (lane == 0) stats[r - r0] = make_float2(mean, 1.f / sqrtf(ss / C + eps));
+  }
+  __syncthreads();
+  auto normed = [&](int r, int c, const float* wv, const float* bv, float* o) {
+    float2 t = stats[r - r0];
+    ldv<VEC>(x + (size_t)r * C + c, o);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) o[e] = (o[e] - t.x) * t.y * wv[e] + bv[e];
+  };
+  for (int c = threadIdx.x * VEC; c < C; c += HR_THREADS * VEC) {
+    float wv[VEC], bv[VEC];
+    ldv<VEC>(w + c, wv);
+    if (b) ldv<VEC>(b + c, bv);
+    else
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) bv[e] = 0.f;
+    // the state rows of a sequence after its token `tok` (the last one): ascending, so an old row moves down in place
+    auto advance = [&](const int* m, int tok) {
+      float* st = state + (size_t)m[2] * (taps - 1) * C + c;
+      for (int r = 0; r < taps - 1; ++r) {
+        int local = tok - m[0] - (taps - 2 - r);
+        float f[VEC];
+        if (local >= 0) {
+          normed(m[0] + local, c, wv, bv, f);
+        } else if (m[3] + local < 0) {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) f[e] = 0.f;
+        } else {
+          ldv<VEC>(st + (size_t)(r + m[1]) * C, f);
+        }
+        stv<VEC>(st + (size_t)r * C, f);
+      }
+    };
+    if (mode == 2) {
+      advance(meta + 4 * blockIdx.x, last - 1);
+      continue;
+    }
+    for (int tok = first; tok < last; ++tok) {
+      const int* m = meta + 4 * tok_seq[tok];
+      const int local = tok - m[0];
+      float acc[VEC], h[VEC], f[VEC];
 #pragma unroll
       for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
       for (int j = 0; j < taps; ++j) {
+        const int src = local - (taps - 1 - j);
+        if (src >= 0) {
+          normed(m[0] + src, c, wv, bv, h);
+        } else if (m[3] + src >= 0) {
+          ldv<VEC>(state + ((size_t)m[2] * (taps - 1) + (taps - 1 + src)) * C + c, h);
+        } else {
+          continue;  // before the sequence's start, whatever the slot holds
+        }
         ldv<VEC>(conv_w + (size_t)j * C + c, f);
-        const float* hj = ring + (size_t)((cur + 1 + j) % taps) * C + c;  // lag taps-1-j; j = taps-1 is the row itself
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) acc[e] += f[e] * hj[e];
+        for (int e = 0; e < VEC; ++e) acc[e] += f[e] * h[e];
       }
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) o[e] = h[c + e] + acc[e];
-      stv<VEC>(out + (size_t)tok * C + c, o);
+      for (int e = 0; e < VEC; ++e) acc[e] += h[e];  // the last tap read the row itself
+      stv<VEC>(out + (size_t)tok * C + c, acc);
+      if (mode == 1 && local == m[1] - 1) advance(m, tok);
     }
-    cur = (cur + 1) % taps;
   }
 }
 
 // z -> a N(z) + b N(z^2) + c N(z^3) + e, powers taken entry by entry, N(v) = v / sqrt(mean(v^2) + eps) over the row.
-// One block per row; the three sums of squares are reduced together.  Rows of up to PN_KEEP * 8 values per thread stay
-// in registers between the sums and the result.
-#define PN_KEEP 4
+// One block per row, as many threads as the row fills with 8 values each (at most 1024); the three sums of squares are
+// reduced together.  Rows of up to PN_KEEP * 8 values per thread stay in registers between the sums and the result.
+#define PN_KEEP 2
 template <typename T, bool VEC8>
-__global__ void __launch_bounds__(HR_THREADS) poly_norm_kernel(const T* z, long long z_stride, T* out, long long out_stride,
-                                                               const float* __restrict__ coef, int F, float eps) {
-  __shared__ float red[3][HR_THREADS / 32];
+__global__ void __launch_bounds__(1024) poly_norm_kernel(const T* z, long long z_stride, T* out, long long out_stride,
+                                                         const float* __restrict__ coef, int F, float eps) {
+  __shared__ float red[3][32];
   const T* src = z + (size_t)blockIdx.x * z_stride;
   T* dst = out + (size_t)blockIdx.x * out_stride;
   float s1 = 0.f, s2 = 0.f, s3 = 0.f;
@@ -292,37 +307,35 @@ __global__ void __launch_bounds__(HR_THREADS) poly_norm_kernel(const T* z, long 
   if (VEC8) {
 #pragma unroll
     for (int k = 0; k < PN_KEEP; ++k) {
-      int c = (threadIdx.x + k * HR_THREADS) * 8;
-      if (c < F) {
-        load8(src + c, keep[k]);
+      int c = (threadIdx.x + k * blockDim.x) * 8;
+      if (c < F) load8(src + c, keep[k]);
+    }
+#pragma unroll
+    for (int k = 0; k < PN_KEEP; ++k)
+      if ((threadIdx.x + k * blockDim.x) * 8 < F)
 #pragma unroll
         for (int e = 0; e < 8; ++e) add(keep[k][e]);
-      }
-    }
   } else {
-    for (int c = threadIdx.x; c < F; c += HR_THREADS) add(to_f(src[c]));
+    for (int c = threadIdx.x; c < F; c += blockDim.x) add(to_f(src[c]));
   }
   s1 = warp_sum(s1);
   s2 = warp_sum(s2);
   s3 = warp_sum(s3);
-  if ((threadIdx.x & 31) == 0) {
+  const int lane = threadIdx.x & 31, nw = (blockDim.x + 31) >> 5;
+  if (lane == 0) {
     red[0][threadIdx.x >> 5] = s1;
     red[1][threadIdx.x >> 5] = s2;
     red[2][threadIdx.x >> 5] = s3;
   }
   __syncthreads();
-  s1 = s2 = s3 = 0.f;
-#pragma unroll
-  for (int i = 0; i < HR_THREADS / 32; ++i) {
-    s1 += red[0][i];
-    s2 += red[1][i];
-    s3 += red[2][i];
-  }
+  s1 = warp_sum(lane < nw ? red[0][lane] : 0.f);
+  s2 = warp_sum(lane < nw ? red[1][lane] : 0.f);
+  s3 = warp_sum(lane < nw ? red[2][lane] : 0.f);
   const float a = coef[0] / sqrtf(s1 / F + eps), b = coef[1] / sqrtf(s2 / F + eps), c3 = coef[2] / sqrtf(s3 / F + eps), e0 = coef[3];
   if (VEC8) {
 #pragma unroll
     for (int k = 0; k < PN_KEEP; ++k) {
-      int c = (threadIdx.x + k * HR_THREADS) * 8;
+      int c = (threadIdx.x + k * blockDim.x) * 8;
       if (c < F) {
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
@@ -333,7 +346,7 @@ __global__ void __launch_bounds__(HR_THREADS) poly_norm_kernel(const T* z, long 
       }
     }
   } else {
-    for (int c = threadIdx.x; c < F; c += HR_THREADS) {
+    for (int c = threadIdx.x; c < F; c += blockDim.x) {
       float v = to_f(src[c]), v2 = v * v;
       dst[c] = from_f<T>(a * v + b * v2 + c3 * (v2 * v) + e0);
     }
@@ -411,23 +424,23 @@ int hyb_row_update(const RowUpdateArgs* args, int dt, cudaStream_t st) {
   return (int)cudaGetLastError();
 }
 
+// carries != 0: some sequence of the step reads its conv_state (it does not start at position 0)
 int hyb_norm_conv(const float* x, const void* w, const void* b, const float* conv_w, float* state, void* out, const int* meta,
-                  const int* tok_seq, int N, int nseq, int C, int taps, int kind, float eps, int tile, int dt, cudaStream_t st) {
+                  const int* tok_seq, int N, int nseq, int C, int taps, int kind, float eps, int tile, int carries, int dt,
+                  cudaStream_t st) {
   if (N == 0) return 0;
   if (taps < 1 || tile < 1 || C < 1 || (taps > 1 && !state)) return -2;
-  size_t smem = (size_t)taps * C * sizeof(float);
-  if (smem > 200 * 1024) return -3;
+  size_t smem = (size_t)(tile + taps) * sizeof(float2);
+  if (smem > 40 * 1024) return -3;
   bool vec = C % 4 == 0 && al16(x) && al16(w) && al16(b) && al16(conv_w) && al16(state) && al16(out);
-  int blocks = (N + tile - 1) / tile;
-#define NC(T, V)                                                                                                        \
-  do {                                                                                                                  \
-    if (smem > 40 * 1024)                                                                                               \
-      cudaFuncSetAttribute(norm_conv_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);             \
-    norm_conv_kernel<T, V><<<blocks, HR_THREADS, smem, st>>>(x, (const T*)w, (const T*)b, conv_w, state, (T*)out, meta, \
-                                                             tok_seq, N, C, taps, kind, eps, tile, 0);                  \
-    if (taps > 1)                                                                                                       \
-      norm_conv_kernel<T, V><<<nseq, HR_THREADS, smem, st>>>(x, (const T*)w, (const T*)b, conv_w, state, (T*)out, meta, \
-                                                             tok_seq, N, C, taps, kind, eps, tile, 1);                  \
+  int blocks = (N + tile - 1) / tile, mode = taps > 1 && !carries ? 1 : 0;
+#define NC(T, V)                                                                                                           \
+  do {                                                                                                                     \
+    norm_conv_kernel<T, V><<<blocks, HR_THREADS, smem, st>>>(x, (const T*)w, (const T*)b, conv_w, state, (T*)out, meta,    \
+                                                             tok_seq, N, C, taps, kind, eps, tile, mode);                  \
+    if (taps > 1 && carries)                                                                                               \
+      norm_conv_kernel<T, V><<<nseq, HR_THREADS, smem, st>>>(x, (const T*)w, (const T*)b, conv_w, state, (T*)out, meta,    \
+                                                             tok_seq, N, C, taps, kind, eps, tile, 2);                     \
   } while (0)
   if (dt == 0) { if (vec) NC(bf16, 4); else NC(bf16, 1); }
   else { if (vec) NC(float, 4); else NC(float, 1); }
@@ -439,8 +452,10 @@ int hyb_poly_norm(const void* z, long long z_stride, void* out, long long out_st
                   int dt, cudaStream_t st) {
   if (rows == 0) return 0;
   if (F < 1) return -2;
-  bool vec = F % 8 == 0 && F <= PN_KEEP * 8 * HR_THREADS && z_stride % 8 == 0 && out_stride % 8 == 0 && al16(z) && al16(out);
-#define PN(T, V) poly_norm_kernel<T, V><<<rows, HR_THREADS, 0, st>>>((const T*)z, z_stride, (T*)out, out_stride, coef, F, eps)
+  bool vec = F % 8 == 0 && F <= PN_KEEP * 8 * 1024 && z_stride % 8 == 0 && out_stride % 8 == 0 && al16(z) && al16(out);
+  int per = vec ? F / 8 : F, th = per >= 1024 ? 1024 : (per + 31) / 32 * 32;
+  if (vec && th > 256 && rows >= 1184) th = ((per + PN_KEEP - 1) / PN_KEEP + 31) / 32 * 32;  // many rows: fewer, busier warps per row
+#define PN(T, V) poly_norm_kernel<T, V><<<rows, th, 0, st>>>((const T*)z, z_stride, (T*)out, out_stride, coef, F, eps)
   if (dt == 0) { if (vec) PN(bf16, true); else PN(bf16, false); }
   else { if (vec) PN(float, true); else PN(float, false); }
 #undef PN

@@ -89,7 +89,7 @@ def lib() -> ctypes.CDLL:
     h.hyb_rotate_heads.argtypes = [vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp]
     h.hyb_latent_attn.argtypes = [vp, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, vp, vp, i32, vp, i32, i32, i32, vp]
     h.hyb_row_update.argtypes = [ctypes.POINTER(_RowUpdateArgs), i32, vp]
-    h.hyb_norm_conv.argtypes = [vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, i32, vp]
+    h.hyb_norm_conv.argtypes = [vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, i32, i32, vp]
     h.hyb_poly_norm.argtypes = [vp, i64, vp, i64, vp, i32, i32, f32, i32, vp]
     h.hyb_embed_pairs.argtypes = [vp, vp, vp, vp, vp, i32, i32, i32, f32, i64, i64, i64, vp, vp, vp, i32, i32, vp]
     h.hyb_causal_softmax.argtypes = [vp, vp, i64, i32, i32, i32, f32, i32, i32, i32, i32, f32, vp, i32, i32, vp]
@@ -1136,11 +1136,11 @@ def norm_conv(x: torch.Tensor, nxt: NextInput, plan: BatchPlan, out_dtype: torch
     if not x.is_contiguous() or nxt.w.dtype != out_dtype:
         raise HybridOpsError("the residual rows are dense; norm weights have the activation type")
     out = torch.empty(N, C, device=x.device, dtype=out_dtype)
-    tile = tile or max(1, min(16, N // (4 * _SM_TARGET)))
+    tile = tile or max(1, min(9 - min(taps, 4), N // _SM_TARGET))  # with its taps - 1 earlier rows: a row per warp
     _check(lib().hyb_norm_conv(x.data_ptr(), nxt.w.data_ptr(), None if nxt.b is None else nxt.b.data_ptr(), nxt.conv_w.data_ptr(),
                                None if taps == 1 else nxt.state.data_ptr(), out.data_ptr(), plan.meta.data_ptr(),
                                plan.tok_seq.data_ptr(), N, len(plan.seqs), C, taps, _NORM_KINDS[nxt.kind], float(nxt.eps), tile,
-                               _dt(out), _st()), "norm_conv")
+                               int(any(p0 > 0 for _, _, _, p0 in plan.seqs)), _dt(out), _st()), "norm_conv")
     return out
 
 
