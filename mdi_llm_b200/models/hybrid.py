@@ -216,6 +216,7 @@ class LatentAttention(nn.Module, _Fused):
 
     expand_from = 64   # prompts: sequences that bring at least this many tokens, or all of theirs, take the expanded form
     query_block = 1024  # most rows of the score matrix alive at a time
+    fused_prompt = True  # False: always the batched matrix products
 
     def __init__(self, width: int, m: Dict[str, Any], eps: float, traits: Optional[Dict[str, Any]] = None) -> None:
         super().__init__()
@@ -280,9 +281,10 @@ class LatentAttention(nn.Module, _Fused):
         return H.linear(o, self.o)
 
     def _expanded(self, q: torch.Tensor, cache: torch.Tensor, plan: H.BatchPlan) -> torch.Tensor:
-        """Prompt form: keys and values are expanded from the cached rows once per step (one matrix product), scores and
-        the weighted sum are batched matrix products over heads, the masked softmax runs on fp32 scores in between, per
-        band of query rows against the keys the band can see.  Decoding instead carries the query into the latent space
+        """Prompt form: keys and values are expanded from the cached rows once per step (one matrix product).  With 16-bit
+        activations the attention over them is one kernel per sequence (``H.prompt_attn``); else (fp32, sizes that kernel
+        does not take) scores and the weighted sum are batched matrix products over heads with the masked softmax on fp32
+        scores in between, per band of query rows against the keys the band can see.  Decoding instead carries the query into the latent space
         and reads the cache directly (``H.latent_attn``): per query that costs ``kv_rank`` instead of ``dim`` multiplies per key
         and head, which only pays when there is a single query.  Returns ``[N, heads, vdim]``."""
         Hh, D, R, V, W = self.H, self.D, self.R, self.V, self.window
@@ -294,6 +296,8 @@ class LatentAttention(nn.Module, _Fused):
             first = max(0, p0 - W + 1) if W > 0 else 0
             kv = H.linear(cache[slot, first:p0 + n], self.w_kv)
             keys = kv.size(0)
+            if self.fused_prompt and H.prompt_attn(q[r0:r0 + n], kv, Hh, DK, V, p0, first, self.scale, W, out[r0:r0 + n]) is not None:
+                continue
             kt = kv[:, :Hh * DK].view(keys, Hh, DK).permute(1, 2, 0)   # [H, D+R, keys]
             v = kv[:, Hh * DK:].view(keys, Hh, V).transpose(0, 1)      # [H, keys, V]
             qh = q[r0:r0 + n].view(n, Hh, DK).transpose(0, 1)          # [H, n, D+R]

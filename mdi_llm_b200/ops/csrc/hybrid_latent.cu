@@ -1,0 +1,442 @@
+// Tensor-core forms of latent attention with 16-bit activations (the fp32 mode and shapes outside the stated multiples use
+// the kernels of hybrid_mixers.cu and library matrix products):
+//
+//  * latent_decode_mma_kernel: one-token steps and short portions, straight on the cached rows [L latent | R rotated key].
+//    All heads read the same rows, so 16 heads of a token are the rows of one matrix-product tile.
+//  * prompt_attn_mma_kernel: prompts, on keys and values expanded per head, scores and weights never leave the SM.
+//
+// Queries of the first kernel and softmax weights of both enter the products as a bf16 number plus the bf16 remainder, so
+// they keep twice the mantissa; sums are fp32.  Warp-level m16n8k16 products: the tiles are 16 and 64 rows high and a
+// step is bound by reading the cache (first kernel) or by its many small dependent tiles (second), see the bounds there.
+#include "hybrid_common.cuh"
+
+namespace hyb {
+
+__device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+// 16 bytes to shared memory; valid == false writes zeros and reads nothing
+__device__ __forceinline__ void cp16(bf16* dst, const bf16* src, bool valid) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(valid ? 16 : 0));
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;"); }
+template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N)); }
+__device__ __forceinline__ void ldm4(uint32_t* r, const bf16* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void ldm4t(uint32_t* r, const bf16* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void ldm2(uint32_t* r, const bf16* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void ldm2t(uint32_t* r, const bf16* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(smem_u32(p)));
+}
+// c[16 x 8] += a[16 x 16] b[16 x 8]; lane (g = lane / 4, t = lane % 4) holds c = {(g, 2t), (g, 2t+1), (g+8, 2t), (g+8, 2t+1)}
+__device__ __forceinline__ void mma(float* c, const uint32_t* a, const uint32_t* b) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
+}
+__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
+  __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+  __nv_bfloat162 l = __floats2bfloat162_rn(x - __bfloat162float(h.x), y - __bfloat162float(h.y));
+  hi = *reinterpret_cast<uint32_t*>(&h);
+  lo = *reinterpret_cast<uint32_t*>(&l);
+}
+
+// Block = one token x 16 heads x one share of its keys, 4 warps.  Tiles of 32 cached rows arrive by asynchronous 16-byte
+// copies, two buffers.  Per tile: warp w computes the scores of keys 8w .. 8w+7 for the 16 heads (queries as hi + lo),
+// then the softmax of heads 4w .. 4w+3 (lane = key), then the weighted sum for its quarter of the latent.
+// Needs L + R a multiple of 16, L a multiple of 32 and at most 32 * NT (NT: 8-column tiles of a warp's quarter).
+#define LD_TILE 32
+template <int NT>
+__global__ void __launch_bounds__(128) latent_decode_mma_kernel(const float* __restrict__ qlat, const bf16* __restrict__ q,
+                                                                long long q_stride, const bf16* __restrict__ cache,
+                                                                long long slot_stride, const int* __restrict__ meta,
+                                                                const int* __restrict__ tok_seq, bf16* __restrict__ out, int N,
+                                                                int H, int D, int R, int L, float scale, int nsplit,
+                                                                float* __restrict__ part_acc, float* __restrict__ part_ml,
+                                                                int window, const float* __restrict__ inv_freq, int nrot,
+                                                                int interleaved) {
+  extern __shared__ __align__(16) unsigned char raw[];
+  __shared__ float ss[16][LD_TILE + 1];
+  __shared__ __align__(16) bf16 ph[16][LD_TILE + 8], pl[16][LD_TILE + 8];
+  __shared__ float corr[16], fin[16];
+  const int Dk = L + R, ld = Dk + 8;
+  bf16* qh = reinterpret_cast<bf16*>(raw);        // [16][ld]
+  bf16* ql = qh + 16 * ld;                        // [16][ld]
+  bf16* kt = ql + 16 * ld;                        // [2][LD_TILE][ld]
+  float2* cs = reinterpret_cast<float2*>(kt + 2 * LD_TILE * ld);  // [nrot / 2] (cos, sin) of the token's angles
+  const int tok = blockIdx.x, h0 = blockIdx.y * 16, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int* m = meta + 4 * tok_seq[tok];
+  const int pos = m[3] + tok - m[0], first = window > 0 ? max(0, pos - window + 1) : 0, nkeys = pos + 1 - first;
+  const bf16* rows = cache + (size_t)m[2] * slot_stride + (size_t)first * Dk;
+  const int chunk = ((nkeys + nsplit - 1) / nsplit + LD_TILE - 1) / LD_TILE * LD_TILE;
+  const int k_begin = blockIdx.z * chunk, k_end = min(nkeys, k_begin + chunk);
+  const int per = Dk >> 3;
+  auto fetch = [&](int t0, bf16* dst) {
+    for (int i = tid; i < LD_TILE * per; i += 128) {
+      int j = i / per, c = (i - j * per) * 8;
+      bool ok = t0 + j < k_end;
+      cp16(dst + j * ld + c, rows + (size_t)(ok ? t0 + j : k_begin) * Dk + c, ok);
+    }
+    cp_commit();
+  };
+  const bool any = k_begin < k_end;
+  if (any) fetch(k_begin, kt);
+  if (inv_freq)
+    for (int i = tid; i < nrot / 2; i += 128) sincosf((float)pos * inv_freq[i], &cs[i].y, &cs[i].x);
+  __syncthreads();
+  for (int i = tid; i < 16 * Dk; i += 128) {
+    int hh = i / Dk, d = i - hh * Dk, h = h0 + hh;
+    float v = 0.f;
+    if (h < H) {
+      if (d < L) {
+        v = qlat[((size_t)h * N + tok) * L + d];
+      } else {
+        const bf16* qr = q + (size_t)tok * q_stride + (size_t)h * (D + R) + D;
+        int r = d - L;
+        v = to_f(qr[r]);
+        if (inv_freq && r < nrot) {
+          int half = nrot / 2, p = interleaved ? r >> 1 : (r < half ? r : r - half);
+          int a = interleaved ? 2 * p : p, b = interleaved ? 2 * p + 1 : p + half;
+          float2 t = cs[p];
+          v = r == a ? v * t.x - to_f(qr[b]) * t.y : v * t.x + to_f(qr[a]) * t.y;
+        }
+      }
+      v *= scale;
+    }
+    bf16 hi = __float2bfloat16_rn(v);
+    qh[hh * ld + d] = hi;
+    ql[hh * ld + d] = __float2bfloat16_rn(v - __bfloat162float(hi));
+  }
+  float mx[4], l[4], acc[NT][4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) { mx[i] = -INFINITY; l[i] = 0.f; }
+#pragma unroll
+  for (int i = 0; i < NT; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
+  const int nt = L >> 5, col0 = warp * (L >> 2), g = lane >> 2, t2 = (lane & 3) * 2;
+  int buf = 0;
+  for (int t0 = k_begin; t0 < k_end; t0 += LD_TILE, buf ^= 1) {
+    bf16* k = kt + buf * LD_TILE * ld;
+    if (t0 + LD_TILE < k_end) { fetch(t0 + LD_TILE, kt + (buf ^ 1) * LD_TILE * ld); cp_wait<1>(); }
+    else cp_wait<0>();
+    __syncthreads();
+    {
+      float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
+      const bf16* ap = qh + (lane & 15) * ld + (lane >> 4) * 8;
+      const bf16* al = ql + (lane & 15) * ld + (lane >> 4) * 8;
+      const bf16* bp = k + (warp * 8 + (lane & 7)) * ld + ((lane >> 3) & 1) * 8;
+#pragma unroll 4
+      for (int kk = 0; kk < Dk; kk += 16) {
+        uint32_t a[4], b[2];
+        ldm2(b, bp + kk);
+        ldm4(a, ap + kk);
+        mma(c0, a, b);
+        ldm4(a, al + kk);
+        mma(c1, a, b);
+      }
+      int c = warp * 8 + t2;
+      ss[g][c] = c0[0] + c1[0];
+      ss[g][c + 1] = c0[1] + c1[1];
+      ss[g + 8][c] = c0[2] + c1[2];
+      ss[g + 8][c + 1] = c0[3] + c1[3];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      int hh = warp * 4 + i;
+      float s = t0 + lane < k_end ? ss[hh][lane] : -INFINITY;
+      float mn = fmaxf(mx[i], warp_max(s));  // finite: a tile holds at least one key
+      float cr = expf(mx[i] - mn), p = expf(s - mn);
+      l[i] = l[i] * cr + warp_sum(p);
+      mx[i] = mn;
+      bf16 hi = __float2bfloat16_rn(p);
+      ph[hh][lane] = hi;
+      pl[hh][lane] = __float2bfloat16_rn(p - __bfloat162float(hi));
+      if (lane == 0) corr[hh] = cr;
+    }
+    __syncthreads();
+    {
+      const float ca = corr[g], cb = corr[g + 8];
+      uint32_t a[2][4], al[2][4];
+#pragma unroll
+      for (int s = 0; s < 2; ++s) {
+        ldm4(a[s], &ph[lane & 15][s * 16 + (lane >> 4) * 8]);
+        ldm4(al[s], &pl[lane & 15][s * 16 + (lane >> 4) * 8]);
+      }
+#pragma unroll
+      for (int i = 0; i < NT; ++i)
+        if (i < nt) {
+          acc[i][0] *= ca; acc[i][1] *= ca; acc[i][2] *= cb; acc[i][3] *= cb;
+#pragma unroll
+          for (int s = 0; s < 2; ++s) {
+            uint32_t b[2];
+            ldm2t(b, k + (s * 16 + (lane & 15)) * ld + col0 + i * 8);
+            mma(acc[i], a[s], b);
+            mma(acc[i], al[s], b);
+          }
+        }
+    }
+    __syncthreads();
+  }
+  if (lane == 0)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      int h = h0 + warp * 4 + i;
+      fin[warp * 4 + i] = nsplit == 1 ? 1.f / l[i] : 1.f;
+      if (nsplit > 1 && h < H) {
+        size_t b = ((size_t)blockIdx.z * H + h) * N + tok;
+        part_ml[b * 2] = mx[i];
+        part_ml[b * 2 + 1] = l[i];
+      }
+    }
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < NT; ++i)
+    if (i < nt) {
+      int c = col0 + i * 8 + t2;
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        int hh = g + 8 * r, h = h0 + hh;
+        if (h >= H) continue;
+        float x = acc[i][2 * r] * fin[hh], y = acc[i][2 * r + 1] * fin[hh];
+        if (nsplit == 1) *reinterpret_cast<__nv_bfloat162*>(out + ((size_t)h * N + tok) * L + c) = __floats2bfloat162_rn(x, y);
+        else *reinterpret_cast<float2*>(part_acc + (((size_t)blockIdx.z * H + h) * N + tok) * L + c) = make_float2(x, y);
+      }
+    }
+}
+
+// Merge of the key shares: one warp per (token, head), nsplit <= 32.  Lane z reads share z's maximum and denominator, the
+// weights e^(m_z - m) are handed round by shuffles while the lanes walk the latent four values at a time.
+__global__ void latent_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml, bf16* __restrict__ out,
+                                    int N, int H, int L, int nsplit) {
+  int tok = blockIdx.x, h = blockIdx.y, w = threadIdx.x >> 5, nw = blockDim.x >> 5, lane = threadIdx.x & 31;
+  float ms = -INFINITY, ls = 0.f;
+  if (lane < nsplit) {
+    const float* ml = part_ml + (((size_t)lane * H + h) * N + tok) * 2;
+    ms = ml[0];
+    ls = ml[1];
+  }
+  float M = warp_max(ms);
+  float ws = lane < nsplit ? expf(ms - M) : 0.f;  // a share without keys: exp(-inf) = 0
+  float inv = 1.f / warp_sum(ls * ws);
+  for (int d0 = w * 128; d0 < L; d0 += nw * 128) {
+    int d = d0 + 4 * lane;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+    for (int z = 0; z < nsplit; ++z) {
+      float wz = __shfl_sync(0xffffffffu, ws, z);
+      if (d < L) {
+        float4 x = *reinterpret_cast<const float4*>(part_acc + (((size_t)z * H + h) * N + tok) * L + d);
+        a.x += x.x * wz; a.y += x.y * wz; a.z += x.z * wz; a.w += x.w * wz;
+      }
+    }
+    if (d < L) {
+      __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(out + ((size_t)h * N + tok) * L + d);
+      o[0] = __floats2bfloat162_rn(a.x * inv, a.y * inv);
+      o[1] = __floats2bfloat162_rn(a.z * inv, a.w * inv);
+    }
+  }
+}
+
+// Prompt attention of one sequence: query row i (position p0 + i) against the expanded keys of positions first .. first +
+// keys - 1, of which it sees those not later than itself and (window > 0) fewer than `window` positions back.
+// q rows: [H][DK] (rotated); kv rows: [H][DK] keys, then [H][V] values; out [n][H][V].
+// Block = 64 query rows of one head, 4 warps of 16 rows; key tiles of 64, two buffers, filled by asynchronous 16-byte copies
+// while the tile before is used.  Scores and softmax weights stay in registers.  Needs DK and V multiples of 16, V <= 8 NV.
+#define PA_ROWS 64
+#define PA_KEYS 64
+template <int NV>
+__global__ void __launch_bounds__(128) prompt_attn_mma_kernel(const bf16* __restrict__ q, long long q_stride,
+                                                              const bf16* __restrict__ kv, long long kv_stride,
+                                                              bf16* __restrict__ out, int n, int H, int DK, int V, int keys,
+                                                              int p0, int first, int window, float scale_log2e) {
+  extern __shared__ __align__(16) unsigned char raw[];
+  const int ldk = DK + 8, ldv = V + 8;
+  bf16* qs = reinterpret_cast<bf16*>(raw);     // [64][ldk]
+  bf16* ks = qs + PA_ROWS * ldk;               // [2][64][ldk]
+  bf16* vs = ks + 2 * PA_KEYS * ldk;           // [2][64][ldv]
+  const int h = blockIdx.y, i0 = (gridDim.x - 1 - blockIdx.x) * PA_ROWS;  // long rows of work first
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t2 = (lane & 3) * 2;
+  const int dk8 = DK >> 3, v8 = V >> 3;
+  const int kb = window > 0 ? max(0, p0 + i0 - window + 1 - first) : 0;
+  const int ke = min(keys, p0 + min(n, i0 + PA_ROWS) - first);
+  const bf16* kbase = kv + (size_t)h * DK;
+  const bf16* vbase = kv + (size_t)H * DK + (size_t)h * V;
+  auto fetch = [&](int j0, int buf) {
+    for (int i = tid; i < PA_KEYS * dk8; i += 128) {
+      int j = i / dk8, c = (i - j * dk8) * 8;
+      bool ok = j0 + j < ke;
+      cp16(ks + (buf * PA_KEYS + j) * ldk + c, kbase + (size_t)(ok ? j0 + j : kb) * kv_stride + c, ok);
+    }
+    for (int i = tid; i < PA_KEYS * v8; i += 128) {
+      int j = i / v8, c = (i - j * v8) * 8;
+      bool ok = j0 + j < ke;
+      cp16(vs + (buf * PA_KEYS + j) * ldv + c, vbase + (size_t)(ok ? j0 + j : kb) * kv_stride + c, ok);
+    }
+    cp_commit();
+  };
+  for (int i = tid; i < PA_ROWS * dk8; i += 128) {
+    int j = i / dk8, c = (i - j * dk8) * 8;
+    bool ok = i0 + j < n;
+    cp16(qs + j * ldk + c, q + (size_t)(ok ? i0 + j : 0) * q_stride + (size_t)h * DK + c, ok);
+  }
+  fetch(kb, 0);  // kb < ke: row i0 sees at least itself
+  float o[NV][4], mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) o[i][e] = 0.f;
+  const int nv2 = V >> 4;
+  const int pr0 = p0 + i0 + warp * 16 + g - first;  // this lane's rows (pr0, pr0 + 8) as key indices
+  int buf = 0;
+  for (int j0 = kb; j0 < ke; j0 += PA_KEYS, buf ^= 1) {
+    if (j0 + PA_KEYS < ke) { fetch(j0 + PA_KEYS, buf ^ 1); cp_wait<1>(); }
+    else cp_wait<0>();
+    __syncthreads();
+    float s[8][4];
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[i][e] = 0.f;
+    const bf16* ap = qs + (warp * 16 + (lane & 15)) * ldk + (lane >> 4) * 8;
+    const bf16* bp = ks + (buf * PA_KEYS + (lane & 7) + (lane >> 4) * 8) * ldk + ((lane >> 3) & 1) * 8;
+#pragma unroll 2
+    for (int kk = 0; kk < DK; kk += 16) {
+      uint32_t a[4], b[4];
+      ldm4(a, ap + kk);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        ldm4(b, bp + i * 16 * ldk + kk);
+        mma(s[2 * i], a, b);
+        mma(s[2 * i + 1], a, b + 2);
+      }
+    }
+    float mn[2] = {mx[0], mx[1]};
+    // tiles wholly inside every row's range need no mask
+    const bool edge = j0 + PA_KEYS - 1 > p0 + i0 - first || (window > 0 && p0 + i0 + PA_ROWS - 1 - first - j0 >= window) || j0 + PA_KEYS > ke;
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        float v = s[i][e] * scale_log2e;
+        if (edge) {
+          int j = j0 + i * 8 + t2 + (e & 1), p = pr0 + (e >> 1) * 8;
+          if (j > p || j >= ke || (window > 0 && p - j >= window)) v = -INFINITY;
+        }
+        s[i][e] = v;
+        mn[e >> 1] = fmaxf(mn[e >> 1], v);
+      }
+    float cr[2];
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      mn[r] = fmaxf(mn[r], __shfl_xor_sync(0xffffffffu, mn[r], 1));
+      mn[r] = fmaxf(mn[r], __shfl_xor_sync(0xffffffffu, mn[r], 2));
+      float safe = mn[r] == -INFINITY ? 0.f : mn[r];  // a row that has seen no key yet
+      cr[r] = exp2f(mx[r] - safe);
+      mx[r] = mn[r];
+      mn[r] = safe;
+      l[r] *= cr[r];
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) { o[i][0] *= cr[0]; o[i][1] *= cr[0]; o[i][2] *= cr[1]; o[i][3] *= cr[1]; }
+    const bf16* vp = vs + (buf * PA_KEYS + (lane & 15)) * ldv + (lane >> 4) * 8;
+#pragma unroll
+    for (int kk = 0; kk < PA_KEYS / 16; ++kk) {
+      uint32_t hi[4], lo[4];
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        float* p = s[2 * kk + u];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          p[e] = exp2f(p[e] - mn[e >> 1]);
+          l[e >> 1] += p[e];
+        }
+        split2(p[0], p[1], hi[2 * u], lo[2 * u]);
+        split2(p[2], p[3], hi[2 * u + 1], lo[2 * u + 1]);
+      }
+#pragma unroll
+      for (int i = 0; i < NV / 2; ++i)
+        if (i < nv2) {
+          uint32_t b[4];
+          ldm4t(b, vp + kk * 16 * ldv + i * 16);
+          mma(o[2 * i], hi, b);
+          mma(o[2 * i + 1], hi, b + 2);
+          mma(o[2 * i], lo, b);
+          mma(o[2 * i + 1], lo, b + 2);
+        }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
+    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
+    int row = i0 + warp * 16 + g + 8 * r;
+    if (row >= n) continue;
+    float inv = 1.f / l[r];
+    bf16* dst = out + ((size_t)row * H + h) * V + t2;
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+      if (i * 8 < V) *reinterpret_cast<__nv_bfloat162*>(dst + i * 8) = __floats2bfloat162_rn(o[i][2 * r] * inv, o[i][2 * r + 1] * inv);
+  }
+}
+
+}  // namespace hyb
+
+using namespace hyb;
+
+extern "C" {
+
+// -3: a shape or alignment these kernels do not take (the caller has another form)
+int hyb_latent_decode_mma(const float* qlat, const void* q, long long q_stride, const void* cache, long long slot_stride,
+                          const int* meta, const int* tok_seq, void* out, int N, int H, int D, int R, int L, float scale, int nsplit,
+                          float* part_acc, float* part_ml, int window, const float* inv_freq, int nrot, int interleaved,
+                          cudaStream_t st) {
+  if (N == 0) return 0;
+  if (nsplit < 1 || nsplit > 32 || (nsplit > 1 && (!part_acc || !part_ml)) || nrot > R || (nrot & 1)) return -2;
+  int Dk = L + R;
+  if (Dk % 16 || L % 32 || L > 512 || slot_stride % 8 || ((uintptr_t)cache & 15)) return -3;
+  size_t smem = (size_t)(32 + 2 * LD_TILE) * (Dk + 8) * sizeof(bf16) + (size_t)(nrot / 2) * sizeof(float2);
+  if (smem > 200 * 1024) return -3;
+  dim3 grid(N, (H + 15) / 16, nsplit);
+#define LM(NT)                                                                                                           \
+  do {                                                                                                                   \
+    cudaFuncSetAttribute(latent_decode_mma_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);          \
+    latent_decode_mma_kernel<NT><<<grid, 128, smem, st>>>(qlat, (const bf16*)q, q_stride, (const bf16*)cache, slot_stride, \
+                                                          meta, tok_seq, (bf16*)out, N, H, D, R, L, scale, nsplit, part_acc, \
+                                                          part_ml, window, inv_freq, nrot, interleaved);                 \
+  } while (0)
+  if (L <= 128) LM(4); else LM(16);
+#undef LM
+  if (nsplit > 1) latent_merge_kernel<<<dim3(N, H), L > 256 ? 128 : 64, 0, st>>>(part_acc, part_ml, (bf16*)out, N, H, L, nsplit);
+  return (int)cudaGetLastError();
+}
+
+int hyb_prompt_attn_mma(const void* q, long long q_stride, const void* kv, long long kv_stride, void* out, int n, int H, int DK,
+                        int V, int keys, int p0, int first, int window, float scale, cudaStream_t st) {
+  if (n == 0) return 0;
+  if (first < 0 || keys != p0 + n - first || (window > 0 ? first > (p0 - window + 1 > 0 ? p0 - window + 1 : 0) : first != 0)) return -2;
+  uintptr_t bits = (uintptr_t)q | (uintptr_t)kv | (uintptr_t)out;
+  if (DK % 16 || V % 16 || V > 256 || q_stride % 8 || kv_stride % 8 || (bits & 15) || (long long)H * DK % 8 || scale <= 0.f) return -3;
+  size_t smem = ((size_t)(PA_ROWS + 2 * PA_KEYS) * (DK + 8) + (size_t)2 * PA_KEYS * (V + 8)) * sizeof(bf16);
+  if (smem > 200 * 1024) return -3;
+  dim3 grid((n + PA_ROWS - 1) / PA_ROWS, H);
+  const float sl = scale * 1.4426950408889634f;
+#define PM(NV)                                                                                                            \
+  do {                                                                                                                    \
+    cudaFuncSetAttribute(prompt_attn_mma_kernel<NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);             \
+    prompt_attn_mma_kernel<NV><<<grid, 128, smem, st>>>((const bf16*)q, q_stride, (const bf16*)kv, kv_stride, (bf16*)out, n, \
+                                                        H, DK, V, keys, p0, first, window, sl);                           \
+  } while (0)
+  if (V <= 64) PM(8); else if (V <= 128) PM(16); else PM(32);
+#undef PM
+  return (int)cudaGetLastError();
+}
+
+}  // extern "C"

@@ -31,7 +31,7 @@ __all__ = ["BatchPlan", "HybridOpsError", "lib", "embed_rows", "cast_into", "nor
            "rotary_inv_freq", "scaled_inv_freq", "linear_f32", "grouped_linear", "window_append", "window_attn", "head_gate", "relu2_",
            "token_side_gate", "router_topk", "moe_gemv", "gather_scale_rows", "combine_rows", "act_mul", "scaled_branches",
            "full_norm_append", "lightning_recurrence", "norm_gate_rows", "gated_sum_norm_accumulate", "embed_pairs",
-           "row_update", "norm_conv", "poly_norm", "latent_prepare", "rotate_heads", "NextInput"]
+           "row_update", "norm_conv", "poly_norm", "latent_prepare", "rotate_heads", "prompt_attn", "NextInput"]
 
 
 class HybridOpsError(RuntimeError):
@@ -88,6 +88,8 @@ def lib() -> ctypes.CDLL:
     h.hyb_latent_prepare.argtypes = [vp, i64, vp, vp, i32, vp, i64, vp, vp, vp, i64, vp, vp, i32, i32, i32, i32, i32, f32, i32, vp]
     h.hyb_rotate_heads.argtypes = [vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp]
     h.hyb_latent_attn.argtypes = [vp, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, vp, vp, i32, vp, i32, i32, i32, vp]
+    h.hyb_latent_decode_mma.argtypes = [vp, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, vp, vp, i32, vp, i32, i32, vp]
+    h.hyb_prompt_attn_mma.argtypes = [vp, i64, vp, i64, vp, i32, i32, i32, i32, i32, i32, i32, i32, f32, vp]
     h.hyb_row_update.argtypes = [ctypes.POINTER(_RowUpdateArgs), i32, vp]
     h.hyb_norm_conv.argtypes = [vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, i32, i32, vp]
     h.hyb_poly_norm.argtypes = [vp, i64, vp, i64, vp, i32, i32, f32, i32, vp]
@@ -447,8 +449,9 @@ def latent_attn(qlat: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, plan: 
     (``window > 0``: the last ``window`` positions up to the token's own).  The query of head ``h`` is
     ``[qlat[h, tok] | q[tok, h, D:]]``, the value of a row is its latent part.  ``qlat`` is used in fp32.  With
     ``inv_freq`` the second part of the query is not rotated yet: that happens as it is loaded (fp32, unrounded).
-    Returns the attended latents ``[H, N, L]``.  ``split`` (CUDA): key shares per query, 0 = chosen from the batch shape
-    and the window."""
+    Returns the attended latents ``[H, N, L]``.  ``split`` (CUDA, at most 32): key shares per query, 0 = chosen from the
+    batch shape and the window.  With bf16 activations, ``L`` a multiple of 32 (at most 512) and ``L + R`` of 16 the products
+    run on the tensor cores, queries and weights as a bf16 number plus its bf16 remainder; else on fp32 values."""
     N = q.size(0)
     if not q.is_cuda:
         out = torch.empty(H, N, L, dtype=q.dtype)
@@ -469,21 +472,51 @@ def latent_attn(qlat: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, plan: 
     qlat = qlat.float()
     qs, _ = _rows(q)
     out = torch.empty(H, N, L, device=q.device, dtype=q.dtype)
-    # few query tokens (decoding) cannot fill the GPU with one block per token and 8 heads: split the keys of each
+    mma = q.dtype == torch.bfloat16 and L % 32 == 0 and L <= 512 and (L + R) % 16 == 0 and cache.stride(0) % 8 == 0 \
+        and cache.data_ptr() % 16 == 0
+    # few query tokens (decoding) cannot fill the GPU with one block per token and group of heads: split the keys of each
     # query over several blocks and merge the partial softmaxes.  The split count depends only on the batch shape
     # and the window, so a captured step stays valid while contexts grow.
-    blocks = N * ((H + 7) // 8)
+    blocks = N * ((H + 15) // 16 if mma else (H + 7) // 8)
     tiles = (window + 31) // 32 if window > 0 else 32
-    nsplit = 1 if blocks >= 2 * _SM_TARGET or split == 1 else (split or max(1, min(32, tiles, (2 * _SM_TARGET) // blocks)))
+    nsplit = 1 if blocks >= 2 * _SM_TARGET or split == 1 else min(32, split or max(1, min(tiles, (2 * _SM_TARGET) // blocks)))
     pa = pm = None
     if nsplit > 1:
         pa = torch.empty(nsplit, H, N, L, device=q.device, dtype=torch.float32)
         pm = torch.empty(nsplit, H, N, 2, device=q.device, dtype=torch.float32)
+    if mma:
+        _check(lib().hyb_latent_decode_mma(qlat.data_ptr(), q.data_ptr(), qs, cache.data_ptr(), cache.stride(0), plan.meta.data_ptr(),
+                                           plan.tok_seq.data_ptr(), out.data_ptr(), N, H, D, R, L, float(scale), nsplit,
+                                           None if pa is None else pa.data_ptr(), None if pm is None else pm.data_ptr(), int(window),
+                                           None if inv_freq is None else inv_freq.data_ptr(), int(nrot), int(pairing == "pairs"), _st()),
+               "latent_decode_mma")
+        return out
     _check(lib().hyb_latent_attn(qlat.data_ptr(), q.data_ptr(), qs, cache.data_ptr(), cache.stride(0), plan.meta.data_ptr(),
                                  plan.tok_seq.data_ptr(), out.data_ptr(), N, H, D, R, L, float(scale), nsplit,
                                  None if pa is None else pa.data_ptr(), None if pm is None else pm.data_ptr(), int(window),
                                  None if inv_freq is None else inv_freq.data_ptr(), int(nrot), int(pairing == "pairs"), _dt(q),
                                  _st()), "latent_attn")
+    return out
+
+
+def prompt_attn(q: torch.Tensor, kv: torch.Tensor, H: int, DK: int, V: int, p0: int, first: int, scale: float,
+                window: int = 0, out: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """Causal attention of one sequence's rows ``q [n, H * DK]`` (positions ``p0 ..``) over ``kv [keys, H * DK + H * V]``: the keys
+    and values of positions ``first .. p0 + n - 1``, all heads side by side; ``window > 0``: the last ``window`` positions up to
+    the row's own.  Scores, softmax and weights stay on chip, weights enter the second product as a bf16 number plus its
+    bf16 remainder.  Returns (and fills) ``out [n, H, V]``; None when the kernel does not take the type, the sizes (``DK`` and
+    ``V`` multiples of 16, ``V`` at most 256) or the device."""
+    n, keys = q.size(0), kv.size(0)
+    smem = 2 * (192 * (DK + 8) + 128 * (V + 8))
+    if not q.is_cuda or q.dtype != torch.bfloat16 or DK % 16 or V % 16 or V > 256 or smem > 200 * 1024 \
+            or any(t.stride(0) % 8 or t.data_ptr() % 16 for t in (q, kv)):
+        return None
+    if keys != p0 + n - first or kv.size(1) != H * (DK + V) or q.size(1) != H * DK:
+        raise HybridOpsError("keys are those of positions first .. p0 + n - 1, heads side by side")
+    out = torch.empty(n, H, V, device=q.device, dtype=q.dtype) if out is None else out
+    assert out.is_contiguous()
+    _check(lib().hyb_prompt_attn_mma(q.data_ptr(), _rows(q)[0], kv.data_ptr(), _rows(kv)[0], out.data_ptr(), n, H, DK, V, keys, int(p0),
+                                     int(first), int(window), float(scale), _st()), "prompt_attn_mma")
     return out
 
 

@@ -330,8 +330,8 @@ def test_one_key_stands_out_just_inside_and_outside_the_window_and_later(where, 
             olat = H.latent_attn(qlat, q, cache, plan, Hh, D, R, L, m.scale, split=split, window=W, inv_freq=m.inv_freq, nrot=R, pairing="pairs")
             got = torch.einsum("hl,hvl->hv", olat[:, 0].double().cpu(), m.uv.double().cpu().view(Hh, V, L))
             torch.testing.assert_close(got.float(), want.float(), **tol)
-        for n, band in ((64, 1024), (70, 17), (pos + 1, 64)):  # the query is the last row of a portion of n tokens
-            m.query_block = band
+        for n, band, fused in ((64, 1024, False), (70, 17, False), (pos + 1, 64, False), (64, 64, True), (79, 64, True), (pos + 1, 64, True)):
+            m.query_block, m.fused_prompt = band, fused  # the query is the last row of a portion of n tokens
             qs = torch.randn(n, Hh * (D + R), generator=g).to(where, dtype)
             qs[-1] = q[0]
             plan = BatchPlan.make([n], [1], [pos + 1 - n], dev)
@@ -363,7 +363,8 @@ def test_both_forms_on_unequal_sequences_in_scattered_slots(where, dtype, shape,
     got = torch.einsum("hnl,hvl->nhv", olat.double().cpu(), m.uv.double().cpu().view(Hh, V, L))
     torch.testing.assert_close(got[rows].float(), want[rows], **tol)
     H.rotate_heads(q, m.inv_freq, plan, Hh, D, R, R, "pairs")
-    torch.testing.assert_close(m._expanded(q, cache, plan)[rows].float().cpu(), want[rows], **tol)
+    for m.fused_prompt in (True, False):
+        torch.testing.assert_close(m._expanded(q, cache, plan)[rows].float().cpu(), want[rows], **tol)
 
 
 @pytest.mark.parametrize("where", WHERE)
