@@ -296,7 +296,7 @@ class LatentAttention(nn.Module, _Fused):
             first = max(0, p0 - W + 1) if W > 0 else 0
             kv = H.linear(cache[slot, first:p0 + n], self.w_kv)
             keys = kv.size(0)
-            if self.fused_prompt and H.prompt_attn(q[r0:r0 + n], kv, Hh, DK, V, p0, first, self.scale, W, out[r0:r0 + n]) is not None:
+            if self.fused_prompt and H.prompt_attn(q[r0:r0 + n], kv, Hh, DK, V, p0, first, self.scale, W, out[r0:r0 + n], split) is not None:
                 continue
             kt = kv[:, :Hh * DK].view(keys, Hh, DK).permute(1, 2, 0)   # [H, D+R, keys]
             v = kv[:, Hh * DK:].view(keys, Hh, V).transpose(0, 1)      # [H, keys, V]

@@ -89,28 +89,34 @@ __global__ void __launch_bounds__(128) latent_decode_mma_kernel(const float* __r
   if (inv_freq)
     for (int i = tid; i < nrot / 2; i += 128) sincosf((float)pos * inv_freq[i], &cs[i].y, &cs[i].x);
   __syncthreads();
-  for (int i = tid; i < 16 * Dk; i += 128) {
-    int hh = i / Dk, d = i - hh * Dk, h = h0 + hh;
-    float v = 0.f;
-    if (h < H) {
-      if (d < L) {
-        v = qlat[((size_t)h * N + tok) * L + d];
-      } else {
-        const bf16* qr = q + (size_t)tok * q_stride + (size_t)h * (D + R) + D;
-        int r = d - L;
-        v = to_f(qr[r]);
-        if (inv_freq && r < nrot) {
-          int half = nrot / 2, p = interleaved ? r >> 1 : (r < half ? r : r - half);
-          int a = interleaved ? 2 * p : p, b = interleaved ? 2 * p + 1 : p + half;
-          float2 t = cs[p];
-          v = r == a ? v * t.x - to_f(qr[b]) * t.y : v * t.x + to_f(qr[a]) * t.y;
-        }
-      }
-      v *= scale;
-    }
+  // queries to hi + lo; the loads of a thread are independent of one another, several in flight
+  auto put = [&](int at, float v) {
     bf16 hi = __float2bfloat16_rn(v);
-    qh[hh * ld + d] = hi;
-    ql[hh * ld + d] = __float2bfloat16_rn(v - __bfloat162float(hi));
+    qh[at] = hi;
+    ql[at] = __float2bfloat16_rn(v - __bfloat162float(hi));
+  };
+  const int l4 = L >> 2;
+#pragma unroll 8
+  for (int i = tid; i < 16 * l4; i += 128) {
+    int hh = i / l4, d = (i - hh * l4) * 4, h = h0 + hh;
+    float4 v = *reinterpret_cast<const float4*>(qlat + ((size_t)min(h, H - 1) * N + tok) * L + d);
+    float sc = h < H ? scale : 0.f;
+    int at = hh * ld + d;
+    put(at, v.x * sc);
+    put(at + 1, v.y * sc);
+    put(at + 2, v.z * sc);
+    put(at + 3, v.w * sc);
+  }
+#pragma unroll 4
+  for (int i = tid; i < 16 * R; i += 128) {
+    int hh = i / R, r = i - hh * R, h = h0 + hh;
+    const bf16* qr = q + (size_t)tok * q_stride + (size_t)min(h, H - 1) * (D + R) + D;
+    const bool turn = inv_freq && r < nrot;
+    const int half = nrot / 2, p = !turn ? 0 : interleaved ? r >> 1 : (r < half ? r : r - half);
+    const int a = !turn ? r : interleaved ? 2 * p : p, b = !turn ? r : interleaved ? 2 * p + 1 : p + half;
+    float va = to_f(qr[a]), vb = to_f(qr[b]);
+    float2 t = turn ? cs[p] : make_float2(1.f, 0.f);
+    put(hh * ld + L + r, (r == a ? va * t.x - vb * t.y : vb * t.x + va * t.y) * (h < H ? scale : 0.f));
   }
   float mx[4], l[4], acc[NT][4];
 #pragma unroll
@@ -247,11 +253,11 @@ __global__ void latent_merge_kernel(const float* __restrict__ part_acc, const fl
 // Prompt attention of one sequence: query row i (position p0 + i) against the expanded keys of positions first .. first +
 // keys - 1, of which it sees those not later than itself and (window > 0) fewer than `window` positions back.
 // q rows: [H][DK] (rotated); kv rows: [H][DK] keys, then [H][V] values; out [n][H][V].
-// Block = 64 query rows of one head, 4 warps of 16 rows; key tiles of 64, two buffers, filled by asynchronous 16-byte copies
-// while the tile before is used.  Scores and softmax weights stay in registers.  Needs DK and V multiples of 16, V <= 8 NV.
+// Block = 64 query rows of one head, 4 warps of 16 rows; key tiles of PA_KEYS, two buffers, filled by asynchronous 16-byte
+// copies while the tile before is used.  Scores and softmax weights stay in registers.  SPLIT: the weights enter the second
+// product with their bf16 remainder.  Needs DK and V multiples of 16, V <= 8 NV.
 #define PA_ROWS 64
-#define PA_KEYS 64
-template <int NV>
+template <int NV, int PA_KEYS, bool SPLIT>
 __global__ void __launch_bounds__(128) prompt_attn_mma_kernel(const bf16* __restrict__ q, long long q_stride,
                                                               const bf16* __restrict__ kv, long long kv_stride,
                                                               bf16* __restrict__ out, int n, int H, int DK, int V, int keys,
@@ -299,9 +305,9 @@ __global__ void __launch_bounds__(128) prompt_attn_mma_kernel(const bf16* __rest
     if (j0 + PA_KEYS < ke) { fetch(j0 + PA_KEYS, buf ^ 1); cp_wait<1>(); }
     else cp_wait<0>();
     __syncthreads();
-    float s[8][4];
+    float s[PA_KEYS / 8][4];
 #pragma unroll
-    for (int i = 0; i < 8; ++i)
+    for (int i = 0; i < PA_KEYS / 8; ++i)
 #pragma unroll
       for (int e = 0; e < 4; ++e) s[i][e] = 0.f;
     const bf16* ap = qs + (warp * 16 + (lane & 15)) * ldk + (lane >> 4) * 8;
@@ -311,7 +317,7 @@ __global__ void __launch_bounds__(128) prompt_attn_mma_kernel(const bf16* __rest
       uint32_t a[4], b[4];
       ldm4(a, ap + kk);
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
+      for (int i = 0; i < PA_KEYS / 16; ++i) {
         ldm4(b, bp + i * 16 * ldk + kk);
         mma(s[2 * i], a, b);
         mma(s[2 * i + 1], a, b + 2);
@@ -321,7 +327,7 @@ __global__ void __launch_bounds__(128) prompt_attn_mma_kernel(const bf16* __rest
     // tiles wholly inside every row's range need no mask
     const bool edge = j0 + PA_KEYS - 1 > p0 + i0 - first || (window > 0 && p0 + i0 + PA_ROWS - 1 - first - j0 >= window) || j0 + PA_KEYS > ke;
 #pragma unroll
-    for (int i = 0; i < 8; ++i)
+    for (int i = 0; i < PA_KEYS / 8; ++i)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         float v = s[i][e] * scale_log2e;
@@ -367,8 +373,10 @@ __global__ void __launch_bounds__(128) prompt_attn_mma_kernel(const bf16* __rest
           ldm4t(b, vp + kk * 16 * ldv + i * 16);
           mma(o[2 * i], hi, b);
           mma(o[2 * i + 1], hi, b + 2);
-          mma(o[2 * i], lo, b);
-          mma(o[2 * i + 1], lo, b + 2);
+          if (SPLIT) {
+            mma(o[2 * i], lo, b);
+            mma(o[2 * i + 1], lo, b + 2);
+          }
         }
     }
     __syncthreads();
@@ -419,22 +427,26 @@ int hyb_latent_decode_mma(const float* qlat, const void* q, long long q_stride, 
 }
 
 int hyb_prompt_attn_mma(const void* q, long long q_stride, const void* kv, long long kv_stride, void* out, int n, int H, int DK,
-                        int V, int keys, int p0, int first, int window, float scale, cudaStream_t st) {
+                        int V, int keys, int p0, int first, int window, float scale, int split, int tile, cudaStream_t st) {
   if (n == 0) return 0;
   if (first < 0 || keys != p0 + n - first || (window > 0 ? first > (p0 - window + 1 > 0 ? p0 - window + 1 : 0) : first != 0)) return -2;
+  if (tile != 32 && tile != 64) return -2;
   uintptr_t bits = (uintptr_t)q | (uintptr_t)kv | (uintptr_t)out;
   if (DK % 16 || V % 16 || V > 256 || q_stride % 8 || kv_stride % 8 || (bits & 15) || (long long)H * DK % 8 || scale <= 0.f) return -3;
-  size_t smem = ((size_t)(PA_ROWS + 2 * PA_KEYS) * (DK + 8) + (size_t)2 * PA_KEYS * (V + 8)) * sizeof(bf16);
+  size_t smem = ((size_t)(PA_ROWS + 2 * tile) * (DK + 8) + (size_t)2 * tile * (V + 8)) * sizeof(bf16);
   if (smem > 200 * 1024) return -3;
   dim3 grid((n + PA_ROWS - 1) / PA_ROWS, H);
   const float sl = scale * 1.4426950408889634f;
-#define PM(NV)                                                                                                            \
+#define PM(NV, KT, SP)                                                                                                    \
   do {                                                                                                                    \
-    cudaFuncSetAttribute(prompt_attn_mma_kernel<NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);             \
-    prompt_attn_mma_kernel<NV><<<grid, 128, smem, st>>>((const bf16*)q, q_stride, (const bf16*)kv, kv_stride, (bf16*)out, n, \
-                                                        H, DK, V, keys, p0, first, window, sl);                           \
+    cudaFuncSetAttribute(prompt_attn_mma_kernel<NV, KT, SP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
+    prompt_attn_mma_kernel<NV, KT, SP><<<grid, 128, smem, st>>>((const bf16*)q, q_stride, (const bf16*)kv, kv_stride,     \
+                                                                (bf16*)out, n, H, DK, V, keys, p0, first, window, sl);    \
   } while (0)
-  if (V <= 64) PM(8); else if (V <= 128) PM(16); else PM(32);
+#define PMT(NV) do { if (tile == 32) { if (split) PM(NV, 32, true); else PM(NV, 32, false); } \
+                     else { if (split) PM(NV, 64, true); else PM(NV, 64, false); } } while (0)
+  if (V <= 64) PMT(8); else if (V <= 128) PMT(16); else PMT(32);
+#undef PMT
 #undef PM
   return (int)cudaGetLastError();
 }

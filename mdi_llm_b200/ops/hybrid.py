@@ -89,7 +89,7 @@ def lib() -> ctypes.CDLL:
     h.hyb_rotate_heads.argtypes = [vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp]
     h.hyb_latent_attn.argtypes = [vp, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, vp, vp, i32, vp, i32, i32, i32, vp]
     h.hyb_latent_decode_mma.argtypes = [vp, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, vp, vp, i32, vp, i32, i32, vp]
-    h.hyb_prompt_attn_mma.argtypes = [vp, i64, vp, i64, vp, i32, i32, i32, i32, i32, i32, i32, i32, f32, vp]
+    h.hyb_prompt_attn_mma.argtypes = [vp, i64, vp, i64, vp, i32, i32, i32, i32, i32, i32, i32, i32, f32, i32, i32, vp]
     h.hyb_row_update.argtypes = [ctypes.POINTER(_RowUpdateArgs), i32, vp]
     h.hyb_norm_conv.argtypes = [vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, i32, i32, vp]
     h.hyb_poly_norm.argtypes = [vp, i64, vp, i64, vp, i32, i32, f32, i32, vp]
@@ -479,7 +479,8 @@ def latent_attn(qlat: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, plan: 
     # and the window, so a captured step stays valid while contexts grow.
     blocks = N * ((H + 15) // 16 if mma else (H + 7) // 8)
     tiles = (window + 31) // 32 if window > 0 else 32
-    nsplit = 1 if blocks >= 2 * _SM_TARGET or split == 1 else min(32, split or max(1, min(tiles, (2 * _SM_TARGET) // blocks)))
+    want = _SM_TARGET if mma else 2 * _SM_TARGET  # the tensor-core form stages 16 queries per block: one block per SM pays
+    nsplit = 1 if blocks >= want or split == 1 else min(32, split or max(1, min(tiles, want // blocks)))
     pa = pm = None
     if nsplit > 1:
         pa = torch.empty(nsplit, H, N, L, device=q.device, dtype=torch.float32)
@@ -500,14 +501,14 @@ def latent_attn(qlat: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, plan: 
 
 
 def prompt_attn(q: torch.Tensor, kv: torch.Tensor, H: int, DK: int, V: int, p0: int, first: int, scale: float,
-                window: int = 0, out: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+                window: int = 0, out: Optional[torch.Tensor] = None, split: bool = False, tile: int = 64) -> Optional[torch.Tensor]:
     """Causal attention of one sequence's rows ``q [n, H * DK]`` (positions ``p0 ..``) over ``kv [keys, H * DK + H * V]``: the keys
     and values of positions ``first .. p0 + n - 1``, all heads side by side; ``window > 0``: the last ``window`` positions up to
-    the row's own.  Scores, softmax and weights stay on chip, weights enter the second product as a bf16 number plus its
-    bf16 remainder.  Returns (and fills) ``out [n, H, V]``; None when the kernel does not take the type, the sizes (``DK`` and
+    the row's own.  Scores, softmax and weights stay on chip; with ``split`` the weights enter the second product as a bf16
+    number plus its bf16 remainder.  ``tile``: keys per step of a block, 32 or 64.  Returns (and fills) ``out [n, H, V]``; None when the kernel does not take the type, the sizes (``DK`` and
     ``V`` multiples of 16, ``V`` at most 256) or the device."""
     n, keys = q.size(0), kv.size(0)
-    smem = 2 * (192 * (DK + 8) + 128 * (V + 8))
+    smem = 2 * ((64 + 2 * tile) * (DK + 8) + 2 * tile * (V + 8))
     if not q.is_cuda or q.dtype != torch.bfloat16 or DK % 16 or V % 16 or V > 256 or smem > 200 * 1024 \
             or any(t.stride(0) % 8 or t.data_ptr() % 16 for t in (q, kv)):
         return None
@@ -516,7 +517,7 @@ def prompt_attn(q: torch.Tensor, kv: torch.Tensor, H: int, DK: int, V: int, p0: 
     out = torch.empty(n, H, V, device=q.device, dtype=q.dtype) if out is None else out
     assert out.is_contiguous()
     _check(lib().hyb_prompt_attn_mma(q.data_ptr(), _rows(q)[0], kv.data_ptr(), _rows(kv)[0], out.data_ptr(), n, H, DK, V, keys, int(p0),
-                                     int(first), int(window), float(scale), _st()), "prompt_attn_mma")
+                                     int(first), int(window), float(scale), int(split), int(tile), _st()), "prompt_attn_mma")
     return out
 
 
