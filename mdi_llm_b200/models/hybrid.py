@@ -282,22 +282,34 @@ class LatentAttention(nn.Module, _Fused):
 
     def _expanded(self, q: torch.Tensor, cache: torch.Tensor, plan: H.BatchPlan) -> torch.Tensor:
         """Prompt form: keys and values are expanded from the cached rows once per step (one matrix product).  With 16-bit
-        activations the attention over them is one kernel per sequence (``H.prompt_attn``); else (fp32, sizes that kernel
+        activations the attention over them is one kernel for all sequences (``H.prompt_attn``); else (fp32, sizes that kernel
         does not take) scores and the weighted sum are batched matrix products over heads with the masked softmax on fp32
         scores in between, per band of query rows against the keys the band can see.  Decoding instead carries the query into the latent space
         and reads the cache directly (``H.latent_attn``): per query that costs ``kv_rank`` instead of ``dim`` multiplies per key
         and head, which only pays when there is a single query.  Returns ``[N, heads, vdim]``."""
         Hh, D, R, V, W = self.H, self.D, self.R, self.V, self.window
         DK = D + R
+        split = self.p32 and q.dtype != torch.float32  # weights as two 16-bit halves: the sum stays on the tensor cores
+        if self.fused_prompt and H.prompt_attn_takes(q, Hh, DK, V):
+            key = f"prompt_spans_{W}"  # the same for every layer of the step with this window
+            if key not in plan.shared:
+                spans, at = [], 0
+                for r0, n, slot, p0 in plan.seqs:
+                    first = max(0, p0 - W + 1) if W > 0 else 0
+                    spans.append((r0, n, at, p0, first))
+                    at += p0 + n - first
+                plan.shared[key] = (spans, torch.tensor(spans, dtype=torch.int32).to(q.device), at)
+            spans, table, keys = plan.shared[key]
+            kv = torch.empty(keys, self.w_kv.size(0), device=q.device, dtype=q.dtype)
+            for (_, n, at, p0, first), (_, _, slot, _) in zip(spans, plan.seqs):
+                torch.mm(cache[slot, first:p0 + n], self.w_kv.t(), out=kv[at:at + p0 + n - first])
+            return H.prompt_attn(q, kv, spans, Hh, DK, V, self.scale, W, split, table=table)
         out = torch.empty(q.size(0), Hh, V, device=q.device, dtype=q.dtype)
         band = min(self.query_block, max(256, (W // 2 + 127) // 128 * 128)) if W > 0 else self.query_block
-        split = self.p32 and q.dtype != torch.float32  # weights as two 16-bit halves: the sum stays on the tensor cores
         for r0, n, slot, p0 in plan.seqs:
             first = max(0, p0 - W + 1) if W > 0 else 0
             kv = H.linear(cache[slot, first:p0 + n], self.w_kv)
             keys = kv.size(0)
-            if self.fused_prompt and H.prompt_attn(q[r0:r0 + n], kv, Hh, DK, V, p0, first, self.scale, W, out[r0:r0 + n], split) is not None:
-                continue
             kt = kv[:, :Hh * DK].view(keys, Hh, DK).permute(1, 2, 0)   # [H, D+R, keys]
             v = kv[:, Hh * DK:].view(keys, Hh, V).transpose(0, 1)      # [H, keys, V]
             qh = q[r0:r0 + n].view(n, Hh, DK).transpose(0, 1)          # [H, n, D+R]

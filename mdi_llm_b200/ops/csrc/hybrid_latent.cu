@@ -250,8 +250,9 @@ __global__ void latent_merge_kernel(const float* __restrict__ part_acc, const fl
   }
 }
 
-// Prompt attention of one sequence: query row i (position p0 + i) against the expanded keys of positions first .. first +
-// keys - 1, of which it sees those not later than itself and (window > 0) fewer than `window` positions back.
+// Prompt attention of all sequences of a step.  spans[5*z] = {first query row, n, first key row, p0, first}: sequence z has
+// query rows i < n at positions p0 + i and the expanded keys of positions first .. p0 + n - 1, of which a row sees those not
+// later than itself and (window > 0) fewer than `window` positions back.
 // q rows: [H][DK] (rotated); kv rows: [H][DK] keys, then [H][V] values; out [n][H][V].
 // Block = 64 query rows of one head, 4 warps of 16 rows; key tiles of PA_KEYS, two buffers, filled by asynchronous 16-byte
 // copies while the tile before is used.  Scores and softmax weights stay in registers.  SPLIT: the weights enter the second
@@ -260,14 +261,21 @@ __global__ void latent_merge_kernel(const float* __restrict__ part_acc, const fl
 template <int NV, int PA_KEYS, bool SPLIT>
 __global__ void __launch_bounds__(128) prompt_attn_mma_kernel(const bf16* __restrict__ q, long long q_stride,
                                                               const bf16* __restrict__ kv, long long kv_stride,
-                                                              bf16* __restrict__ out, int n, int H, int DK, int V, int keys,
-                                                              int p0, int first, int window, float scale_log2e) {
+                                                              bf16* __restrict__ out, const int* __restrict__ spans, int H,
+                                                              int DK, int V, int window, float scale_log2e) {
+  const int* sp = spans + 5 * blockIdx.z;
+  const int n = sp[1], p0 = sp[3], first = sp[4], keys = p0 + n - first;
+  const int tiles = (n + PA_ROWS - 1) / PA_ROWS;
+  if ((int)blockIdx.x >= tiles) return;
+  q += (size_t)sp[0] * q_stride;
+  kv += (size_t)sp[2] * kv_stride;
+  out += (size_t)sp[0] * H * V;
   extern __shared__ __align__(16) unsigned char raw[];
   const int ldk = DK + 8, ldv = V + 8;
   bf16* qs = reinterpret_cast<bf16*>(raw);     // [64][ldk]
   bf16* ks = qs + PA_ROWS * ldk;               // [2][64][ldk]
   bf16* vs = ks + 2 * PA_KEYS * ldk;           // [2][64][ldv]
-  const int h = blockIdx.y, i0 = (gridDim.x - 1 - blockIdx.x) * PA_ROWS;  // long rows of work first
+  const int h = blockIdx.y, i0 = (tiles - 1 - (int)blockIdx.x) * PA_ROWS;  // long rows of work first
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t2 = (lane & 3) * 2;
   const int dk8 = DK >> 3, v8 = V >> 3;
   const int kb = window > 0 ? max(0, p0 + i0 - window + 1 - first) : 0;
@@ -426,22 +434,22 @@ int hyb_latent_decode_mma(const float* qlat, const void* q, long long q_stride, 
   return (int)cudaGetLastError();
 }
 
-int hyb_prompt_attn_mma(const void* q, long long q_stride, const void* kv, long long kv_stride, void* out, int n, int H, int DK,
-                        int V, int keys, int p0, int first, int window, float scale, int split, int tile, cudaStream_t st) {
-  if (n == 0) return 0;
-  if (first < 0 || keys != p0 + n - first || (window > 0 ? first > (p0 - window + 1 > 0 ? p0 - window + 1 : 0) : first != 0)) return -2;
+int hyb_prompt_attn_mma(const void* q, long long q_stride, const void* kv, long long kv_stride, void* out, const int* spans,
+                        int nseq, int longest, int H, int DK, int V, int window, float scale, int split, int tile, cudaStream_t st) {
+  if (nseq == 0 || longest == 0) return 0;
   if (tile != 32 && tile != 64) return -2;
   uintptr_t bits = (uintptr_t)q | (uintptr_t)kv | (uintptr_t)out;
   if (DK % 16 || V % 16 || V > 256 || q_stride % 8 || kv_stride % 8 || (bits & 15) || (long long)H * DK % 8 || scale <= 0.f) return -3;
   size_t smem = ((size_t)(PA_ROWS + 2 * tile) * (DK + 8) + (size_t)2 * tile * (V + 8)) * sizeof(bf16);
   if (smem > 200 * 1024) return -3;
-  dim3 grid((n + PA_ROWS - 1) / PA_ROWS, H);
+  if (nseq > 65535 || H > 65535) return -3;
+  dim3 grid((longest + PA_ROWS - 1) / PA_ROWS, H, nseq);
   const float sl = scale * 1.4426950408889634f;
 #define PM(NV, KT, SP)                                                                                                    \
   do {                                                                                                                    \
     cudaFuncSetAttribute(prompt_attn_mma_kernel<NV, KT, SP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
     prompt_attn_mma_kernel<NV, KT, SP><<<grid, 128, smem, st>>>((const bf16*)q, q_stride, (const bf16*)kv, kv_stride,     \
-                                                                (bf16*)out, n, H, DK, V, keys, p0, first, window, sl);    \
+                                                                (bf16*)out, spans, H, DK, V, window, sl);                 \
   } while (0)
 #define PMT(NV) do { if (tile == 32) { if (split) PM(NV, 32, true); else PM(NV, 32, false); } \
                      else { if (split) PM(NV, 64, true); else PM(NV, 64, false); } } while (0)

@@ -31,7 +31,7 @@ __all__ = ["BatchPlan", "HybridOpsError", "lib", "embed_rows", "cast_into", "nor
            "rotary_inv_freq", "scaled_inv_freq", "linear_f32", "grouped_linear", "window_append", "window_attn", "head_gate", "relu2_",
            "token_side_gate", "router_topk", "moe_gemv", "gather_scale_rows", "combine_rows", "act_mul", "scaled_branches",
            "full_norm_append", "lightning_recurrence", "norm_gate_rows", "gated_sum_norm_accumulate", "embed_pairs",
-           "row_update", "norm_conv", "poly_norm", "latent_prepare", "rotate_heads", "prompt_attn", "NextInput"]
+           "row_update", "norm_conv", "poly_norm", "latent_prepare", "rotate_heads", "prompt_attn", "prompt_attn_takes", "NextInput"]
 
 
 class HybridOpsError(RuntimeError):
@@ -89,7 +89,7 @@ def lib() -> ctypes.CDLL:
     h.hyb_rotate_heads.argtypes = [vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp]
     h.hyb_latent_attn.argtypes = [vp, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, vp, vp, i32, vp, i32, i32, i32, vp]
     h.hyb_latent_decode_mma.argtypes = [vp, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, vp, vp, i32, vp, i32, i32, vp]
-    h.hyb_prompt_attn_mma.argtypes = [vp, i64, vp, i64, vp, i32, i32, i32, i32, i32, i32, i32, i32, f32, i32, i32, vp]
+    h.hyb_prompt_attn_mma.argtypes = [vp, i64, vp, i64, vp, vp, i32, i32, i32, i32, i32, i32, f32, i32, i32, vp]
     h.hyb_row_update.argtypes = [ctypes.POINTER(_RowUpdateArgs), i32, vp]
     h.hyb_norm_conv.argtypes = [vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, i32, i32, vp]
     h.hyb_poly_norm.argtypes = [vp, i64, vp, i64, vp, i32, i32, f32, i32, vp]
@@ -500,24 +500,36 @@ def latent_attn(qlat: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, plan: 
     return out
 
 
-def prompt_attn(q: torch.Tensor, kv: torch.Tensor, H: int, DK: int, V: int, p0: int, first: int, scale: float,
-                window: int = 0, out: Optional[torch.Tensor] = None, split: bool = False, tile: int = 64) -> Optional[torch.Tensor]:
-    """Causal attention of one sequence's rows ``q [n, H * DK]`` (positions ``p0 ..``) over ``kv [keys, H * DK + H * V]``: the keys
-    and values of positions ``first .. p0 + n - 1``, all heads side by side; ``window > 0``: the last ``window`` positions up to
-    the row's own.  Scores, softmax and weights stay on chip; with ``split`` the weights enter the second product as a bf16
-    number plus its bf16 remainder.  ``tile``: keys per step of a block, 32 or 64.  Returns (and fills) ``out [n, H, V]``; None when the kernel does not take the type, the sizes (``DK`` and
-    ``V`` multiples of 16, ``V`` at most 256) or the device."""
-    n, keys = q.size(0), kv.size(0)
+def prompt_attn_takes(q: torch.Tensor, H: int, DK: int, V: int, tile: int = 64) -> bool:
+    """Whether :func:`prompt_attn` has a kernel for the device, type and sizes (bf16 on CUDA, ``DK`` and ``V`` multiples of 16,
+    ``V`` at most 256)."""
     smem = 2 * ((64 + 2 * tile) * (DK + 8) + 2 * tile * (V + 8))
-    if not q.is_cuda or q.dtype != torch.bfloat16 or DK % 16 or V % 16 or V > 256 or smem > 200 * 1024 \
-            or any(t.stride(0) % 8 or t.data_ptr() % 16 for t in (q, kv)):
-        return None
-    if keys != p0 + n - first or kv.size(1) != H * (DK + V) or q.size(1) != H * DK:
-        raise HybridOpsError("keys are those of positions first .. p0 + n - 1, heads side by side")
-    out = torch.empty(n, H, V, device=q.device, dtype=q.dtype) if out is None else out
-    assert out.is_contiguous()
-    _check(lib().hyb_prompt_attn_mma(q.data_ptr(), _rows(q)[0], kv.data_ptr(), _rows(kv)[0], out.data_ptr(), n, H, DK, V, keys, int(p0),
-                                     int(first), int(window), float(scale), int(split), int(tile), _st()), "prompt_attn_mma")
+    return q.is_cuda and q.dtype == torch.bfloat16 and DK % 16 == 0 and V % 16 == 0 and V <= 256 and smem <= 200 * 1024 \
+        and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
+
+
+def prompt_attn(q: torch.Tensor, kv: torch.Tensor, spans: Sequence[Tuple[int, int, int, int, int]], H: int, DK: int, V: int, scale: float,
+                window: int = 0, split: bool = False, tile: int = 64, table: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal attention of the sequences of a step, one launch.  ``spans[z] = (first row, n, first key row, p0, first)``:
+    sequence ``z`` has the rows ``q[first row :][:n]`` (``[N, H * DK]``) at positions ``p0 ..`` and, from its first key row in
+    ``kv [keys, H * DK + H * V]`` on, the keys and values of positions ``first .. p0 + n - 1``, all heads side by side;
+    ``window > 0``: a row sees the last ``window`` positions up to its own.  Scores, softmax and weights stay on chip; with ``split``
+    the weights enter the second product as a bf16 number plus its bf16 remainder.  ``tile``: keys per step of a block, 32 or
+    64.  ``table``: ``spans`` as int32 on the device when the caller has it.  Returns ``[N, H, V]``; see :func:`prompt_attn_takes`."""
+    if not prompt_attn_takes(q, H, DK, V, tile):
+        raise HybridOpsError("prompt_attn does not take these sizes or this type")
+    for r0, n, k0, p0, first in spans:
+        lo = max(0, p0 - window + 1) if window > 0 else 0
+        if n < 1 or r0 < 0 or r0 + n > q.size(0) or k0 < 0 or not 0 <= first <= lo or k0 + p0 + n - first > kv.size(0):
+            raise HybridOpsError("a span names rows outside the step or misses keys its rows can see")
+    if kv.size(1) != H * (DK + V) or q.size(1) != H * DK or kv.dtype != q.dtype or kv.stride(0) % 8 or kv.data_ptr() % 16:
+        raise HybridOpsError("queries are [N, H * DK], keys and values [keys, H * DK + H * V], rows 16-byte aligned")
+    out = torch.empty(q.size(0), H, V, device=q.device, dtype=q.dtype)
+    if table is None:
+        table = torch.tensor(spans, dtype=torch.int32).to(q.device)
+    _check(lib().hyb_prompt_attn_mma(q.data_ptr(), _rows(q)[0], kv.data_ptr(), _rows(kv)[0], out.data_ptr(), table.data_ptr(), len(spans),
+                                     max(sp[1] for sp in spans), H, DK, V, int(window), float(scale), int(split), int(tile), _st()),
+           "prompt_attn_mma")
     return out
 
 
