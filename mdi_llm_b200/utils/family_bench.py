@@ -407,7 +407,7 @@ def _ratesun_kernels(model: Any, T: int, batch: int) -> List[Dict[str, Any]]:
         if phase == "prefill":
             rec("rotate_heads", "latent_prepare", phase,
                 lambda: H.rotate_heads(q, mix.inv_freq, plan, Hh, D, R, mix.nrot, mix.pairing), 4.0 * N * Hh * R)
-            rec("latent_attn_expanded[window]", "latent_attn_expanded(gemm+softmax)", phase, lambda: mix._expanded(q, st["cache"], plan),
+            rec("latent_attn_expanded[window]", "latent_attn_expanded", phase, lambda: mix._expanded(q, st["cache"], plan),
                 2.0 * N * Hh * (D + R + V), 2.0 * T * L * Hh * (D + V) + 2.0 * Hh * keys * (D + R + V))
         else:
             qlat = torch.randn(Hh, N, L, device=dev)
@@ -537,7 +537,7 @@ def _hybrid_kernels(model: Any, T: int, batch: int) -> List[Dict[str, Any]]:
                     ms = _time(lambda: mix._expanded(q, st["cache"], plan), 5, 3, flush)
                     total_keys = sum(s + n for n, s in zip(lengths, starts))
                     flops = 2.0 * total_keys * L * Hh * (D + V) + 2.0 * Hh * keys * (D + R + V)
-                    rec("latent_attn_expanded(gemm+softmax)", phase, ms, 2.0 * N * Hh * (D + R + V), flops)
+                    rec("latent_attn_expanded", phase, ms, 2.0 * N * Hh * (D + R + V), flops)
                     s32 = torch.randn(Hh, min(N, 1024), N, device=dev)
                     ms = _time(lambda: H.causal_softmax(s32, N - s32.size(1), mix.scale, dt), 5, 3, flush)
                     rec("causal_softmax", phase, ms, s32.numel() * 6.0, 0.0)
