@@ -214,6 +214,7 @@ MIXER_KEYS = {
     "channel_delta": ("heads", "kv_heads", "dim", "vdim", "conv"),
     "attention": ("heads", "kv_heads", "dim", "vdim", "scale"),
     "lightning": ("heads", "dim", "vdim", "decay"),
+    "mamba2": ("heads", "vdim", "state", "groups", "conv", "norm_groups"),
 }
 
 # What an architecture of the family fixes beyond its config.json: the shape of a block ("sandwich": norms before and
@@ -228,7 +229,8 @@ MIXER_KEYS = {
 #              sink: True (a zero-score slot in the softmax denominator) | "learned" (its score is a tensor, one number
 #              per head); qk_norm "unit" (divide by the RMS) | "weight" (RMS norm with a learned weight per entry,
 #              shared by the heads) | "full" (RMS norm over the WHOLE projection, all heads at once, with a weight per
-#              entry, BEFORE the rotation); bias on q, k, v; gate "head" | "channel";
+#              entry, BEFORE the rotation) | "none"; rot, the pairing of the rotated entries, "pairs" (2i with 2i+1) |
+#              "halves" (i with i + dims/2); bias on q, k, v; gate "head" | "channel";
 #              p32 (the prompt form sums the values with softmax weights of more than the activation type's mantissa:
 #              fp32 weights, or with 16-bit activations their rounding and its remainder as two 16-bit operands)
 #   moe:       router "sigmoid" (independent scores) | "softmax" (over the chosen logits) | "softmax_all" (scores are
@@ -238,16 +240,20 @@ MIXER_KEYS = {
 #              up clamped by the entry's ``limit``, g sigmoid(1.702 g) (u + 1)); a ``shared`` always-on expert is read
 #              from the layer's mlp entry; shared_gate: the shared expert's output is weighed by one sigmoid per token
 #   dense_act: activation of a dense feed-forward, "gelu" (erf) | "relu2" | "polynorm" (a learned mix of the first three
-#              powers, each divided by its root mean square over the feed-forward's width)
+#              powers, each divided by its root mean square over the feed-forward's width) | "geglu" (two projections in,
+#              down (gelu_tanh(gate x) * up x))
 #   latent:    rot, the pairing of the rotated entries, "halves" (i with i + dims/2) | "pairs" (2i with 2i+1); gate (a
-#              sigmoid per output channel); p32 as for attention.  A mixer entry may name ``mask.size`` (a sliding window)
-#              and ``kv_from``
+#              sigmoid per output channel); sink (a learned score per head in the softmax denominator); p32 as for
+#              attention.  A mixer entry may name ``mask.size`` (a sliding window) and ``kv_from``
 #   depth_average: what a layer passes on is a learned mix of the embedding output and every layer's result so far
 # Per layer, an attention mixer may also name ``softcap`` (scores pass through cap * tanh(score / cap)) and
 # ``kv_from: j`` (no key/value projections: it reads the keys and values layer j cached); a mixture of experts may name
-# ``router.identity`` (that many extra router outputs whose "expert" returns its input).
-_ATTENTION_DEFAULT = {"mask": "window", "sink": False, "qk_norm": "unit", "bias": False, "gate": "head", "p32": False}
-_LATENT_DEFAULT = {"rot": "halves", "gate": True, "p32": False}
+# ``router.identity`` (that many extra router outputs whose "expert" returns its input).  A mixer's ``rot.scaling`` stretches
+# its rotary frequencies: by wavelength (keys factor, low, high, original) or by a ramp over the pair index (keys factor,
+# original, fast, slow; this one also scales the rotated entries).  A layer entry may name ``weights_of: j`` beside its
+# mixer: it has no tensors, it runs layer j's modules on a cache or state of its own.
+_ATTENTION_DEFAULT = {"mask": "window", "sink": False, "qk_norm": "unit", "rot": "pairs", "bias": False, "gate": "head", "p32": False}
+_LATENT_DEFAULT = {"rot": "halves", "gate": True, "sink": False, "p32": False}
 _MOE_DEFAULT = {"router": "sigmoid", "router_bias": False, "expert": "relu2", "shared_gate": False}
 ARCHITECTURE_TRAITS = {
     "Badapel": {"block": "sandwich", "norm": "layer", "tied_head": True},
@@ -261,6 +267,9 @@ ARCHITECTURE_TRAITS = {
                 "moe": {"router": "softmax_all", "expert": "clamped", "shared_gate": True}},
     "Ratesun": {"block": "sandwich", "norm": "layer", "tied_head": True, "dense_act": "polynorm", "depth_average": True,
                 "latent": {"rot": "pairs", "gate": False, "p32": True}},
+    "Dufelix": {"block": "sandwich", "norm": "rms", "tied_head": False, "dense_act": "geglu",
+                "attention": {"qk_norm": "none", "rot": "halves", "gate": "head", "p32": True},
+                "latent": {"rot": "pairs", "gate": False, "sink": True, "p32": True}},
 }
 FF_KINDS = ("dense", "moe")
 
@@ -342,13 +351,14 @@ class HybridConfig:
             raise ValueError("input convolutions and the average over depth are implemented for sandwich blocks")
         if self.depth_average and self.loop is not None:
             raise ValueError("the average over depth counts layers once: it does not combine with a loop")
-        if self.dense_act not in ("gelu", "relu2", "polynorm"):
+        if self.dense_act not in ("gelu", "relu2", "polynorm", "geglu"):
             raise ValueError(f"unknown dense feed-forward activation {self.dense_act!r}")
         if self.block not in ("sandwich", "prenorm", "parallel", "postnorm") or self.norm not in ("layer", "rms"):
             raise ValueError(f"unknown block {self.block!r} or norm {self.norm!r}")
         if self.positions not in ("none", "learned") or (self.positions == "learned" and self.max_positions < 1):
             raise ValueError("learned positions need max_positions >= 1")
-        if self.attention["mask"] not in ("window", "chunk") or self.attention["qk_norm"] not in ("unit", "weight", "full") \
+        if self.attention["mask"] not in ("window", "chunk") or self.attention["qk_norm"] not in ("unit", "weight", "full", "none") \
+                or self.attention["rot"] not in ("pairs", "halves") \
                 or self.attention["gate"] not in ("head", "channel") or self.attention["sink"] not in (False, True, "learned") \
                 or self.moe["router"] not in ("sigmoid", "softmax", "softmax_all") \
                 or self.moe["expert"] not in ("relu2", "gated_silu", "clamped"):
@@ -379,6 +389,18 @@ class HybridConfig:
                 if self.moe["expert"] == "clamped" and ("limit" not in mlp["expert"] or (mlp.get("shared") and "limit" not in mlp["shared"])):
                     raise ValueError(f"layer {i}: clamped experts need a limit")
             m = spec["mixer"]
+            if spec.get("weights_of") is not None:
+                j = self.weights_layer(i)
+                bare = lambda e: {k: v for k, v in e.items() if k != "weights_of"}  # noqa: E731
+                if bare(self.layers[j]) != bare(spec):
+                    raise ValueError(f"layer {i}: everything beside weights_of equals layer {j}'s entry")
+                if self.depth_average or self.token_side is not None or m.get("kv_from") is not None:
+                    raise ValueError(f"layer {i}: weights_of does not combine with tensors or caches that belong to one layer")
+            if kind == "mamba2":
+                if int(m["heads"]) % int(m["groups"]) or (int(m["heads"]) * int(m["vdim"])) % int(m["norm_groups"]):
+                    raise ValueError(f"layer {i}: groups divide the heads, norm_groups divide heads * vdim")
+                if int(m["conv"]) < 1:
+                    raise ValueError(f"layer {i}: the convolution has at least one tap")
             if kind in ("attention", "channel_delta") and int(m["heads"]) % int(m["kv_heads"]):
                 raise ValueError(f"layer {i}: heads must be a multiple of kv_heads")
             if kind == "lightning" and len(m["decay"]) != int(m["heads"]):
@@ -409,6 +431,16 @@ class HybridConfig:
     @property
     def padded_vocab_size(self) -> int:
         return self.vocab
+
+    def weights_layer(self, i: int) -> int:
+        """The layer whose tensors layer ``i`` uses: itself, or what its ``weights_of`` leads to."""
+        seen = []
+        while self.layers[i].get("weights_of") is not None:
+            seen.append(i)
+            i = int(self.layers[i]["weights_of"])
+            if not 0 <= i < len(self.layers) or i in seen:
+                raise ValueError(f"layer {seen[0]}: weights_of names a layer with tensors of its own")
+        return i
 
     def layer_runs(self) -> list:
         """Execution order as ``(layer index, starts a pass)``; a looped layer appears once per pass."""

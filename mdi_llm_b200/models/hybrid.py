@@ -16,8 +16,11 @@ Mixers (all written against the packed-batch operations of :mod:`mdi_llm_b200.op
 
 * :class:`LightningAttention` — ``S_t = decay_h S_(t-1) + k_t v_t^T`` with one fixed decay per head, SiLU on q, k, v,
   an RMS norm over all heads' read-outs together and a sigmoid gate per channel.
+* :class:`StateSpace` — ``S_t = a_t S_(t-1) + dt_t B_t x_t^T`` with one data-dependent decay per head and token, a short
+  convolution over x, B and C, and a gated RMS norm in equal parts (Mamba-2).
 
-Feed-forwards: :class:`DenseFF` and :class:`MoEFF` (sigmoid router, top-k, the score scales the expert's *input*).
+Feed-forwards: :class:`DenseFF`, :class:`GatedFF` and :class:`MoEFF` (sigmoid router, top-k, the score scales the expert's
+*input*).  A layer that names ``weights_of`` runs another layer's modules on a cache or state of its own.
 
 A layer is a *sandwich* block (``x += m norm_b(f(norm_a(x)))`` for the mixer and again for the feed-forward, optionally
 with a short convolution behind ``norm_a``, a gated per-layer token embedding and an average over depth), a
@@ -41,7 +44,7 @@ from ..ops import hybrid as H
 from .config import HybridConfig
 
 __all__ = ["HybridLM", "StatePool", "SandwichBlock", "PreNormBlock", "ParallelBlock", "PostNormBlock", "LatentAttention",
-           "GatedLinearAttention", "ChannelDelta", "WindowAttention", "LightningAttention", "DenseFF", "GatedFF", "MoEFF", "read_safetensors", "write_safetensors", "load_hybrid"]
+           "GatedLinearAttention", "ChannelDelta", "WindowAttention", "LightningAttention", "StateSpace", "DenseFF", "GatedFF", "MoEFF", "read_safetensors", "write_safetensors", "load_hybrid"]
 
 _ST_DTYPES = {"BF16": torch.bfloat16, "F32": torch.float32, "F16": torch.float16, "I32": torch.int32, "I64": torch.int64}
 
@@ -124,6 +127,11 @@ class StatePool:
             return {"cache": ((self.max_seq_length, m["kv_rank"] + m["rot_dim"]), self.dtype)}
         if spec["type"] == "attention":  # one row per position: the kv_heads keys, then the kv_heads values
             return {"cache": ((self.max_seq_length, m["kv_heads"] * (m["dim"] + m["vdim"])), self.dtype)}
+        if spec["type"] == "mamba2":
+            out = {"state": ((m["heads"], m["state"], m["vdim"]), torch.float32)}
+            if m["conv"] > 1:
+                out["conv"] = ((m["conv"] - 1, m["heads"] * m["vdim"] + 2 * m["groups"] * m["state"]), self.dtype)
+            return out
         out = {"state": ((m["heads"], m["dim"], m["vdim"]), torch.float32)}
         if spec["type"] == "channel_delta" and m["conv"] > 1:
             ch = 2 * m["kv_heads"] * m["dim"] + m["heads"] * m["vdim"]
@@ -184,9 +192,13 @@ def _param(*shape: int) -> nn.Parameter:
 class _Fused:
     """Mixin: several projections that read the same input become one weight; the originals turn into row views."""
 
-    def fuse(self, names: Sequence[str]) -> None:
+    def fuse(self, names: Sequence[str], pad: bool = False) -> None:
+        """``pad``: zero rows behind the last projection up to a multiple of 8, so that rows of the product stay 16-byte
+        aligned in the 16-bit type."""
         ws = [getattr(self, n) for n in names]
-        fused = torch.cat([w.data for w in ws], 0).contiguous()
+        rows = sum(w.size(0) for w in ws)
+        zeros = [ws[0].data.new_zeros((-rows) % 8, ws[0].size(1))] if pad else []
+        fused = torch.cat([w.data for w in ws] + zeros, 0).contiguous()
         self.w_in = fused
         self.cols: Dict[str, Tuple[int, int]] = {}
         r = 0
@@ -209,8 +221,8 @@ class _Fused:
 
 
 class LatentAttention(nn.Module, _Fused):
-    """``traits`` (see ``models/config.py``) pick the pairing of the rotated entries, the sigmoid gate per output channel and
-    whether the prompt form keeps its softmax weights beyond the activation type's mantissa.  A mixer entry may name
+    """``traits`` (see ``models/config.py``) pick the pairing of the rotated entries, the sigmoid gate per output channel, a
+    learned score per head in the softmax denominator (tensor ``sink``) and whether the prompt form keeps its softmax weights beyond the activation type's mantissa.  A mixer entry may name
     ``mask.size`` (position ``i`` sees the last ``size`` positions up to its own) and ``kv_from``: the layer then has no ``dkv``,
     it reads the latent and the rotated key part that layer cached, through its own ``uk`` and ``uv``."""
 
@@ -220,10 +232,11 @@ class LatentAttention(nn.Module, _Fused):
 
     def __init__(self, width: int, m: Dict[str, Any], eps: float, traits: Optional[Dict[str, Any]] = None) -> None:
         super().__init__()
-        t = {"rot": "halves", "gate": True, "p32": False, **(traits or {})}
+        t = {"rot": "halves", "gate": True, "sink": False, "p32": False, **(traits or {})}
         self.H, self.D, self.R, self.V = m["heads"], m["dim"], m["rot_dim"], m["vdim"]
         self.L, self.QR, self.scale, self.eps = m["kv_rank"], m["q_rank"], float(m["scale"]), eps
-        self.nrot, self.rot_base = int(m["rot"]["dims"]), float(m["rot"]["base"])
+        self.nrot, self.rot_base, self.rot_scaling = int(m["rot"]["dims"]), float(m["rot"]["base"]), m["rot"].get("scaling")
+        self.amp = H.rotary_amplitude(self.rot_scaling)
         if self.nrot > self.R or self.nrot % 2:
             raise ValueError("rot.dims must be even and at most rot_dim")
         self.window = int((m.get("mask") or {}).get("size", 0) or 0)
@@ -239,11 +252,17 @@ class LatentAttention(nn.Module, _Fused):
         if t["gate"]:
             self.g = _param(H_ * V, width)
             self.tensor_names["g"] = "g"
+        self.sink = self.sink32 = None
+        if t["sink"]:
+            self.sink = _param(H_)
+            self.tensor_names["sink"] = "sink"
         self.inv_freq: Optional[torch.Tensor] = None
 
     def finalize(self) -> None:
-        self.fuse(("dq",) + (() if self.borrows else ("dkv",)) + (() if self.g is None else ("g",)))
-        self.inv_freq = H.rotary_inv_freq(self.nrot, self.rot_base, self.dq.device)
+        self.fuse(("dq",) + (() if self.borrows else ("dkv",)) + (() if self.g is None else ("g",)), pad=True)
+        self.inv_freq = H.scaled_inv_freq(self.nrot, self.rot_base, self.rot_scaling, self.dq.device)
+        if self.sink is not None:
+            self.sink32 = self.sink.data.float().contiguous()
         # prompts expand a cached row [latent | rotated key part] into every head's whole key and value with ONE matrix
         # product: the rotated part rides along through an identity block (a product with one is exact)
         Hh, D, R, V, L = self.H, self.D, self.R, self.V, self.L
@@ -257,22 +276,22 @@ class LatentAttention(nn.Module, _Fused):
     def prompt_form(self, plan: H.BatchPlan) -> bool:
         """Whether the step runs as matrix products over expanded keys and values: it brings a prompt or a long portion, and
         no sequence that continues a long context with a few tokens."""
-        return max(n for _, n, _, _ in plan.seqs) >= self.expand_from and all(n >= self.expand_from or p0 == 0 for _, n, _, p0 in plan.seqs)
+        return H.whole_prompts(plan, self.expand_from)
 
     def forward(self, h: torch.Tensor, plan: H.BatchPlan, st: Dict[str, torch.Tensor]) -> torch.Tensor:
         N = h.size(0)
         Hh, D, R, V, L = self.H, self.D, self.R, self.V, self.L
         p = H.linear(h, self.w_in)
         cq = H.latent_prepare(self.col(p, "dq"), self.dq_norm, None if self.borrows else self.col(p, "dkv"), self.dkv_norm,
-                              self.inv_freq, st["cache"], plan, R, L, self.nrot, self.eps, self.pairing)
+                              self.inv_freq, st["cache"], plan, R, L, self.nrot, self.eps, self.pairing, self.amp)
         q = H.linear(cq, self.uq)
         if self.prompt_form(plan):
-            H.rotate_heads(q, self.inv_freq, plan, Hh, D, R, self.nrot, self.pairing)
+            H.rotate_heads(q, self.inv_freq, plan, Hh, D, R, self.nrot, self.pairing, self.amp)
             o = self._expanded(q, st["cache"], plan)
         else:
             qlat = H.matmul_f32(q.view(N, Hh, D + R)[:, :, :D].transpose(0, 1), self.uk.view(Hh, D, L))
             olat = H.latent_attn(qlat, q, st["cache"], plan, Hh, D, R, L, self.scale, window=self.window, inv_freq=self.inv_freq,
-                                 nrot=self.nrot, pairing=self.pairing)
+                                 nrot=self.nrot, pairing=self.pairing, amp=self.amp, sink=self.sink32)
             o = torch.empty(N, Hh, V, device=h.device, dtype=h.dtype)
             torch.bmm(olat, self.uv.view(Hh, V, L).transpose(1, 2), out=o.transpose(0, 1))
         o = o.view(N, Hh * V)
@@ -303,7 +322,7 @@ class LatentAttention(nn.Module, _Fused):
             kv = torch.empty(keys, self.w_kv.size(0), device=q.device, dtype=q.dtype)
             for (_, n, at, p0, first), (_, _, slot, _) in zip(spans, plan.seqs):
                 torch.mm(cache[slot, first:p0 + n], self.w_kv.t(), out=kv[at:at + p0 + n - first])
-            return H.prompt_attn(q, kv, spans, Hh, DK, V, self.scale, W, split, table=table)
+            return H.prompt_attn(q, kv, spans, Hh, DK, V, self.scale, W, split, table=table, sink=self.sink32)
         out = torch.empty(q.size(0), Hh, V, device=q.device, dtype=q.dtype)
         band = min(self.query_block, max(256, (W // 2 + 127) // 128 * 128)) if W > 0 else self.query_block
         for r0, n, slot, p0 in plan.seqs:
@@ -319,7 +338,8 @@ class LatentAttention(nn.Module, _Fused):
                 k0 = max(0, p0 + a - W + 1 - first) if W > 0 else 0
                 k0 = max(0, k0 - (k0 - k1) % 8)  # a few hidden keys in front: rows of whole 16-byte groups
                 s = H.matmul_f32(qh[:, a:b], kt[:, :, k0:k1]).contiguous()
-                pr = H.causal_softmax(s, p0 + a, self.scale, q.dtype, window=W, key0=first + k0, split=split)
+                pr = H.causal_softmax(s, p0 + a, self.scale, q.dtype, window=W, key0=first + k0, split=split,
+                                      sink=self.sink32 is not None, sink_vals=self.sink32)
                 vv = v[:, k0:k1]
                 dst = out[r0 + a:r0 + b].transpose(0, 1)
                 if split:
@@ -398,18 +418,20 @@ class WindowAttention(nn.Module, _Fused):
     ``v <- (1 - lam) v + lam v_first`` (``lam`` the layer's ``vmix`` scalar; the first such layer keeps its own), and
     caches the blend.
 
-    Further variants: ``qk_norm="full"`` norms the whole q projection (all heads at once) and the whole k projection
+    Further variants: ``qk_norm="none"`` leaves q and k as the rotation does; ``rot="halves"`` pairs entry ``i`` with
+    ``i + dims/2``; ``qk_norm="full"`` norms the whole q projection (all heads at once) and the whole k projection
     with a weight per entry BEFORE the rotation; ``sink="learned"`` gives the sink a score per head (tensor ``sink``);
     a mixer entry may name ``softcap`` (scores become ``cap tanh(score / cap)`` after the scale) and ``kv_from``: the
     layer then has no key/value projections, prepares only its queries and reads the cache of the layer it names."""
 
     expand_from = 64   # a step whose every sequence brings at least this many tokens runs as batched matrix products
+    fused_prompt = True  # False: always the batched matrix products
     query_block = 1024  # query rows per band
     score_bytes = 1 << 28  # fp32 scores alive at a time in the chunked prompt form
 
     def __init__(self, width: int, m: Dict[str, Any], eps: float, traits: Optional[Dict[str, Any]] = None) -> None:
         super().__init__()
-        t = {"mask": "window", "sink": False, "qk_norm": "unit", "bias": False, "gate": "head", "p32": False, **(traits or {})}
+        t = {"mask": "window", "sink": False, "qk_norm": "unit", "rot": "pairs", "bias": False, "gate": "head", "p32": False, **(traits or {})}
         self.H, self.G, self.D, self.V = int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"])
         self.scale, self.eps = float(m["scale"]), eps
         self.window = int((m.get("mask") or {}).get("size", 0) or 0)
@@ -417,13 +439,16 @@ class WindowAttention(nn.Module, _Fused):
         self.v_mix = bool(m.get("v_mix"))
         self.softcap = float(m.get("softcap") or 0.0)
         self.borrows = m.get("kv_from") is not None
-        self.full_norm = t["qk_norm"] == "full"
+        self.full_norm, self.head_norm, self.pairing = t["qk_norm"] == "full", t["qk_norm"] != "none", str(t["rot"])
         if self.borrows and (self.v_mix or not self.full_norm):
             raise ValueError("kv_from is implemented for the full-projection q/k norm, without value mixing")
         rot = m.get("rot") or {}
         self.nrot, self.rot_base, self.rot_scaling = int(rot.get("dims", 0)), float(rot.get("base", 10000.0)), rot.get("scaling")
+        self.amp = H.rotary_amplitude(self.rot_scaling)
         if self.nrot > self.D or self.nrot % 2:
             raise ValueError("rot.dims must be even and at most dim")
+        if self.full_norm and (self.pairing != "pairs" or self.amp != 1.0):
+            raise ValueError("the full-projection q/k norm is implemented with neighbour rotation, unscaled")
         Hh, G, D, V = self.H, self.G, self.D, self.V
         self.q = _param(Hh * D, width)
         self.g, self.o = _param(Hh if t["gate"] == "head" else Hh * V, width), _param(width, Hh * V)
@@ -457,10 +482,11 @@ class WindowAttention(nn.Module, _Fused):
         self.b_in: Optional[torch.Tensor] = None
 
     def finalize(self) -> None:
-        self.fuse(("q", "g") if self.borrows else ("q", "k", "v", "g"))
+        self.fuse(("q", "g") if self.borrows else ("q", "k", "v", "g"), pad=True)
         if self.has_bias:  # one bias vector for the fused projection; the gate has none
             kv = () if self.borrows else (self.k_b.data, self.v_b.data)
-            self.b_in = torch.cat((self.q_b.data, *kv, torch.zeros_like(self.g.data[:, 0]))).contiguous()
+            b = torch.cat((self.q_b.data, *kv))
+            self.b_in = torch.cat((b, b.new_zeros(self.w_in.size(0) - b.numel()))).contiguous()
         if self.sink_w is not None:
             self.sink32 = self.sink_w.data.float().contiguous()
         if self.v_mix:
@@ -490,11 +516,13 @@ class WindowAttention(nn.Module, _Fused):
             else:
                 lam = self.lam
         H.window_append(q, self.col(p, "k"), v, self.inv_freq, st["cache"], plan, self.H, self.G, self.D,
-                        self.V, self.nrot, self.eps, self.q_norm, self.k_norm, v_first, lam)
+                        self.V, self.nrot, self.eps, self.q_norm, self.k_norm, v_first, lam, self.head_norm, self.pairing, self.amp)
         return self._attend(q, g, st["cache"], plan)
 
     def _attend(self, q: torch.Tensor, g: torch.Tensor, cache: torch.Tensor, plan: H.BatchPlan) -> torch.Tensor:
         """Prepared queries against the cache rows of each token's slot, gated and projected."""
+        if self._takes_fused(q) and H.whole_prompts(plan, self.expand_from):
+            return H.linear(self._fused(q, g, cache, plan), self.o)
         if min(n for _, n, _, _ in plan.seqs) >= self.expand_from:
             o = self._chunked(q, cache, plan) if self.mask_kind == "chunk" and self.window > 0 else self._banded(q, cache, plan)
             o = H.head_gate(o, g) if g.size(1) == self.H else H.headmajor_gate(o, g)
@@ -502,6 +530,28 @@ class WindowAttention(nn.Module, _Fused):
             o = H.window_attn(q, g, cache, plan, self.H, self.G, self.D, self.V, self.scale, self.window,
                               mask=self.mask_kind, sink=self.sink, cap=self.softcap, sink_vals=self.sink32)
         return H.linear(o, self.o)
+
+    def _takes_fused(self, q: torch.Tensor) -> bool:
+        """Whether prompts run as one attention kernel straight on the cache rows (16-bit activations, sliding window or no
+        mask, no soft cap, no sink or a learned one)."""
+        return self.fused_prompt and (self.mask_kind == "window" or self.window == 0) and self.softcap == 0.0 \
+            and (not self.sink or self.sink32 is not None) and H.prompt_attn_takes(q, self.H, self.D, self.V)
+
+    def _fused(self, q: torch.Tensor, g: torch.Tensor, cache: torch.Tensor, plan: H.BatchPlan) -> torch.Tensor:
+        W, S = self.window, cache.size(1)
+        key = f"cache_spans_{W}_{S}"  # the same for every layer of the step with this window
+        if key not in plan.shared:
+            spans = []
+            for r0, n, slot, p0 in plan.seqs:
+                first = max(0, p0 - W + 1) if W > 0 else 0
+                spans.append((r0, n, slot * S + first, p0, first))
+            plan.shared[key] = (spans, torch.tensor(spans, dtype=torch.int32).to(q.device))
+        spans, table = plan.shared[key]
+        per_head = g.size(1) == self.H
+        o = H.prompt_attn(q, cache.view(-1, cache.size(2)), spans, self.H, self.D, self.V, self.scale, W, self.p32, table=table,
+                          kv_heads=self.G, sink=self.sink32, gate=g if per_head else None)
+        o = o.view(q.size(0), self.H * self.V)
+        return o if per_head else H.headmajor_gate(o.unsqueeze(0), g)
 
     def _band(self, out: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, slot: int, r0: int, p0: int, a: int, b: int,
               key0: int, window: int) -> None:
@@ -738,7 +788,7 @@ class _LN(nn.Module):
 
 class SandwichBlock(nn.Module):
     """``x += m norm1b(mixer(norm1(x)))``, then ``x += m norm2b(ff(norm2(x)))`` when the layer has a feed-forward, then the
-    gated per-layer token embedding when the model has one (``side``).
+    gated per-layer token embedding when the model has one (``side``).  ``norm``: layer norms (weight and bias) or RMS norms.
 
     ``taps`` > 0: what a sublayer reads is ``h + conv(h)`` with ``h`` the normed rows and ``conv`` a causal convolution over time
     per channel (tensors ``canon1`` / ``canon2 [width, taps]``), whose last inputs are part of a slot's state.  ``index`` (the
@@ -746,21 +796,22 @@ class SandwichBlock(nn.Module):
     on, ``sum_j dwa[j] depth[j]`` over the embedding output and every result up to its own, is written to the next row.
 
     Every update of the stream is one kernel that adds the normed output, keeps the rounded copy the token embedding's
-    gate reads, takes the average over depth and, on steps of one token per sequence, goes on to the norm and the
-    convolution of the next sublayer (the next block's, when ``follower`` names it)."""
+    gate reads, takes the average over depth and goes on to the norm of the next sublayer (the next block's, when the caller
+    names it as ``follower``) and, on steps of one token per sequence, its convolution."""
 
     def __init__(self, width: int, mixer: nn.Module, ff: Optional[nn.Module], eps: float, mult: float = 1.0,
-                 side: Optional["TokenSide"] = None, taps: int = 0, index: Optional[int] = None) -> None:
+                 side: Optional["TokenSide"] = None, taps: int = 0, index: Optional[int] = None, norm: str = "layer") -> None:
         super().__init__()
+        self.kind = norm
+        _Norm = _LN if norm == "layer" else _RMS
         self.mix, self.mlp, self.eps, self.mult, self.side, self.index = mixer, ff, eps, float(mult), side, index
-        self.norm1, self.norm1b = _LN(width), _LN(width)
+        self.norm1, self.norm1b = _Norm(width), _Norm(width)
         self.canon1 = _param(width, taps) if taps else None
         self.canon2 = _param(width, taps) if taps and ff is not None else None
         if ff is not None:
-            self.norm2, self.norm2b = _LN(width), _LN(width)
+            self.norm2, self.norm2b = _Norm(width), _Norm(width)
         self.dwa = _param(index + 2) if index is not None else None
         self.conv1 = self.conv2 = self.depth_w = None  # fp32 forms, made by finalize
-        self.follower: Tuple["SandwichBlock", ...] = ()  # a tuple: the next block is not a submodule of this one
 
     def norm_names(self) -> List[str]:
         return ["norm1", "norm1b"] + (["norm2", "norm2b"] if self.mlp is not None else [])
@@ -777,30 +828,35 @@ class SandwichBlock(nn.Module):
             self.depth_w = self.dwa.data.float().contiguous()
 
     def _input1(self, st: Dict[str, torch.Tensor]) -> H.NextInput:
-        return H.NextInput(self.norm1.w, self.norm1.b, self.eps, "layer", self.conv1, st.get("canon1"))
+        return H.NextInput(self.norm1.w, self.norm1.b, self.eps, self.kind, self.conv1, st.get("canon1"))
 
     def _input2(self, st: Dict[str, torch.Tensor]) -> H.NextInput:
-        return H.NextInput(self.norm2.w, self.norm2.b, self.eps, "layer", self.conv2, st.get("canon2"))
+        return H.NextInput(self.norm2.w, self.norm2.b, self.eps, self.kind, self.conv2, st.get("canon2"))
 
     def forward(self, x: torch.Tensor, plan: H.BatchPlan, st: Dict[str, torch.Tensor], dtype: torch.dtype,
                 tokens: Optional[torch.Tensor] = None, side_table: Optional[torch.Tensor] = None,
-                next_st: Optional[Dict[str, torch.Tensor]] = None) -> None:
-        """``next_st``: the state of the layer run that follows, for the input of its first sublayer."""
-        one, depth = plan.one_token, plan.shared.get("depth")
+                follower: Optional["SandwichBlock"] = None, next_st: Optional[Dict[str, torch.Tensor]] = None) -> None:
+        """``follower``, ``next_st``: the block and the state of the layer run that goes on from this one's result, for the
+        input of its first sublayer."""
+        depth = plan.shared.get("depth")
+        joins = lambda nxt: plan.one_token or nxt.conv_w is None  # noqa: E731
         h = plan.shared.pop("sublayer_input", None)  # left by the previous block's last update
         if h is None:
             h = H.norm_conv(x, self._input1(st), plan, dtype)
         y, w, b = self.mix(h, plan, st), self.norm1b.w, self.norm1b.b
         if self.mlp is not None:
             nxt = self._input2(st)
-            h = H.row_update(x, y, w, b, self.eps, "layer", self.mult, nxt=nxt if one else None, plan=plan, out_dtype=dtype)
+            h = H.row_update(x, y, w, b, self.eps, self.kind, self.mult, nxt=nxt if joins(nxt) else None, plan=plan, out_dtype=dtype)
             y, w, b = self.mlp(H.norm_conv(x, nxt, plan, dtype) if h is None else h), self.norm2b.w, self.norm2b.b
-        kind = "layer"
+        kind = self.kind
         if self.side is not None:
             xa = x if dtype == torch.float32 else torch.empty(x.shape, device=x.device, dtype=dtype)
-            H.row_update(x, y, w, b, self.eps, "layer", self.mult, copy=None if xa is x else xa)
+            H.row_update(x, y, w, b, self.eps, kind, self.mult, copy=None if xa is x else xa)
             y, w, b, kind = self.side.output(xa, tokens, side_table), self.side.norm, None, "rms"
-        nxt = self.follower[0]._input1(next_st) if one and self.follower and next_st is not None else None
+        nxt = None
+        if follower is not None:
+            nxt = follower._input1(next_st)
+            nxt = nxt if joins(nxt) else None
         h = H.row_update(x, y, w, b, self.eps, kind, self.mult, depth=depth, index=0 if self.index is None else self.index + 1,
                          depth_w=self.depth_w, nxt=nxt, plan=plan, out_dtype=dtype)
         if h is not None:
@@ -887,6 +943,39 @@ class LightningAttention(nn.Module, _Fused):
         o = H.lightning_recurrence(self.col(p, "q"), self.col(p, "k"), self.col(p, "v"), self.decay, st["state"], plan,
                                    self.H, self.D, self.V, act=True)
         return H.linear(H.norm_gate_rows(o, self.norm, self.col(p, "g"), self.eps, h.dtype), self.o)
+
+
+class StateSpace(nn.Module, _Fused):
+    """Mamba-2: one input projection ``[z | x | B | C | dt]`` (``heads*vdim | heads*vdim | groups*state | groups*state | heads``),
+    a causal convolution with bias and SiLU over x, B and C, the state-space recurrence of
+    :func:`mdi_llm_b200.ops.hybrid.ssd_recurrence` (fp32 state ``[state, vdim]`` per head and slot), the gate ``silu(z)`` BEFORE an
+    RMS norm in ``norm_groups`` equal parts, and the output projection."""
+
+    tensor_names = {"in": "in_proj", "conv": "conv", "conv.b": "conv_b", "dt_bias": "dt_bias", "A_log": "A_log", "D": "skip",
+                    "norm": "norm", "o": "o"}
+
+    def __init__(self, width: int, m: Dict[str, Any], eps: float) -> None:
+        super().__init__()
+        self.H, self.V, self.N, self.G = int(m["heads"]), int(m["vdim"]), int(m["state"]), int(m["groups"])
+        self.taps, self.parts, self.eps = int(m["conv"]), int(m["norm_groups"]), eps
+        self.inner, self.ch = self.H * self.V, self.H * self.V + 2 * self.G * self.N
+        self.in_proj = _param(self.inner + self.ch + self.H, width)
+        self.conv, self.conv_b = _param(self.ch, self.taps), _param(self.ch)
+        self.dt_bias, self.A_log, self.skip = _param(self.H), _param(self.H), _param(self.H)
+        self.norm, self.o = _param(self.inner), _param(width, self.inner)
+
+    def finalize(self) -> None:
+        self.fuse(("in_proj",), pad=True)
+        self.dt_bias32, self.A_log32, self.skip32 = (t.data.float().contiguous() for t in (self.dt_bias, self.A_log, self.skip))
+
+    def forward(self, h: torch.Tensor, plan: H.BatchPlan, st: Dict[str, torch.Tensor]) -> torch.Tensor:
+        a, b = self.inner, self.inner + self.ch
+        p = H.linear(h, self.w_in)
+        past = st["conv"] if self.taps > 1 else p.new_zeros(1, 0, self.ch)
+        xbc = H.conv_silu(p[:, a:b], self.conv, past, plan, self.conv_b)
+        y = H.ssd_recurrence(xbc, p[:, b:b + self.H], self.dt_bias32, self.A_log32, self.skip32, st["state"], plan, self.H, self.G,
+                             self.N, self.V)
+        return H.linear(H.silu_gate_norm(y, p[:, :a], self.norm, self.parts, self.eps, h.dtype), self.o)
 
 
 class PostNormBlock(nn.Module):
@@ -1021,6 +1110,9 @@ class HybridLM(nn.Module):
         self.loop_in = _param(C, 2 * C) if config.loop is not None else None
         blocks = []
         for i, spec in enumerate(config.layers):
+            if config.weights_layer(i) != i:
+                blocks.append(None)
+                continue
             m, kind = spec["mixer"], spec["type"]
             if kind == "latent_attention":
                 mixer: nn.Module = LatentAttention(C, m, eps, config.latent)
@@ -1028,6 +1120,8 @@ class HybridLM(nn.Module):
                 mixer = WindowAttention(C, m, eps, config.attention)
             elif kind == "lightning":
                 mixer = LightningAttention(C, m, eps)
+            elif kind == "mamba2":
+                mixer = StateSpace(C, m, eps)
             elif kind == "gla":
                 mixer = GatedLinearAttention(C, m, eps, ranks.get(f"l{i}.mix.a1", 16))
             else:
@@ -1041,23 +1135,23 @@ class HybridLM(nn.Module):
                            config.moe["router_bias"], config.moe["expert"], int(sh.get("ff", 0)),
                            int(mlp["router"].get("identity", 0) or 0), float(mlp["expert"].get("limit", 0.0)),
                            float(sh.get("limit", 0.0)), bool(config.moe["shared_gate"]))
+            elif config.dense_act == "geglu":
+                ff = GatedFF(C, mlp["ff"], "gelu_tanh")
             else:
                 ff = DenseFF(C, mlp["ff"], config.dense_act, eps)
             sd = int(config.token_side["dim"]) if config.token_side else 0
             side = TokenSide(C, sd, i * sd) if sd and config.block in ("sandwich", "prenorm") else None
             if config.block == "sandwich":
                 blocks.append(SandwichBlock(C, mixer, ff, eps, config.residual_mult, side, config.canon_taps,
-                                            i if config.depth_average else None))
+                                            i if config.depth_average else None, config.norm))
             elif config.block == "parallel":
                 blocks.append(ParallelBlock(C, mixer, ff, eps, config.norm, config.norm_offset, config.layer_scale))
             elif config.block == "postnorm":
                 blocks.append(PostNormBlock(C, mixer, ff, eps, config.norm))
             else:
                 blocks.append(PreNormBlock(C, mixer, ff, eps, config.norm, config.residual_mult, side))
-        self.blocks = nn.ModuleList(blocks)
-        if config.block == "sandwich" and config.loop is None:
-            for blk, nxt in zip(blocks, blocks[1:]):
-                blk.follower = (nxt,)
+        # a layer with another layer's weights IS that layer's block; its cache or state belongs to the layer run
+        self.blocks = nn.ModuleList(blocks[config.weights_layer(i)] for i in range(len(blocks)))
         self.bigram = _param(int(config.bigram["buckets"]) + 1, C) if config.bigram is not None else None
         self.final_norm = _LN(C) if config.norm == "layer" else _RMS(C)
         self.side_embed = _param(config.vocab, len(config.layers) * int(config.token_side["dim"])) if config.token_side else None
@@ -1081,6 +1175,8 @@ class HybridLM(nn.Module):
         if self.head_w is not None:
             out["head"] = self.head_w
         for i, blk in enumerate(self.blocks):
+            if self.config.weights_layer(i) != i:
+                continue
             for n in blk.norm_names():
                 out[f"l{i}.{n}"] = getattr(blk, n).w
                 if getattr(blk, n).b is not None:
@@ -1144,7 +1240,9 @@ class HybridLM(nn.Module):
         return self.finalize()
 
     def finalize(self) -> "HybridLM":
-        for blk in self.blocks:
+        for i, blk in enumerate(self.blocks):
+            if self.config.weights_layer(i) != i:
+                continue
             blk.mix.finalize()
             if isinstance(blk.mlp, (MoEFF, GatedFF, DenseFF)):
                 blk.mlp.finalize()
@@ -1201,7 +1299,9 @@ class HybridLM(nn.Module):
                 x = depth[run + 1]
             blk = self.blocks[li]
             if isinstance(blk, SandwichBlock):
-                blk(x, plan, pool.runs[run], dt, tokens, self.side_embed, pool.runs[run + 1] if run + 1 < n_runs else None)
+                goes_on = run + 1 < n_runs and not self.runs[run + 1][1]  # the next run reads this one's result as it is
+                blk(x, plan, pool.runs[run], dt, tokens, self.side_embed, self.blocks[self.runs[run + 1][0]] if goes_on else None,
+                    pool.runs[run + 1] if goes_on else None)
             else:
                 blk(x, plan, pool.runs[run], dt, tokens, self.side_embed)
             if depth is not None:

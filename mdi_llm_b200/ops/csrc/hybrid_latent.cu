@@ -5,46 +5,14 @@
 //    All heads read the same rows, so 16 heads of a token are the rows of one matrix-product tile.
 //  * prompt_attn_mma_kernel: prompts, on keys and values expanded per head, scores and weights never leave the SM.
 //
+// In both, a learned score per head (`sink`) may join the softmax denominator without a key or a value.
+//
 // Queries of the first kernel and softmax weights of both enter the products as a bf16 number plus the bf16 remainder, so
 // they keep twice the mantissa; sums are fp32.  Warp-level m16n8k16 products: the tiles are 16 and 64 rows high and a
 // step is bound by reading the cache (first kernel) or by its many small dependent tiles (second), see the bounds there.
-#include "hybrid_common.cuh"
+#include "hybrid_mma.cuh"
 
 namespace hyb {
-
-__device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-// 16 bytes to shared memory; valid == false writes zeros and reads nothing
-__device__ __forceinline__ void cp16(bf16* dst, const bf16* src, bool valid) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(valid ? 16 : 0));
-}
-__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;"); }
-template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N)); }
-__device__ __forceinline__ void ldm4(uint32_t* r, const bf16* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void ldm4t(uint32_t* r, const bf16* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void ldm2(uint32_t* r, const bf16* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void ldm2t(uint32_t* r, const bf16* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(smem_u32(p)));
-}
-// c[16 x 8] += a[16 x 16] b[16 x 8]; lane (g = lane / 4, t = lane % 4) holds c = {(g, 2t), (g, 2t+1), (g+8, 2t), (g+8, 2t+1)}
-__device__ __forceinline__ void mma(float* c, const uint32_t* a, const uint32_t* b) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
-}
-__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
-  __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-  __nv_bfloat162 l = __floats2bfloat162_rn(x - __bfloat162float(h.x), y - __bfloat162float(h.y));
-  hi = *reinterpret_cast<uint32_t*>(&h);
-  lo = *reinterpret_cast<uint32_t*>(&l);
-}
 
 // Block = one token x 16 heads x one share of its keys, 4 warps.  Tiles of 32 cached rows arrive by asynchronous 16-byte
 // copies, two buffers.  Per tile: warp w computes the scores of keys 8w .. 8w+7 for the 16 heads (queries as hi + lo),
@@ -59,7 +27,7 @@ __global__ void __launch_bounds__(128) latent_decode_mma_kernel(const float* __r
                                                                 int H, int D, int R, int L, float scale, int nsplit,
                                                                 float* __restrict__ part_acc, float* __restrict__ part_ml,
                                                                 int window, const float* __restrict__ inv_freq, int nrot,
-                                                                int interleaved) {
+                                                                int interleaved, float amp, const float* __restrict__ sink) {
   extern __shared__ __align__(16) unsigned char raw[];
   __shared__ float ss[16][LD_TILE + 1];
   __shared__ __align__(16) bf16 ph[16][LD_TILE + 8], pl[16][LD_TILE + 8];
@@ -87,7 +55,11 @@ __global__ void __launch_bounds__(128) latent_decode_mma_kernel(const float* __r
   const bool any = k_begin < k_end;
   if (any) fetch(k_begin, kt);
   if (inv_freq)
-    for (int i = tid; i < nrot / 2; i += 128) sincosf((float)pos * inv_freq[i], &cs[i].y, &cs[i].x);
+    for (int i = tid; i < nrot / 2; i += 128) {
+      float sn, co;
+      sincosf((float)pos * inv_freq[i], &sn, &co);
+      cs[i] = make_float2(co * amp, sn * amp);
+    }
   __syncthreads();
   // queries to hi + lo; the loads of a thread are independent of one another, several in flight
   auto put = [&](int at, float v) {
@@ -194,7 +166,12 @@ __global__ void __launch_bounds__(128) latent_decode_mma_kernel(const float* __r
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       int h = h0 + warp * 4 + i;
-      fin[warp * 4 + i] = nsplit == 1 ? 1.f / l[i] : 1.f;
+      float f = 1.f;
+      if (nsplit == 1) {
+        float sv = sink && h < H ? sink[h] : -INFINITY, M = fmaxf(mx[i], sv), e = expf(mx[i] - M);
+        f = e / (l[i] * e + expf(sv - M));
+      }
+      fin[warp * 4 + i] = f;
       if (nsplit > 1 && h < H) {
         size_t b = ((size_t)blockIdx.z * H + h) * N + tok;
         part_ml[b * 2] = mx[i];
@@ -220,7 +197,7 @@ __global__ void __launch_bounds__(128) latent_decode_mma_kernel(const float* __r
 // Merge of the key shares: one warp per (token, head), nsplit <= 32.  Lane z reads share z's maximum and denominator, the
 // weights e^(m_z - m) are handed round by shuffles while the lanes walk the latent four values at a time.
 __global__ void latent_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml, bf16* __restrict__ out,
-                                    int N, int H, int L, int nsplit) {
+                                    int N, int H, int L, int nsplit, const float* __restrict__ sink) {
   int tok = blockIdx.x, h = blockIdx.y, w = threadIdx.x >> 5, nw = blockDim.x >> 5, lane = threadIdx.x & 31;
   float ms = -INFINITY, ls = 0.f;
   if (lane < nsplit) {
@@ -228,9 +205,10 @@ __global__ void latent_merge_kernel(const float* __restrict__ part_acc, const fl
     ms = ml[0];
     ls = ml[1];
   }
-  float M = warp_max(ms);
+  const float sv = sink ? sink[h] : -INFINITY;
+  float M = fmaxf(warp_max(ms), sv);
   float ws = lane < nsplit ? expf(ms - M) : 0.f;  // a share without keys: exp(-inf) = 0
-  float inv = 1.f / warp_sum(ls * ws);
+  float inv = 1.f / (warp_sum(ls * ws) + expf(sv - M));
   for (int d0 = w * 128; d0 < L; d0 += nw * 128) {
     int d = d0 + 4 * lane;
     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -253,7 +231,9 @@ __global__ void latent_merge_kernel(const float* __restrict__ part_acc, const fl
 // Prompt attention of all sequences of a step.  spans[5*z] = {first query row, n, first key row, p0, first}: sequence z has
 // query rows i < n at positions p0 + i and the expanded keys of positions first .. p0 + n - 1, of which a row sees those not
 // later than itself and (window > 0) fewer than `window` positions back.
-// q rows: [H][DK] (rotated); kv rows: [H][DK] keys, then [H][V] values; out [n][H][V].
+// q rows: [H][DK] (rotated); kv rows: [G][DK] keys, then [G][V] values; out [n][H][V]; query head h reads head h / (H / G).
+// sink (optional, fp32 [H]): one more score in a row's denominator.  gate (optional, [rows][H]): a head's
+// output is multiplied by its sigmoid.
 // Block = 64 query rows of one head, 4 warps of 16 rows; key tiles of PA_KEYS, two buffers, filled by asynchronous 16-byte
 // copies while the tile before is used.  Scores and softmax weights stay in registers.  SPLIT: the weights enter the second
 // product with their bf16 remainder.  Needs DK and V multiples of 16, V <= 8 NV.
@@ -262,7 +242,9 @@ template <int NV, int PA_KEYS, bool SPLIT>
 __global__ void __launch_bounds__(128) prompt_attn_mma_kernel(const bf16* __restrict__ q, long long q_stride,
                                                               const bf16* __restrict__ kv, long long kv_stride,
                                                               bf16* __restrict__ out, const int* __restrict__ spans, int H,
-                                                              int DK, int V, int window, float scale_log2e) {
+                                                              int G, int DK, int V, int window, float scale_log2e,
+                                                              const float* __restrict__ sink, const bf16* __restrict__ gate,
+                                                              long long gate_stride) {
   const int* sp = spans + 5 * blockIdx.z;
   const int n = sp[1], p0 = sp[3], first = sp[4], keys = p0 + n - first;
   const int tiles = (n + PA_ROWS - 1) / PA_ROWS;
@@ -270,6 +252,7 @@ __global__ void __launch_bounds__(128) prompt_attn_mma_kernel(const bf16* __rest
   q += (size_t)sp[0] * q_stride;
   kv += (size_t)sp[2] * kv_stride;
   out += (size_t)sp[0] * H * V;
+  if (gate) gate += (size_t)sp[0] * gate_stride;
   extern __shared__ __align__(16) unsigned char raw[];
   const int ldk = DK + 8, ldv = V + 8;
   bf16* qs = reinterpret_cast<bf16*>(raw);     // [64][ldk]
@@ -280,8 +263,9 @@ __global__ void __launch_bounds__(128) prompt_attn_mma_kernel(const bf16* __rest
   const int dk8 = DK >> 3, v8 = V >> 3;
   const int kb = window > 0 ? max(0, p0 + i0 - window + 1 - first) : 0;
   const int ke = min(keys, p0 + min(n, i0 + PA_ROWS) - first);
-  const bf16* kbase = kv + (size_t)h * DK;
-  const bf16* vbase = kv + (size_t)H * DK + (size_t)h * V;
+  const int hk = h / (H / G);
+  const bf16* kbase = kv + (size_t)hk * DK;
+  const bf16* vbase = kv + (size_t)G * DK + (size_t)hk * V;
   auto fetch = [&](int j0, int buf) {
     for (int i = tid; i < PA_KEYS * dk8; i += 128) {
       int j = i / dk8, c = (i - j * dk8) * 8;
@@ -395,7 +379,14 @@ __global__ void __launch_bounds__(128) prompt_attn_mma_kernel(const bf16* __rest
     l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
     int row = i0 + warp * 16 + g + 8 * r;
     if (row >= n) continue;
-    float inv = 1.f / l[r];
+    float inv;
+    if (sink) {
+      float sv = sink[h] * 1.4426950408889634f, M = fmaxf(mx[r], sv), e = exp2f(mx[r] - M);
+      inv = e / (l[r] * e + exp2f(sv - M));
+    } else {
+      inv = 1.f / l[r];
+    }
+    if (gate) inv *= sigmoidf_(to_f(gate[(size_t)row * gate_stride + h]));
     bf16* dst = out + ((size_t)row * H + h) * V + t2;
 #pragma unroll
     for (int i = 0; i < NV; ++i)
@@ -413,7 +404,7 @@ extern "C" {
 int hyb_latent_decode_mma(const float* qlat, const void* q, long long q_stride, const void* cache, long long slot_stride,
                           const int* meta, const int* tok_seq, void* out, int N, int H, int D, int R, int L, float scale, int nsplit,
                           float* part_acc, float* part_ml, int window, const float* inv_freq, int nrot, int interleaved,
-                          cudaStream_t st) {
+                          float amp, const float* sink, cudaStream_t st) {
   if (N == 0) return 0;
   if (nsplit < 1 || nsplit > 32 || (nsplit > 1 && (!part_acc || !part_ml)) || nrot > R || (nrot & 1)) return -2;
   int Dk = L + R;
@@ -426,20 +417,21 @@ int hyb_latent_decode_mma(const float* qlat, const void* q, long long q_stride, 
     cudaFuncSetAttribute(latent_decode_mma_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);          \
     latent_decode_mma_kernel<NT><<<grid, 128, smem, st>>>(qlat, (const bf16*)q, q_stride, (const bf16*)cache, slot_stride, \
                                                           meta, tok_seq, (bf16*)out, N, H, D, R, L, scale, nsplit, part_acc, \
-                                                          part_ml, window, inv_freq, nrot, interleaved);                 \
+                                                          part_ml, window, inv_freq, nrot, interleaved, amp, sink);      \
   } while (0)
   if (L <= 128) LM(4); else LM(16);
 #undef LM
-  if (nsplit > 1) latent_merge_kernel<<<dim3(N, H), L > 256 ? 128 : 64, 0, st>>>(part_acc, part_ml, (bf16*)out, N, H, L, nsplit);
+  if (nsplit > 1) latent_merge_kernel<<<dim3(N, H), L > 256 ? 128 : 64, 0, st>>>(part_acc, part_ml, (bf16*)out, N, H, L, nsplit, sink);
   return (int)cudaGetLastError();
 }
 
 int hyb_prompt_attn_mma(const void* q, long long q_stride, const void* kv, long long kv_stride, void* out, const int* spans,
-                        int nseq, int longest, int H, int DK, int V, int window, float scale, int split, int tile, cudaStream_t st) {
+                        int nseq, int longest, int H, int G, int DK, int V, int window, float scale, int split, int tile,
+                        const float* sink, const void* gate, long long gate_stride, cudaStream_t st) {
   if (nseq == 0 || longest == 0) return 0;
-  if (tile != 32 && tile != 64) return -2;
+  if ((tile != 32 && tile != 64) || G < 1 || H % G) return -2;
   uintptr_t bits = (uintptr_t)q | (uintptr_t)kv | (uintptr_t)out;
-  if (DK % 16 || V % 16 || V > 256 || q_stride % 8 || kv_stride % 8 || (bits & 15) || (long long)H * DK % 8 || scale <= 0.f) return -3;
+  if (DK % 16 || V % 16 || V > 256 || q_stride % 8 || kv_stride % 8 || (bits & 15) || scale <= 0.f) return -3;
   size_t smem = ((size_t)(PA_ROWS + 2 * tile) * (DK + 8) + (size_t)2 * tile * (V + 8)) * sizeof(bf16);
   if (smem > 200 * 1024) return -3;
   if (nseq > 65535 || H > 65535) return -3;
@@ -449,7 +441,8 @@ int hyb_prompt_attn_mma(const void* q, long long q_stride, const void* kv, long 
   do {                                                                                                                    \
     cudaFuncSetAttribute(prompt_attn_mma_kernel<NV, KT, SP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
     prompt_attn_mma_kernel<NV, KT, SP><<<grid, 128, smem, st>>>((const bf16*)q, q_stride, (const bf16*)kv, kv_stride,     \
-                                                                (bf16*)out, spans, H, DK, V, window, sl);                 \
+                                                                (bf16*)out, spans, H, G, DK, V, window, sl, sink,         \
+                                                                (const bf16*)gate, gate_stride);                          \
   } while (0)
 #define PMT(NV) do { if (tile == 32) { if (split) PM(NV, 32, true); else PM(NV, 32, false); } \
                      else { if (split) PM(NV, 64, true); else PM(NV, 64, false); } } while (0)

@@ -135,7 +135,7 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const T* __restrict
                                                              const float* __restrict__ inv_freq, T* __restrict__ cache,
                                                              long long slot_stride, const int* __restrict__ meta,
                                                              const int* __restrict__ tok_seq, int R, int L, int nrot,
-                                                             int interleaved, float eps, int vec) {
+                                                             int interleaved, float eps, int vec, float amp) {
   __shared__ float red[2][8];
   int tok = blockIdx.x;
   const T* qs = dq + (size_t)tok * dq_stride;
@@ -193,6 +193,8 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const T* __restrict
     rot_pair(i, nrot, interleaved, a, b);
     float sn, cs;
     sincosf((float)pos * inv_freq[i], &sn, &cs);
+    sn *= amp;
+    cs *= amp;
     float u = to_f(src[L + a]), v = to_f(src[L + b]);
     dst[L + a] = from_f<T>(u * cs - v * sn);
     dst[L + b] = from_f<T>(v * cs + u * sn);
@@ -201,16 +203,21 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const T* __restrict
 }
 
 // The last R entries of each of the H heads (D + R wide) of every row of q are rotated in place; a thread owns both
-// members of a pair.  The angles of a token are evaluated once and shared by its heads.
+// members of a pair.  The angles of a token are evaluated once and shared by its heads; amp multiplies cosine and sine.
 template <typename T>
 __global__ void rotate_heads_kernel(T* __restrict__ q, long long q_stride, const float* __restrict__ inv_freq,
                                     const int* __restrict__ meta, const int* __restrict__ tok_seq, int H, int D, int R,
-                                    int nrot, int interleaved) {
+                                    int nrot, int interleaved, float amp) {
   extern __shared__ float cssn[];  // [nrot/2] cosines, [nrot/2] sines
   int tok = blockIdx.x, half = nrot / 2;
   const int* m = meta + 4 * tok_seq[tok];
   float pos = (float)(m[3] + tok - m[0]);
-  for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(pos * inv_freq[i], &cssn[half + i], &cssn[i]);
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float sn, cs;
+    sincosf(pos * inv_freq[i], &sn, &cs);
+    cssn[i] = cs * amp;
+    cssn[half + i] = sn * amp;
+  }
   __syncthreads();
   for (int idx = threadIdx.x; idx < H * half; idx += blockDim.x) {
     int h = idx / half, i = idx - h * half, a, b;
@@ -235,7 +242,7 @@ __global__ void latent_attn_kernel(const float* __restrict__ qlat, const T* __re
                                    const int* __restrict__ tok_seq, T* __restrict__ out, int N, int H, int D, int R,
                                    int L, float scale, int nsplit, float* __restrict__ part_acc,
                                    float* __restrict__ part_ml, int window, const float* __restrict__ inv_freq, int nrot,
-                                   int interleaved) {
+                                   int interleaved, float amp, const float* __restrict__ sink) {
   extern __shared__ float smem[];
   int Dk = L + R, ldk = Dk + 1;
   float* sq = smem;                       // [LAT_WARPS][Dk]
@@ -259,6 +266,8 @@ __global__ void latent_attn_kernel(const float* __restrict__ qlat, const T* __re
           rot_pair(i, nrot, interleaved, a, b);
           float sn, cs;
           sincosf((float)pos * inv_freq[i], &sn, &cs);
+          sn *= amp;
+          cs *= amp;
           v = r == a ? v * cs - to_f(qr[b]) * sn : v * cs + to_f(qr[a]) * sn;
         }
       }
@@ -321,11 +330,17 @@ __global__ void latent_attn_kernel(const float* __restrict__ qlat, const T* __re
     mx = mnew;
   }
   if (active && nsplit == 1) {
+    float e = 1.f;
+    if (sink) {  // the score without a value: shift to max(mx, it), add its weight to the denominator
+      float sv = sink[h], M = fmaxf(mx, sv);
+      e = expf(mx - M);
+      l = l * e + expf(sv - M);
+    }
 #pragma unroll
     for (int i = 0; i < LAT_MAXV; ++i)
       if (i < nv) {
         int d = lane + 32 * i;
-        if (d < L) out[((size_t)h * N + tok) * L + d] = from_f<T>(acc[i] / l);
+        if (d < L) out[((size_t)h * N + tok) * L + d] = from_f<T>(acc[i] * e / l);
       }
   } else if (active) {
     size_t base = ((size_t)blockIdx.z * H + h) * N + tok;
@@ -345,11 +360,11 @@ __global__ void latent_attn_kernel(const float* __restrict__ qlat, const T* __re
 // out[h, tok] = sum_z acc_z e^(m_z - m) / sum_z l_z e^(m_z - m), m = max_z m_z (an empty share has m = -inf, l = 0)
 template <typename T>
 __global__ void latent_combine_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
-                                      T* __restrict__ out, int N, int H, int L, int nsplit) {
+                                      T* __restrict__ out, int N, int H, int L, int nsplit, const float* __restrict__ sink) {
   int tok = blockIdx.x, h = blockIdx.y;
-  float m = -INFINITY;
+  float m = sink ? sink[h] : -INFINITY;
   for (int z = 0; z < nsplit; ++z) m = fmaxf(m, part_ml[(((size_t)z * H + h) * N + tok) * 2]);
-  float den = 0.f;
+  float den = sink ? expf(sink[h] - m) : 0.f;
   for (int z = 0; z < nsplit; ++z) {
     size_t b = ((size_t)z * H + h) * N + tok;
     float lz = part_ml[b * 2 + 1];
@@ -487,18 +502,19 @@ __global__ void causal_softmax_kernel(const float* __restrict__ s, T* __restrict
 // ---------------------------------------------------------------------------------------------------------
 // short causal convolution + SiLU over packed sequences, with the last taps-1 inputs kept per slot
 // ---------------------------------------------------------------------------------------------------------
-// y[t, c] = silu(sum_j w[c, j] * x[t - (taps-1-j), c]); inputs before this step come from state[slot]
+// y[t, c] = silu(b[c] + sum_j w[c, j] * x[t - (taps-1-j), c]) (b optional); inputs before this step come from state[slot]
 // ([taps-1, C], oldest first; zero for a fresh slot).
 template <typename T>
 __global__ void conv_silu_kernel(const T* __restrict__ x, long long x_stride, const T* __restrict__ w,
-                                 const T* __restrict__ state, T* __restrict__ y, long long y_stride,
-                                 const int* __restrict__ meta, const int* __restrict__ tok_seq, int C, int taps) {
+                                 const T* __restrict__ b, const T* __restrict__ state, T* __restrict__ y,
+                                 long long y_stride, const int* __restrict__ meta, const int* __restrict__ tok_seq, int C,
+                                 int taps) {
   int tok = blockIdx.x;
   const int* m = meta + 4 * tok_seq[tok];
   int local = tok - m[0];
   const T* st = state + (size_t)m[2] * (taps - 1) * C;
   for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x) {
-    float acc = 0.f;
+    float acc = b ? to_f(b[c]) : 0.f;
     for (int j = 0; j < taps; ++j) {
       int src = local - (taps - 1 - j);
       float v = src >= 0 ? to_f(x[(size_t)(m[0] + src) * x_stride + c]) : to_f(st[(size_t)(taps - 1 + src) * C + c]);
@@ -506,6 +522,72 @@ __global__ void conv_silu_kernel(const T* __restrict__ x, long long x_stride, co
     }
     y[(size_t)tok * y_stride + c] = from_f<T>(siluf_(acc));
   }
+}
+// The same for prompts in rows of whole 16-byte groups: a thread owns 8 channels of `tile` consecutive token rows, keeps
+// the taps and the last taps - 1 inputs in registers and reads every input row once (plus taps - 1 rows in front).
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128) conv_silu_rows_kernel(const T* __restrict__ x, long long x_stride,
+                                                             const T* __restrict__ w, const T* __restrict__ b,
+                                                             const T* __restrict__ state, T* __restrict__ y,
+                                                             long long y_stride, const int* __restrict__ meta,
+                                                             const int* __restrict__ tok_seq, int N, int C, int tile) {
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
+  if (c >= C) return;
+  float wt[TAPS][8], bias[8], past[TAPS][8];
+#pragma unroll
+  for (int e = 0; e < 8; ++e) {
+    bias[e] = b ? to_f(b[c + e]) : 0.f;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) wt[j][e] = to_f(w[(size_t)(c + e) * TAPS + j]);
+  }
+  const int first = blockIdx.x * tile, last = min(N, first + tile);
+  int seq = -1, start = 0;
+  for (int tok = first; tok < last; ++tok) {
+    if (tok_seq[tok] != seq) {  // a sequence begins, or the tile begins inside one: its last TAPS - 1 inputs
+      seq = tok_seq[tok];
+      const int* m = meta + 4 * seq;
+      start = m[0];
+      const T* st = state + (size_t)m[2] * (TAPS - 1) * C + c;
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) {
+        int src = tok - start - (TAPS - 1 - j);
+        load8(src >= 0 ? x + (size_t)(start + src) * x_stride + c : st + (size_t)(TAPS - 1 + src) * C, past[j]);
+      }
+    }
+    load8(x + (size_t)tok * x_stride + c, past[TAPS - 1]);
+    float o[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      float acc = bias[e];
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) acc += wt[j][e] * past[j][e];
+      o[e] = siluf_(acc);
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) past[j][e] = past[j + 1][e];
+    }
+    store8(y + (size_t)tok * y_stride + c, o);
+  }
+}
+// Steps of one token per sequence: the convolution and the shift of its stored inputs in one pass, a thread per channel.
+template <typename T>
+__global__ void conv_silu_step_kernel(const T* __restrict__ x, long long x_stride, const T* __restrict__ w,
+                                      const T* __restrict__ b, T* __restrict__ state, T* __restrict__ y, long long y_stride,
+                                      const int* __restrict__ meta, const int* __restrict__ tok_seq, int C, int taps) {
+  const int tok = blockIdx.x, c = blockIdx.y * blockDim.x + threadIdx.x;
+  if (c >= C) return;
+  T* st = state + (size_t)meta[4 * tok_seq[tok] + 2] * (taps - 1) * C + c;
+  const T cur = x[(size_t)tok * x_stride + c];
+  const T* wr = w + (size_t)c * taps;
+  float acc = b ? to_f(b[c]) : 0.f;
+#pragma unroll 4
+  for (int j = 0; j < taps - 1; ++j) {
+    T v = st[(size_t)j * C];
+    acc += to_f(wr[j]) * to_f(v);
+    if (j) st[(size_t)(j - 1) * C] = v;
+  }
+  if (taps > 1) st[(size_t)(taps - 2) * C] = cur;
+  acc += to_f(wr[taps - 1]) * to_f(cur);
+  y[(size_t)tok * y_stride + c] = from_f<T>(siluf_(acc));
 }
 // After the convolution: state[slot] <- the last taps-1 inputs of the sequence (old rows shift up when the step
 // brought fewer than taps-1 tokens).  One thread per channel walks the rows oldest first, so it never reads a row
@@ -932,7 +1014,8 @@ int hyb_softcap(const void* in, float* out, long long total, float cap, float sc
 
 int hyb_latent_prepare(const void* dq, long long dq_stride, const void* qw, void* cq, int Q, const void* ckv, long long ckv_stride,
                        const void* w, const float* inv_freq, void* cache, long long slot_stride, const int* meta,
-                       const int* tok_seq, int N, int R, int L, int nrot, int interleaved, float eps, int dt, cudaStream_t st) {
+                       const int* tok_seq, int N, int R, int L, int nrot, int interleaved, float eps, float amp, int dt,
+                       cudaStream_t st) {
   if (N == 0) return 0;
   if (nrot > R || (nrot & 1) || Q < 1) return -2;
   uintptr_t bits = (uintptr_t)dq | (uintptr_t)qw | (uintptr_t)cq | (uintptr_t)ckv | (uintptr_t)w | (uintptr_t)cache;
@@ -941,28 +1024,28 @@ int hyb_latent_prepare(const void* dq, long long dq_stride, const void* qw, void
                (latent_prepare_kernel<bf16><<<N, 256, 0, st>>>((const bf16*)dq, dq_stride, (const bf16*)qw, (bf16*)cq, Q,
                                                                (const bf16*)ckv, ckv_stride, (const bf16*)w, inv_freq,
                                                                (bf16*)cache, slot_stride, meta, tok_seq, R, L, nrot,
-                                                               interleaved, eps, vec)),
+                                                               interleaved, eps, vec, amp)),
                (latent_prepare_kernel<float><<<N, 256, 0, st>>>((const float*)dq, dq_stride, (const float*)qw, (float*)cq, Q,
                                                                 (const float*)ckv, ckv_stride, (const float*)w, inv_freq,
                                                                 (float*)cache, slot_stride, meta, tok_seq, R, L, nrot,
-                                                                interleaved, eps, vec)));
+                                                                interleaved, eps, vec, amp)));
   return (int)cudaGetLastError();
 }
 
 int hyb_rotate_heads(void* q, long long q_stride, const float* inv_freq, const int* meta, const int* tok_seq, int N, int H, int D,
-                     int R, int nrot, int interleaved, int dt, cudaStream_t st) {
+                     int R, int nrot, int interleaved, float amp, int dt, cudaStream_t st) {
   if (N == 0 || nrot == 0) return 0;
   if (nrot > R || (nrot & 1) || nrot > 8192) return -2;
   HYB_DISPATCH(dt,
-               (rotate_heads_kernel<bf16><<<N, 256, nrot * sizeof(float), st>>>((bf16*)q, q_stride, inv_freq, meta, tok_seq, H, D, R, nrot, interleaved)),
-               (rotate_heads_kernel<float><<<N, 256, nrot * sizeof(float), st>>>((float*)q, q_stride, inv_freq, meta, tok_seq, H, D, R, nrot, interleaved)));
+               (rotate_heads_kernel<bf16><<<N, 256, nrot * sizeof(float), st>>>((bf16*)q, q_stride, inv_freq, meta, tok_seq, H, D, R, nrot, interleaved, amp)),
+               (rotate_heads_kernel<float><<<N, 256, nrot * sizeof(float), st>>>((float*)q, q_stride, inv_freq, meta, tok_seq, H, D, R, nrot, interleaved, amp)));
   return (int)cudaGetLastError();
 }
 
 int hyb_latent_attn(const float* qlat, const void* q, long long q_stride, const void* cache, long long slot_stride,
                     const int* meta, const int* tok_seq, void* out, int N, int H, int D, int R, int L, float scale,
                     int nsplit, float* part_acc, float* part_ml, int window, const float* inv_freq, int nrot, int interleaved,
-                    int dt, cudaStream_t st) {
+                    float amp, const float* sink, int dt, cudaStream_t st) {
   if (N == 0) return 0;
   if (L > 1024 || nsplit < 1 || (nsplit > 1 && (!part_acc || !part_ml))) return -3;
   if (inv_freq && (nrot > R || (nrot & 1))) return -2;
@@ -975,8 +1058,8 @@ int hyb_latent_attn(const float* qlat, const void* q, long long q_stride, const 
     cudaFuncSetAttribute(latent_attn_kernel<T, MV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                \
     latent_attn_kernel<T, MV><<<grid, LAT_WARPS * 32, smem, st>>>(qlat, (const T*)q, q_stride, (const T*)cache, slot_stride, \
                                                                   meta, tok_seq, (T*)out, N, H, D, R, L, scale, nsplit,     \
-                                                                  part_acc, part_ml, window, inv_freq, nrot, interleaved);  \
-    if (nsplit > 1) latent_combine_kernel<T><<<dim3(N, H), 128, 0, st>>>(part_acc, part_ml, (T*)out, N, H, L, nsplit);      \
+                                                                  part_acc, part_ml, window, inv_freq, nrot, interleaved, amp, sink); \
+    if (nsplit > 1) latent_combine_kernel<T><<<dim3(N, H), 128, 0, st>>>(part_acc, part_ml, (T*)out, N, H, L, nsplit, sink); \
   } while (0)
 #define LAV(T) do { if (L <= 128) LA(T, 4); else if (L <= 512) LA(T, 16); else LA(T, 32); } while (0)
   if (dt == 0) LAV(bf16); else LAV(float);
@@ -1000,19 +1083,32 @@ int hyb_causal_softmax(const float* s, void* p, long long rows, int rows_per_hea
   return (int)cudaGetLastError();
 }
 
-int hyb_conv_silu(const void* x, long long x_stride, const void* w, void* state, void* y, long long y_stride,
+int hyb_conv_silu(const void* x, long long x_stride, const void* w, const void* b, void* state, void* y, long long y_stride,
                   const int* meta, const int* tok_seq, int N, int nseq, int C, int taps, int dt, cudaStream_t st) {
   if (N == 0) return 0;
+  if (taps < 1 || C < 1) return -2;
   dim3 grid(N, (C + 255) / 256), sgrid(nseq, (C + 255) / 256);
-  if (dt == 0) {
-    conv_silu_kernel<bf16><<<grid, 256, 0, st>>>((const bf16*)x, x_stride, (const bf16*)w, (const bf16*)state,
-                                                 (bf16*)y, y_stride, meta, tok_seq, C, taps);
-    if (taps > 1) conv_state_kernel<bf16><<<sgrid, 256, 0, st>>>((const bf16*)x, x_stride, (bf16*)state, meta, C, taps);
-  } else {
-    conv_silu_kernel<float><<<grid, 256, 0, st>>>((const float*)x, x_stride, (const float*)w, (const float*)state,
-                                                  (float*)y, y_stride, meta, tok_seq, C, taps);
-    if (taps > 1) conv_state_kernel<float><<<sgrid, 256, 0, st>>>((const float*)x, x_stride, (float*)state, meta, C, taps);
+  if (N == nseq) {
+    HYB_DISPATCH(dt, (conv_silu_step_kernel<bf16><<<grid, 256, 0, st>>>((const bf16*)x, x_stride, (const bf16*)w, (const bf16*)b, (bf16*)state, (bf16*)y, y_stride, meta, tok_seq, C, taps)),
+                 (conv_silu_step_kernel<float><<<grid, 256, 0, st>>>((const float*)x, x_stride, (const float*)w, (const float*)b, (float*)state, (float*)y, y_stride, meta, tok_seq, C, taps)));
+    return (int)cudaGetLastError();
   }
+  uintptr_t bits = (uintptr_t)x | (uintptr_t)y | (uintptr_t)state;
+  const bool vec = taps >= 2 && taps <= 4 && (bits & 15) == 0 && ((C | x_stride | y_stride) & 7) == 0;
+  if (vec) {
+    const int cb = (C / 8 + 127) / 128, tile = max(1, min(16, (int)((long long)N * cb / 592)));
+    dim3 vgrid((N + tile - 1) / tile, cb);
+#define CR(T, TP) conv_silu_rows_kernel<T, TP><<<vgrid, 128, 0, st>>>((const T*)x, x_stride, (const T*)w, (const T*)b, (const T*)state, (T*)y, y_stride, meta, tok_seq, N, C, tile)
+    if (dt == 0) { if (taps == 2) CR(bf16, 2); else if (taps == 3) CR(bf16, 3); else CR(bf16, 4); }
+    else { if (taps == 2) CR(float, 2); else if (taps == 3) CR(float, 3); else CR(float, 4); }
+#undef CR
+  } else {
+    HYB_DISPATCH(dt, (conv_silu_kernel<bf16><<<grid, 256, 0, st>>>((const bf16*)x, x_stride, (const bf16*)w, (const bf16*)b, (const bf16*)state, (bf16*)y, y_stride, meta, tok_seq, C, taps)),
+                 (conv_silu_kernel<float><<<grid, 256, 0, st>>>((const float*)x, x_stride, (const float*)w, (const float*)b, (const float*)state, (float*)y, y_stride, meta, tok_seq, C, taps)));
+  }
+  if (taps > 1)
+    HYB_DISPATCH(dt, (conv_state_kernel<bf16><<<sgrid, 256, 0, st>>>((const bf16*)x, x_stride, (bf16*)state, meta, C, taps)),
+                 (conv_state_kernel<float><<<sgrid, 256, 0, st>>>((const float*)x, x_stride, (float*)state, meta, C, taps)));
   return (int)cudaGetLastError();
 }
 
@@ -1114,7 +1210,8 @@ __device__ __forceinline__ float gelu_tanhf_(float z) {
 }
 
 // One block per token.  Warps walk the H query heads and then the G key heads: rotate the first `nrot` entries
-// (entry 2i with 2i+1, angle pos * inv_freq[i]), divide the head by its root mean square over D, store queries
+// (entry 2i with 2i+1, or with interleaved == 0 entry i with i + nrot/2; angle pos * inv_freq[i], cosine and sine times
+// amp), with norm != 0 divide the head by its root mean square over D, store queries
 // in place and keys into the slot's cache row; the values are copied behind the keys.  D <= 256.
 // qw / kw (optional, [D], shared by the heads) multiply the normalised query / key.  With `lam` the value written is
 // (1 - lam) * v + lam * v_first, the blend with another layer's values of the same token, evaluated in fp32.
@@ -1125,7 +1222,7 @@ __global__ void window_append_kernel(T* __restrict__ q, long long q_stride, cons
                                      T* __restrict__ cache, long long slot_stride, const int* __restrict__ meta,
                                      const int* __restrict__ tok_seq, int H, int G, int D, int V, int nrot, float eps,
                                      const T* __restrict__ qw, const T* __restrict__ kw, const T* __restrict__ v_first,
-                                     long long vf_stride, const T* __restrict__ lam) {
+                                     long long vf_stride, const T* __restrict__ lam, int norm, int interleaved, float amp) {
   int t = blockIdx.x;
   const int* m = meta + 4 * tok_seq[t];
   int pos = m[3] + (t - m[0]);
@@ -1145,16 +1242,21 @@ __global__ void window_append_kernel(T* __restrict__ q, long long q_stride, cons
       if (d < D) {
         float x = to_f(src[d]);
         if (d < nrot) {
-          float o = to_f(src[d ^ 1]), sn, cs;
-          sincosf(fpos * inv_freq[d >> 1], &sn, &cs);
-          x = (d & 1) ? x * cs + o * sn : x * cs - o * sn;
+          const int half = nrot >> 1;
+          const bool second = interleaved ? d & 1 : d >= half;
+          float o = to_f(src[interleaved ? d ^ 1 : (second ? d - half : d + half)]), sn, cs;
+          sincosf(fpos * inv_freq[interleaved ? d >> 1 : (second ? d - half : d)], &sn, &cs);
+          sn *= amp;
+          cs *= amp;
+          x = second ? x * cs + o * sn : x * cs - o * sn;
         }
         y[c] = x;
         ss += x * x;
       }
     }
-    ss = warp_sum(ss);  // also orders every lane's loads before the in-place stores below
-    float inv = 1.f / sqrtf(ss / D + eps);
+    ss = warp_sum(ss);
+    float inv = norm ? 1.f / sqrtf(ss / D + eps) : 1.f;
+    __syncwarp();  // every lane has loaded before the in-place stores
 #pragma unroll
     for (int c = 0; c < WA_MAXD; ++c) {
       int d = lane + 32 * c;
@@ -1832,7 +1934,8 @@ extern "C" {
 int hyb_window_append(void* q, long long q_stride, const void* k, long long k_stride, const void* v, long long v_stride,
                       const float* inv_freq, void* cache, long long slot_stride, const int* meta, const int* tok_seq,
                       int N, int H, int G, int D, int V, int nrot, float eps, const void* qw, const void* kw,
-                      const void* v_first, long long vf_stride, const void* lam, int dt, cudaStream_t st) {
+                      const void* v_first, long long vf_stride, const void* lam, int norm, int interleaved, float amp, int dt,
+                      cudaStream_t st) {
   if (N == 0) return 0;
   if (D > 32 * WA_MAXD || nrot > D || (nrot & 1) || (nrot > 0 && !inv_freq)) return -3;
   if (lam && !v_first) return -2;
@@ -1840,12 +1943,12 @@ int hyb_window_append(void* q, long long q_stride, const void* k, long long k_st
                (window_append_kernel<bf16><<<N, 128, 0, st>>>((bf16*)q, q_stride, (const bf16*)k, k_stride, (const bf16*)v,
                                                               v_stride, inv_freq, (bf16*)cache, slot_stride, meta, tok_seq,
                                                               H, G, D, V, nrot, eps, (const bf16*)qw, (const bf16*)kw,
-                                                              (const bf16*)v_first, vf_stride, (const bf16*)lam)),
+                                                              (const bf16*)v_first, vf_stride, (const bf16*)lam, norm, interleaved, amp)),
                (window_append_kernel<float><<<N, 128, 0, st>>>((float*)q, q_stride, (const float*)k, k_stride,
                                                                (const float*)v, v_stride, inv_freq, (float*)cache,
                                                                slot_stride, meta, tok_seq, H, G, D, V, nrot, eps,
                                                                (const float*)qw, (const float*)kw, (const float*)v_first,
-                                                               vf_stride, (const float*)lam)));
+                                                               vf_stride, (const float*)lam, norm, interleaved, amp)));
   return (int)cudaGetLastError();
 }
 

@@ -31,7 +31,8 @@ __all__ = ["BatchPlan", "HybridOpsError", "lib", "embed_rows", "cast_into", "nor
            "rotary_inv_freq", "scaled_inv_freq", "linear_f32", "grouped_linear", "window_append", "window_attn", "head_gate", "relu2_",
            "token_side_gate", "router_topk", "moe_gemv", "gather_scale_rows", "combine_rows", "act_mul", "scaled_branches",
            "full_norm_append", "lightning_recurrence", "norm_gate_rows", "gated_sum_norm_accumulate", "embed_pairs",
-           "row_update", "norm_conv", "poly_norm", "latent_prepare", "rotate_heads", "prompt_attn", "prompt_attn_takes", "NextInput"]
+           "row_update", "norm_conv", "poly_norm", "latent_prepare", "rotate_heads", "prompt_attn", "prompt_attn_takes", "NextInput",
+           "rotary_amplitude", "whole_prompts", "ssd_recurrence", "silu_gate_norm"]
 
 
 class HybridOpsError(RuntimeError):
@@ -55,6 +56,12 @@ class _RowUpdateArgs(ctypes.Structure):
                 + [(n, c_float) for n in ("eps1", "eps2", "mult")])
 
 
+class _SsdArgs(ctypes.Structure):
+    _fields_ = ([(n, c_void_p) for n in ("xbc", "dt", "dt_bias", "a_log", "d", "state", "y", "meta", "ctab", "stab", "u", "decay", "before")]
+                + [(n, c_longlong) for n in ("xbc_stride", "dt_stride")]
+                + [(n, c_int) for n in ("H", "G", "N", "V", "nseq", "nchunks")])
+
+
 def lib() -> ctypes.CDLL:
     """Load ``_mdi_hybrid.so``, compiling it first when it is missing or older than its source."""
     global _lib
@@ -72,7 +79,7 @@ def lib() -> ctypes.CDLL:
     h.hyb_cast_rows.argtypes = [vp, i64, i32, vp, i64, i32, i32, i32, vp]
     h.hyb_norm_rows.argtypes = [vp, i64, i32, vp, vp, i32, vp, i64, i32, i32, i32, f32, i32, i32, f32, f32, vp, vp]
     h.hyb_gelu_rows.argtypes = [vp, i64, i32, i32, vp]
-    h.hyb_window_append.argtypes = [vp, i64, vp, i64, vp, i64, vp, vp, i64, vp, vp, i32, i32, i32, i32, i32, i32, f32, vp, vp, vp, i64, vp, i32, vp]
+    h.hyb_window_append.argtypes = [vp, i64, vp, i64, vp, i64, vp, vp, i64, vp, vp, i32, i32, i32, i32, i32, i32, f32, vp, vp, vp, i64, vp, i32, i32, f32, i32, vp]
     h.hyb_window_attn.argtypes = [vp, i64, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, i32, vp, vp, i32, i32, i32, f32, vp, i32, vp]
     h.hyb_head_gate.argtypes = [vp, vp, i64, vp, i32, i32, i32, i32, vp]
     h.hyb_token_side_gate.argtypes = [vp, i64, vp, i64, i32, vp, vp, i32, i32, i32, vp]
@@ -85,11 +92,14 @@ def lib() -> ctypes.CDLL:
     h.hyb_scaled_branches.argtypes = [vp, i64, vp, i64, vp, vp, i64, vp, i64, vp, i32, i32, i32, vp]
     h.hyb_headmajor_gate.argtypes = [vp, vp, i64, vp, i32, i32, i32, i32, vp]
     h.hyb_softcap.argtypes = [vp, vp, i64, f32, f32, i32, vp]
-    h.hyb_latent_prepare.argtypes = [vp, i64, vp, vp, i32, vp, i64, vp, vp, vp, i64, vp, vp, i32, i32, i32, i32, i32, f32, i32, vp]
-    h.hyb_rotate_heads.argtypes = [vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp]
-    h.hyb_latent_attn.argtypes = [vp, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, vp, vp, i32, vp, i32, i32, i32, vp]
-    h.hyb_latent_decode_mma.argtypes = [vp, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, vp, vp, i32, vp, i32, i32, vp]
-    h.hyb_prompt_attn_mma.argtypes = [vp, i64, vp, i64, vp, vp, i32, i32, i32, i32, i32, i32, f32, i32, i32, vp]
+    h.hyb_latent_prepare.argtypes = [vp, i64, vp, vp, i32, vp, i64, vp, vp, vp, i64, vp, vp, i32, i32, i32, i32, i32, f32, f32, i32, vp]
+    h.hyb_rotate_heads.argtypes = [vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, i32, f32, i32, vp]
+    h.hyb_latent_attn.argtypes = [vp, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, vp, vp, i32, vp, i32, i32, f32, vp, i32, vp]
+    h.hyb_latent_decode_mma.argtypes = [vp, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, vp, vp, i32, vp, i32, i32, f32, vp, vp]
+    h.hyb_prompt_attn_mma.argtypes = [vp, i64, vp, i64, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, i32, i32, vp, vp, i64, vp]
+    h.hyb_ssd_scan.argtypes = [ctypes.POINTER(_SsdArgs), i32, vp]
+    h.hyb_ssd_chunked.argtypes = [ctypes.POINTER(_SsdArgs), i32, vp]
+    h.hyb_silu_gate_norm.argtypes = [vp, vp, i64, vp, vp, i32, i32, i32, f32, i32, vp]
     h.hyb_row_update.argtypes = [ctypes.POINTER(_RowUpdateArgs), i32, vp]
     h.hyb_norm_conv.argtypes = [vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, i32, i32, vp]
     h.hyb_poly_norm.argtypes = [vp, i64, vp, i64, vp, i32, i32, f32, i32, vp]
@@ -99,7 +109,7 @@ def lib() -> ctypes.CDLL:
     h.hyb_lightning.argtypes = [vp, i64, vp, i64, vp, i64, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp, vp, i32, vp, i32, vp]
     h.hyb_norm_gate_rows.argtypes = [vp, vp, vp, i64, vp, i32, i32, f32, i32, vp]
     h.hyb_gated_sum_norm.argtypes = [vp, i64, vp, i64, vp, i64, vp, vp, i64, i32, i32, f32, i32, vp, i32, vp]
-    h.hyb_conv_silu.argtypes = [vp, i64, vp, vp, vp, i64, vp, vp, i32, i32, i32, i32, i32, vp]
+    h.hyb_conv_silu.argtypes = [vp, i64, vp, vp, vp, vp, i64, vp, vp, i32, i32, i32, i32, i32, vp]
     h.hyb_gated_recurrence.argtypes = [ctypes.POINTER(_RecArgs), i32, i32, i32, i32, vp, vp, vp, vp]
     _lib = h
     return h
@@ -165,6 +175,12 @@ class BatchPlan:
         return [r + n - 1 for r, n, _, _ in self.seqs]
 
 
+def whole_prompts(plan: BatchPlan, least: int) -> bool:
+    """Whether a step is a matter of matrix products over many query rows: it brings a prompt or a portion of at least ``least``
+    tokens, and no sequence that continues a context with fewer."""
+    return max(n for _, n, _, _ in plan.seqs) >= least and all(n >= least or p0 == 0 for _, n, _, p0 in plan.seqs)
+
+
 def rotary_inv_freq(dims: int, base: float, device: torch.device) -> torch.Tensor:
     """``base^(-2i/dims)`` for ``i < dims/2``, evaluated in float64 and rounded once to fp32."""
     i = torch.arange(dims // 2, dtype=torch.float64)
@@ -175,12 +191,28 @@ def rotary_inv_freq(dims: int, base: float, device: torch.device) -> torch.Tenso
 # matrix products (vendor GEMM on both devices; fp32 means fp32: TF32 is switched off for the call)
 # ---------------------------------------------------------------------------------------------------------
 def scaled_inv_freq(dims: int, base: float, scaling: Optional[dict], device: torch.device) -> torch.Tensor:
-    """Rotary frequencies with the wavelength-dependent stretch used for context extension: with ``l = 2 pi / f``,
-    ``f`` is kept for ``l < original/high``, divided by ``factor`` for ``l > original/low``, and blended linearly in
-    ``s = (original/l - low) / (high - low)`` between the two.  float64, rounded once to fp32."""
+    """Rotary frequencies ``f = base^(-2i/dims)``, optionally stretched for context extension; float64, rounded once to fp32.
+
+    * ``scaling = {factor, low, high, original}``, by wavelength ``l = 2 pi / f``: ``f`` is kept for ``l < original/high``,
+      divided by ``factor`` for ``l > original/low``, and blended linearly in ``s = (original/l - low) / (high - low)``
+      between the two.
+    * ``scaling = {factor, original, fast, slow}``, by the pair's index (YaRN): the index at which a pair makes ``t`` turns
+      over ``original`` positions is ``dims ln(original / (2 pi t)) / (2 ln base)``; up to that of ``fast`` (rounded down)
+      ``f`` is kept, from that of ``slow`` (rounded up) on it is divided by ``factor``, with a linear ramp between.  The
+      rotated entries are also scaled, see :func:`rotary_amplitude`."""
     i = torch.arange(dims // 2, dtype=torch.float64)
     f = float(base) ** (-2.0 * i / dims)
-    if scaling:
+    if scaling and "fast" in scaling:
+        factor, orig = float(scaling["factor"]), float(scaling["original"])
+
+        def index(turns: float) -> float:
+            return dims * math.log(orig / (2.0 * math.pi * turns)) / (2.0 * math.log(float(base)))
+
+        lo = max(math.floor(index(float(scaling["fast"]))), 0)
+        hi = min(math.ceil(index(float(scaling["slow"]))), dims - 1)
+        ramp = torch.clamp((i - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+        f = f / factor * ramp + f * (1.0 - ramp)
+    elif scaling:
         factor, low, high = float(scaling["factor"]), float(scaling["low"]), float(scaling["high"])
         orig = float(scaling["original"])
         wl = 2.0 * math.pi / f
@@ -188,6 +220,11 @@ def scaled_inv_freq(dims: int, base: float, scaling: Optional[dict], device: tor
         mid = (1.0 - s) * f / factor + s * f
         f = torch.where(wl < orig / high, f, torch.where(wl > orig / low, f / factor, mid))
     return f.to(torch.float32).to(device)
+
+
+def rotary_amplitude(scaling: Optional[dict]) -> float:
+    """What cosine and sine are multiplied by: ``0.1 ln(factor) + 1`` with the ramp over the pair index, else 1."""
+    return 0.1 * math.log(float(scaling["factor"])) + 1.0 if scaling and "fast" in scaling else 1.0
 
 
 def linear_f32(x: torch.Tensor, w32: torch.Tensor, b32: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -380,13 +417,14 @@ def softcap(logits: torch.Tensor, cap: float, scale: float = 1.0) -> torch.Tenso
 # ---------------------------------------------------------------------------------------------------------
 # latent attention
 # ---------------------------------------------------------------------------------------------------------
-def _rotate_torch(x: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor, nrot: int, pairing: str) -> torch.Tensor:
+def _rotate_torch(x: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor, nrot: int, pairing: str,
+                  amp: float = 1.0) -> torch.Tensor:
     """``x [tokens, ..., R]``: the first ``nrot`` entries of the last axis rotated by ``pos * inv_freq``, in fp32."""
     xf = x.float().clone()
     if nrot == 0:
         return xf
     ang = positions.float()[:, None] * inv_freq[None, :]
-    c, s = torch.cos(ang), torch.sin(ang)
+    c, s = torch.cos(ang) * amp, torch.sin(ang) * amp
     while c.dim() < xf.dim():
         c, s = c.unsqueeze(1), s.unsqueeze(1)
     i, j = (slice(0, nrot, 2), slice(1, nrot, 2)) if pairing == "pairs" else (slice(0, nrot // 2), slice(nrot // 2, nrot))
@@ -398,16 +436,16 @@ def _rotate_torch(x: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tens
 
 def latent_prepare(dq: torch.Tensor, qw: torch.Tensor, ckv: Optional[torch.Tensor], w: Optional[torch.Tensor],
                    inv_freq: torch.Tensor, cache: Optional[torch.Tensor], plan: BatchPlan, R: int, L: int, nrot: int, eps: float,
-                   pairing: str = "halves") -> torch.Tensor:
+                   pairing: str = "halves", amp: float = 1.0) -> torch.Tensor:
     """Per token: the query latent ``dq`` RMS-normed with ``qw`` (returned), and, with ``ckv``, the token's cache row: the
     latent (first ``L`` of the ``ckv`` row) RMS-normed with ``w``, the shared key part (last ``R``) rotated, both written
     to ``cache[slot, pos]``.  ``ckv is None``: a layer that reads another layer's cache.  The rotation pairs entry ``i``
     with ``i + nrot/2`` (``pairing="halves"``) or ``2i`` with ``2i+1`` (``"pairs"``) of the first ``nrot`` entries, angle
-    ``pos * inv_freq[i]``."""
+    ``pos * inv_freq[i]``, cosine and sine times ``amp``."""
     if not dq.is_cuda:
         if ckv is not None:
             lat = _norm_torch(ckv[:, :L], w, None, eps, "rms").to(cache.dtype)
-            kr = _rotate_torch(ckv[:, L:], plan.positions, inv_freq, nrot, pairing).to(cache.dtype)
+            kr = _rotate_torch(ckv[:, L:], plan.positions, inv_freq, nrot, pairing, amp).to(cache.dtype)
             for r0, n, slot, p0 in plan.seqs:
                 cache[slot, p0:p0 + n, :L] = lat[r0:r0 + n]
                 cache[slot, p0:p0 + n, L:] = kr[r0:r0 + n]
@@ -421,21 +459,21 @@ def latent_prepare(dq: torch.Tensor, qw: torch.Tensor, ckv: Optional[torch.Tenso
     _check(lib().hyb_latent_prepare(dq.data_ptr(), ds, qw.data_ptr(), cq.data_ptr(), Q, None if none else ckv.data_ptr(),
                                     0 if none else _rows(ckv)[0], None if none else w.data_ptr(), inv_freq.data_ptr(),
                                     None if none else cache.data_ptr(), 0 if none else cache.stride(0), plan.meta.data_ptr(),
-                                    plan.tok_seq.data_ptr(), dq.size(0), R, L, nrot, int(pairing == "pairs"), float(eps), _dt(dq),
+                                    plan.tok_seq.data_ptr(), dq.size(0), R, L, nrot, int(pairing == "pairs"), float(eps), float(amp), _dt(dq),
                                     _st()), "latent_prepare")
     return cq
 
 
 def rotate_heads(q: torch.Tensor, inv_freq: torch.Tensor, plan: BatchPlan, H: int, D: int, R: int, nrot: int,
-                 pairing: str = "halves") -> torch.Tensor:
+                 pairing: str = "halves", amp: float = 1.0) -> torch.Tensor:
     """The last ``R`` values of each of the ``H`` heads of ``q [N, H * (D + R)]`` rotated in place (as in
     :func:`latent_prepare`)."""
     if not q.is_cuda:
         qv = q.view(q.size(0), H, D + R)
-        qv[..., D:] = _rotate_torch(qv[..., D:], plan.positions, inv_freq, nrot, pairing).to(q.dtype)
+        qv[..., D:] = _rotate_torch(qv[..., D:], plan.positions, inv_freq, nrot, pairing, amp).to(q.dtype)
         return q
     _check(lib().hyb_rotate_heads(q.data_ptr(), _rows(q)[0], inv_freq.data_ptr(), plan.meta.data_ptr(), plan.tok_seq.data_ptr(),
-                                  q.size(0), H, D, R, nrot, int(pairing == "pairs"), _dt(q), _st()), "rotate_heads")
+                                  q.size(0), H, D, R, nrot, int(pairing == "pairs"), float(amp), _dt(q), _st()), "rotate_heads")
     return q
 
 
@@ -444,11 +482,12 @@ _SM_TARGET = 148  # one block per SM of a B200
 
 def latent_attn(qlat: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, plan: BatchPlan, H: int, D: int, R: int, L: int,
                 scale: float, split: int = 0, window: int = 0, inv_freq: Optional[torch.Tensor] = None, nrot: int = 0,
-                pairing: str = "halves") -> torch.Tensor:
+                pairing: str = "halves", amp: float = 1.0, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal softmax attention of ``H`` heads over the cached rows ``[L latent | R rotated key]`` of each token's slot
     (``window > 0``: the last ``window`` positions up to the token's own).  The query of head ``h`` is
     ``[qlat[h, tok] | q[tok, h, D:]]``, the value of a row is its latent part.  ``qlat`` is used in fp32.  With
-    ``inv_freq`` the second part of the query is not rotated yet: that happens as it is loaded (fp32, unrounded).
+    ``inv_freq`` the second part of the query is not rotated yet: that happens as it is loaded (fp32, unrounded; cosine and
+    sine times ``amp``).  ``sink`` (fp32 ``[H]``): one more score per head in the denominator, without a key or a value.
     Returns the attended latents ``[H, N, L]``.  ``split`` (CUDA, at most 32): key shares per query, 0 = chosen from the
     batch shape and the window.  With bf16 activations, ``L`` a multiple of 32 (at most 512) and ``L + R`` of 16 the products
     run on the tensor cores, queries and weights as a bf16 number plus its bf16 remainder; else on fp32 values."""
@@ -457,7 +496,7 @@ def latent_attn(qlat: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, plan: 
         out = torch.empty(H, N, L, dtype=q.dtype)
         qr = q.view(N, H, D + R)[..., D:].float()
         if inv_freq is not None:
-            qr = _rotate_torch(qr, plan.positions, inv_freq, nrot, pairing)
+            qr = _rotate_torch(qr, plan.positions, inv_freq, nrot, pairing, amp)
         qq = torch.cat((qlat.float(), qr.permute(1, 0, 2)), -1) * scale  # [H, N, L+R]
         for r0, n, slot, p0 in plan.seqs:
             rows = cache[slot, :p0 + n].float()
@@ -466,9 +505,15 @@ def latent_attn(qlat: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, plan: 
             hidden = keys > pos
             if window > 0:
                 hidden = hidden | (pos - keys >= window)
-            out[:, r0:r0 + n] = (torch.softmax(s.masked_fill(hidden, float("-inf")), -1) @ rows[:, :L]).to(q.dtype)
+            s = s.masked_fill(hidden, float("-inf"))
+            if sink is not None:
+                s = torch.cat((s, sink.float()[:, None, None].expand(H, n, 1)), -1)
+            out[:, r0:r0 + n] = (torch.softmax(s, -1)[..., :p0 + n] @ rows[:, :L]).to(q.dtype)
         return out
     assert qlat.is_contiguous()
+    if sink is not None and (sink.dtype != torch.float32 or sink.numel() != H or not sink.is_contiguous()):
+        raise HybridOpsError("sink scores are dense fp32, one per head")
+    sk = None if sink is None else sink.data_ptr()
     qlat = qlat.float()
     qs, _ = _rows(q)
     out = torch.empty(H, N, L, device=q.device, dtype=q.dtype)
@@ -489,14 +534,14 @@ def latent_attn(qlat: torch.Tensor, q: torch.Tensor, cache: torch.Tensor, plan: 
         _check(lib().hyb_latent_decode_mma(qlat.data_ptr(), q.data_ptr(), qs, cache.data_ptr(), cache.stride(0), plan.meta.data_ptr(),
                                            plan.tok_seq.data_ptr(), out.data_ptr(), N, H, D, R, L, float(scale), nsplit,
                                            None if pa is None else pa.data_ptr(), None if pm is None else pm.data_ptr(), int(window),
-                                           None if inv_freq is None else inv_freq.data_ptr(), int(nrot), int(pairing == "pairs"), _st()),
-               "latent_decode_mma")
+                                           None if inv_freq is None else inv_freq.data_ptr(), int(nrot), int(pairing == "pairs"), float(amp), sk,
+                                           _st()), "latent_decode_mma")
         return out
     _check(lib().hyb_latent_attn(qlat.data_ptr(), q.data_ptr(), qs, cache.data_ptr(), cache.stride(0), plan.meta.data_ptr(),
                                  plan.tok_seq.data_ptr(), out.data_ptr(), N, H, D, R, L, float(scale), nsplit,
                                  None if pa is None else pa.data_ptr(), None if pm is None else pm.data_ptr(), int(window),
-                                 None if inv_freq is None else inv_freq.data_ptr(), int(nrot), int(pairing == "pairs"), _dt(q),
-                                 _st()), "latent_attn")
+                                 None if inv_freq is None else inv_freq.data_ptr(), int(nrot), int(pairing == "pairs"), float(amp), sk,
+                                 _dt(q), _st()), "latent_attn")
     return out
 
 
@@ -509,26 +554,37 @@ def prompt_attn_takes(q: torch.Tensor, H: int, DK: int, V: int, tile: int = 64) 
 
 
 def prompt_attn(q: torch.Tensor, kv: torch.Tensor, spans: Sequence[Tuple[int, int, int, int, int]], H: int, DK: int, V: int, scale: float,
-                window: int = 0, split: bool = False, tile: int = 64, table: Optional[torch.Tensor] = None) -> torch.Tensor:
+                window: int = 0, split: bool = False, tile: int = 64, table: Optional[torch.Tensor] = None, kv_heads: int = 0,
+                sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of the sequences of a step, one launch.  ``spans[z] = (first row, n, first key row, p0, first)``:
     sequence ``z`` has the rows ``q[first row :][:n]`` (``[N, H * DK]``) at positions ``p0 ..`` and, from its first key row in
     ``kv [keys, H * DK + H * V]`` on, the keys and values of positions ``first .. p0 + n - 1``, all heads side by side;
     ``window > 0``: a row sees the last ``window`` positions up to its own.  Scores, softmax and weights stay on chip; with ``split``
     the weights enter the second product as a bf16 number plus its bf16 remainder.  ``tile``: keys per step of a block, 32 or
-    64.  ``table``: ``spans`` as int32 on the device when the caller has it.  Returns ``[N, H, V]``; see :func:`prompt_attn_takes`."""
+    64.  ``table``: ``spans`` as int32 on the device when the caller has it.  ``kv_heads = G`` (0: ``H``): rows of ``kv`` are
+    ``[G * DK | G * V]`` and query head ``h`` reads head ``h // (H / G)``.  ``sink`` (fp32 ``[H]``): one more score per head in the
+    denominator.  ``gate [N, H]``: a head's output is multiplied by its sigmoid.  Returns ``[N, H, V]``; see
+    :func:`prompt_attn_takes`."""
+    G = int(kv_heads) or H
     if not prompt_attn_takes(q, H, DK, V, tile):
         raise HybridOpsError("prompt_attn does not take these sizes or this type")
     for r0, n, k0, p0, first in spans:
         lo = max(0, p0 - window + 1) if window > 0 else 0
         if n < 1 or r0 < 0 or r0 + n > q.size(0) or k0 < 0 or not 0 <= first <= lo or k0 + p0 + n - first > kv.size(0):
             raise HybridOpsError("a span names rows outside the step or misses keys its rows can see")
-    if kv.size(1) != H * (DK + V) or q.size(1) != H * DK or kv.dtype != q.dtype or kv.stride(0) % 8 or kv.data_ptr() % 16:
-        raise HybridOpsError("queries are [N, H * DK], keys and values [keys, H * DK + H * V], rows 16-byte aligned")
+    if H % G or kv.size(1) != G * (DK + V) or q.size(1) != H * DK or kv.dtype != q.dtype or kv.stride(0) % 8 or kv.data_ptr() % 16:
+        raise HybridOpsError("queries are [N, H * DK], keys and values [keys, G * DK + G * V], rows 16-byte aligned")
+    if sink is not None and (sink.dtype != torch.float32 or sink.numel() != H or not sink.is_contiguous()):
+        raise HybridOpsError("sink scores are dense fp32, one per head")
+    if gate is not None and (gate.dtype != q.dtype or gate.size(1) != H):
+        raise HybridOpsError("the gate has one column per head, in the activation type")
     out = torch.empty(q.size(0), H, V, device=q.device, dtype=q.dtype)
     if table is None:
         table = torch.tensor(spans, dtype=torch.int32).to(q.device)
     _check(lib().hyb_prompt_attn_mma(q.data_ptr(), _rows(q)[0], kv.data_ptr(), _rows(kv)[0], out.data_ptr(), table.data_ptr(), len(spans),
-                                     max(sp[1] for sp in spans), H, DK, V, int(window), float(scale), int(split), int(tile), _st()),
+                                     max(sp[1] for sp in spans), H, G, DK, V, int(window), float(scale), int(split), int(tile),
+                                     None if sink is None else sink.data_ptr(), None if gate is None else gate.data_ptr(),
+                                     0 if gate is None else _rows(gate)[0], _st()),
            "prompt_attn_mma")
     return out
 
@@ -585,9 +641,11 @@ def causal_softmax(scores: torch.Tensor, first_pos: int, scale: float, out_dtype
 def window_append(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, inv_freq: Optional[torch.Tensor], cache: torch.Tensor,
                   plan: BatchPlan, H: int, G: int, D: int, V: int, nrot: int, eps: float,
                   qw: Optional[torch.Tensor] = None, kw: Optional[torch.Tensor] = None,
-                  v_first: Optional[torch.Tensor] = None, lam: Optional[torch.Tensor] = None) -> None:
-    """Per token: rotate the first ``nrot`` entries of every query and key head (entry ``2i`` paired with ``2i+1``,
-    angle ``pos * inv_freq[i]``), divide each head by its root mean square over ``D`` (``eps`` inside the root), keep
+                  v_first: Optional[torch.Tensor] = None, lam: Optional[torch.Tensor] = None, norm: bool = True,
+                  pairing: str = "pairs", amp: float = 1.0) -> None:
+    """Per token: rotate the first ``nrot`` entries of every query and key head (entry ``2i`` paired with ``2i+1``, or with
+    ``pairing="halves"`` entry ``i`` with ``i + nrot/2``; angle ``pos * inv_freq[i]``, cosine and sine times ``amp``), divide
+    each head by its root mean square over ``D`` (``eps`` inside the root; not with ``norm=False``), keep
     the queries in place and write ``[keys | values]`` to ``cache[slot, pos]`` (row = ``G*D`` keys then ``G*V`` values).
     ``qw`` / ``kw`` (``[D]``, shared by the heads) multiply the normalised queries / keys.  With ``lam`` (a one-element
     tensor) the values written are ``(1 - lam) v + lam v_first``, evaluated in fp32 (``v_first [N, G*V]``: the values
@@ -596,14 +654,9 @@ def window_append(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, inv_freq: O
         N = q.size(0)
 
         def prep(x: torch.Tensor, heads: int, w: Optional[torch.Tensor]) -> torch.Tensor:
-            xf = x.float().reshape(N, heads, D).clone()
-            if nrot:
-                ang = plan.positions.float()[:, None] * inv_freq[None, :]
-                c, s_ = torch.cos(ang)[:, None, :], torch.sin(ang)[:, None, :]
-                u, w_ = xf[..., 0:nrot:2].clone(), xf[..., 1:nrot:2].clone()
-                xf[..., 0:nrot:2] = u * c - w_ * s_
-                xf[..., 1:nrot:2] = w_ * c + u * s_
-            xf = xf / torch.sqrt((xf * xf).mean(-1, keepdim=True) + eps)
+            xf = _rotate_torch(x.reshape(N, heads, D), plan.positions, inv_freq, nrot, pairing, amp)
+            if norm:
+                xf = xf / torch.sqrt((xf * xf).mean(-1, keepdim=True) + eps)
             if w is not None:
                 xf = xf * w.float()
             return xf.reshape(N, heads * D).to(x.dtype)
@@ -623,7 +676,8 @@ def window_append(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, inv_freq: O
                                    plan.meta.data_ptr(), plan.tok_seq.data_ptr(), q.size(0), H, G, D, V, int(nrot),
                                    float(eps), None if qw is None else qw.data_ptr(), None if kw is None else kw.data_ptr(),
                                    None if lam is None else v_first.data_ptr(), 0 if lam is None else _rows(v_first)[0],
-                                   None if lam is None else lam.data_ptr(), _dt(q), _st()), "window_append")
+                                   None if lam is None else lam.data_ptr(), int(bool(norm)), int(pairing == "pairs"), float(amp),
+                                   _dt(q), _st()), "window_append")
 
 
 _MASK_KINDS = {"window": 0, "chunk": 1}
@@ -881,15 +935,15 @@ def matmul_f32(a: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
 # ---------------------------------------------------------------------------------------------------------
 # short convolution and the gated recurrences
 # ---------------------------------------------------------------------------------------------------------
-def conv_silu(x: torch.Tensor, w: torch.Tensor, state: torch.Tensor, plan: BatchPlan) -> torch.Tensor:
-    """Causal per-channel convolution over time (``w [C, taps]``, last column = current token) then SiLU.
+def conv_silu(x: torch.Tensor, w: torch.Tensor, state: torch.Tensor, plan: BatchPlan, b: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal per-channel convolution over time (``w [C, taps]``, last column = current token; bias ``b [C]``) then SiLU.
     ``state [slots, taps-1, C]`` supplies the inputs before this step and is updated to the step's last ones."""
     C, taps = w.shape
     if not x.is_cuda:
         y = torch.empty(x.size(0), C, dtype=x.dtype)
         for r0, n, slot, _ in plan.seqs:
             full = torch.cat((state[slot], x[r0:r0 + n]), 0).float()  # [taps-1+n, C]
-            acc = torch.zeros(n, C)
+            acc = torch.zeros(n, C) if b is None else b.float().repeat(n, 1)
             for j in range(taps):
                 acc += full[j:j + n] * w[:, j].float()
             y[r0:r0 + n] = F.silu(acc).to(x.dtype)
@@ -898,7 +952,9 @@ def conv_silu(x: torch.Tensor, w: torch.Tensor, state: torch.Tensor, plan: Batch
         return y
     xs, _ = _rows(x)
     y = torch.empty(x.size(0), C, device=x.device, dtype=x.dtype)
-    _check(lib().hyb_conv_silu(x.data_ptr(), xs, w.data_ptr(), state.data_ptr(), y.data_ptr(), C, plan.meta.data_ptr(),
+    if not w.is_contiguous() or (b is not None and (b.dtype != x.dtype or b.numel() != C or not b.is_contiguous())):
+        raise HybridOpsError("the convolution's weights are dense, its bias has the activation type")
+    _check(lib().hyb_conv_silu(x.data_ptr(), xs, w.data_ptr(), None if b is None else b.data_ptr(), state.data_ptr(), y.data_ptr(), C, plan.meta.data_ptr(),
                                plan.tok_seq.data_ptr(), x.size(0), len(plan.seqs), C, taps, _dt(x), _st()), "conv_silu")
     return y
 
@@ -1020,6 +1076,21 @@ def full_norm_append(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[tor
            "full_norm_append")
 
 
+def _chunk_tables(plan: BatchPlan, length: int, device: torch.device) -> Tuple[torch.Tensor, torch.Tensor, int]:
+    """The step's sequences cut into chunks of ``length`` tokens: ``{first row, tokens, sequence, 0}`` per chunk and ``{first
+    chunk, chunks}`` per sequence (int32, on the device), and the number of chunks.  The same for every layer of a step."""
+    key = f"chunks_{length}"
+    tabs = plan.shared.get(key)
+    if tabs is None:
+        chunks, per_seq = [], []
+        for i, (r0, n, _, _) in enumerate(plan.seqs):
+            per_seq.append((len(chunks), (n + length - 1) // length))
+            chunks += [(r0 + c, min(length, n - c), i, 0) for c in range(0, n, length)]
+        tabs = (torch.tensor(chunks, dtype=torch.int32).to(device), torch.tensor(per_seq, dtype=torch.int32).to(device), len(chunks))
+        plan.shared[key] = tabs
+    return tabs
+
+
 lightning_chunk_from = 16  # a step whose longest sequence brings at least this many tokens takes the chunked kernel
 
 
@@ -1054,15 +1125,7 @@ def lightning_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, deca
     ctab = stab = scratch = None
     nchunks = 0
     if variant == 2:
-        tabs = plan.shared.get("lightning_chunks")  # the same for every such layer of the step
-        if tabs is None:
-            chunks, per_seq = [], []
-            for i, (r0, n, _, _) in enumerate(plan.seqs):
-                per_seq.append((len(chunks), (n + 63) // 64))
-                chunks += [(r0 + c, min(64, n - c), i, 0) for c in range(0, n, 64)]
-            tabs = (torch.tensor(chunks, dtype=torch.int32).to(v.device), torch.tensor(per_seq, dtype=torch.int32).to(v.device), len(chunks))
-            plan.shared["lightning_chunks"] = tabs
-        ctab, stab, nchunks = tabs
+        ctab, stab, nchunks = _chunk_tables(plan, 64, v.device)
         scratch = torch.empty(nchunks, H, D, V, device=v.device, dtype=torch.float32)
     _check(lib().hyb_lightning(q.data_ptr(), _rows(q)[0], k.data_ptr(), _rows(k)[0], v.data_ptr(), _rows(v)[0],
                                decay.data_ptr(), state.data_ptr(), plan.meta.data_ptr(), out.data_ptr(), len(plan.seqs),
@@ -1081,6 +1144,93 @@ def norm_gate_rows(o: torch.Tensor, w: torch.Tensor, g: torch.Tensor, eps: float
     out = torch.empty(o.shape, device=o.device, dtype=out_dtype)
     _check(lib().hyb_norm_gate_rows(o.data_ptr(), w.data_ptr(), g.data_ptr(), _rows(g)[0], out.data_ptr(), o.size(0), o.size(1),
                                     float(eps), _dt(out), _st()), "norm_gate_rows")
+    return out
+
+
+ssd_chunk_from = 16  # as above, for the state-space recurrence with 16-bit activations
+ssd_chunk_len = 64   # tokens per chunk: 64 or 128
+
+
+def _ssd_chunk_smem(length: int, dim: int) -> int:
+    """Bytes of shared memory the chunked form's largest kernel needs."""
+    d = -(-dim // 16) * 16
+    return 2 * (2 * length * (d + 8) + 72 * length + 2 * 72 * d)
+
+
+def ssd_recurrence(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, d: torch.Tensor,
+                   state: torch.Tensor, plan: BatchPlan, heads: int, groups: int, dim: int, vdim: int, variant: int = 0,
+                   chunk: int = 0) -> torch.Tensor:
+    """State-space recurrence with one decay per head and token.  ``xbc [N, heads*vdim + 2*groups*dim]`` holds ``x | B | C``
+    (already activated), ``dt [N, heads]`` the raw step sizes (a column slice), ``dt_bias``, ``a_log``, ``d`` fp32 ``[heads]``:
+
+        ``dt <- softplus(dt + dt_bias)``,  ``S <- exp(-exp(a_log) dt) S + dt B x^T``,  ``y = S^T C + d x``
+
+    with ``S [dim, vdim]`` fp32 in ``state[slot, head]`` (read at the start of the step, written back at its end) and head
+    ``h`` on the ``B``, ``C`` of group ``h // (heads / groups)``.  Returns fp32 ``[N, heads * vdim]``.  ``variant`` (CUDA): 1 the
+    token scan; 2 chunks of ``chunk`` (64 or 128) tokens as tensor-core products, all chunks of the step in parallel (bf16);
+    0 chooses by the longest sequence and the type."""
+    N, H, G, D, V = xbc.size(0), heads, groups, dim, vdim
+    if state.dtype != torch.float32 or dt_bias.dtype != torch.float32 or a_log.dtype != torch.float32 or d.dtype != torch.float32:
+        raise HybridOpsError("recurrent state, decays and skip factors are fp32")
+    if xbc.size(1) != H * V + 2 * G * D or dt.size(1) != H or H % G:
+        raise HybridOpsError("x, B, C are [heads * vdim | groups * dim | groups * dim], dt has one column per head")
+    if not xbc.is_cuda:
+        out = torch.empty(N, H * V, dtype=torch.float32)
+        x, B, C = xbc.float().split((H * V, G * D, G * D), 1)
+        x = x.reshape(N, H, V)
+        B, C = (t.reshape(N, G, D).repeat_interleave(H // G, 1) for t in (B, C))
+        step = F.softplus(dt.float() + dt_bias)
+        decay = torch.exp(-torch.exp(a_log) * step)
+        for r0, n, slot, _ in plan.seqs:
+            S = state[slot].clone()
+            for t in range(r0, r0 + n):
+                S = decay[t][:, None, None] * S + B[t][:, :, None] * (step[t][:, None] * x[t])[:, None, :]
+                out[t] = (torch.einsum("hdv,hd->hv", S, C[t]) + d[:, None] * x[t]).reshape(-1)
+            state[slot] = S
+        return out
+    length = int(chunk) or ssd_chunk_len
+    if not variant:
+        long = max(n for _, n, _, _ in plan.seqs) >= ssd_chunk_from
+        if long and not chunk and _ssd_chunk_smem(length, D) > 200 * 1024:
+            length = 64
+        variant = 2 if long and xbc.dtype == torch.bfloat16 and _ssd_chunk_smem(length, D) <= 200 * 1024 else 1
+    if dt.dtype != xbc.dtype or not (state.is_contiguous() and dt_bias.is_contiguous() and a_log.is_contiguous() and d.is_contiguous()) \
+            or dt_bias.numel() != H or a_log.numel() != H or d.numel() != H or tuple(state.shape[1:]) != (H, D, V):
+        raise HybridOpsError("dt has the activation type; state and per-head numbers are dense")
+    out = torch.empty(N, H * V, device=xbc.device, dtype=torch.float32)
+    a = _SsdArgs()
+    a.xbc, a.dt, a.xbc_stride, a.dt_stride = xbc.data_ptr(), dt.data_ptr(), _rows(xbc)[0], _rows(dt)[0]
+    a.dt_bias, a.a_log, a.d, a.state, a.y = dt_bias.data_ptr(), a_log.data_ptr(), d.data_ptr(), state.data_ptr(), out.data_ptr()
+    a.meta, a.H, a.G, a.N, a.V, a.nseq = plan.meta.data_ptr(), H, G, D, V, len(plan.seqs)
+    if variant == 1:
+        _check(lib().hyb_ssd_scan(ctypes.byref(a), _dt(xbc), _st()), "ssd_scan")
+        return out
+    if xbc.dtype != torch.bfloat16:
+        raise HybridOpsError("the chunked form takes 16-bit activations")
+    ctab, stab, nchunks = _chunk_tables(plan, length, xbc.device)
+    u = torch.empty(nchunks, H, D, V, device=xbc.device, dtype=torch.float32)
+    before = torch.empty(nchunks, H, 2, D, V, device=xbc.device, dtype=torch.bfloat16)
+    decay = torch.empty(nchunks, H, device=xbc.device, dtype=torch.float32)
+    a.ctab, a.stab, a.nchunks = ctab.data_ptr(), stab.data_ptr(), nchunks
+    a.u, a.before, a.decay = u.data_ptr(), before.data_ptr(), decay.data_ptr()
+    _check(lib().hyb_ssd_chunked(ctypes.byref(a), length, _st()), "ssd_chunked")
+    return out
+
+
+def silu_gate_norm(y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, parts: int, eps: float, out_dtype: torch.dtype) -> torch.Tensor:
+    """``u = y * silu(z)`` for fp32 ``y [N, n]``; each of ``parts`` equal parts of a row of ``u`` is divided by its own root mean
+    square (``eps`` inside the root); times ``w [n]``, in ``out_dtype``."""
+    N, n = y.shape
+    if n % parts:
+        raise HybridOpsError("the parts of the norm are equal")
+    if not y.is_cuda:
+        u = (y * F.silu(z.float())).view(N, parts, n // parts)
+        return (_norm_torch(u, None, None, eps, "rms").reshape(N, n) * w.float()).to(out_dtype)
+    if y.dtype != torch.float32 or not y.is_contiguous() or w.dtype != out_dtype or z.dtype != out_dtype or not w.is_contiguous():
+        raise HybridOpsError("read-outs are dense fp32; weight and gate have the activation type")
+    out = torch.empty(N, n, device=y.device, dtype=out_dtype)
+    _check(lib().hyb_silu_gate_norm(y.data_ptr(), z.data_ptr(), _rows(z)[0], w.data_ptr(), out.data_ptr(), N, n, int(parts), float(eps),
+                                    _dt(out), _st()), "silu_gate_norm")
     return out
 
 
@@ -1202,8 +1352,8 @@ def row_update(x: torch.Tensor, y: Optional[torch.Tensor] = None, w: Optional[to
     * ``depth [rows, N, C]`` (fp32; ``x`` IS ``depth[index]``): ``depth[index + 1] = sum_(j <= index) depth_w[j] depth[j]``, the
       average over depth with ``depth_w`` fp32 ``[index + 1]``;
     * ``nxt``: returns what the next sublayer reads of the result (the average if there is one, else ``x``) in
-      ``out_dtype``: its norm and convolution (see :func:`norm_conv`).  On CUDA this needs a step of one token per
-      sequence; other steps call :func:`norm_conv` afterwards."""
+      ``out_dtype``: its norm and convolution (see :func:`norm_conv`).  On CUDA a convolution needs a step of one token per
+      sequence; other steps call :func:`norm_conv` afterwards.  A norm alone goes with any step."""
     if x.dtype != torch.float32:
         raise HybridOpsError("the residual stream is fp32")
     if depth is not None and depth_w.numel() != index + 1:
@@ -1220,8 +1370,8 @@ def row_update(x: torch.Tensor, y: Optional[torch.Tensor] = None, w: Optional[to
             depth[index + 1].copy_(acc)
             x = depth[index + 1]
         return None if nxt is None else norm_conv(x, nxt, plan, out_dtype)
-    if nxt is not None and not plan.one_token:
-        raise HybridOpsError("the next sublayer's input is fused only into steps of one token per sequence")
+    if nxt is not None and nxt.conv_w is not None and not plan.one_token:
+        raise HybridOpsError("the next sublayer's convolution is fused only into steps of one token per sequence")
     if not x.is_contiguous() or (depth is not None and not depth.is_contiguous()) or (copy is not None and not copy.is_contiguous()):
         raise HybridOpsError("residual rows are dense")
     N, C = x.shape

@@ -132,7 +132,7 @@ def test_traits_and_state_of_the_architecture():
     m = build(FULL, ("cpu", torch.float32))
     c = m.config
     assert (c.block, c.norm, c.dense_act, c.depth_average, c.tied_head) == ("sandwich", "layer", "polynorm", True, True)
-    assert c.latent == {"rot": "pairs", "gate": False, "p32": True}
+    assert c.latent == {"rot": "pairs", "gate": False, "sink": False, "p32": True}
     pool = m.new_pool(3, 16)
     assert pool.runs[1]["cache"] is pool.runs[0]["cache"] and pool.runs[3]["cache"] is pool.runs[2]["cache"]
     assert pool.runs[0]["canon1"].shape == (3, 2, 22) and pool.runs[0]["canon1"].dtype == torch.float32
