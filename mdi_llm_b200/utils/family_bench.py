@@ -30,6 +30,10 @@ whole q and k projections, a score cap and learned sinks, a layer on another lay
 linear recurrence, clamped gated experts with identity experts and a token-gated shared expert) beside the
 parallel-block design of the same width, whose attention and mixture of experts are the closest existing kernels; the
 recurrence is set beside the gated linear attention of the sandwich design, timed in the same run.
+
+``bench.py --family dufelix`` measures the RMS sandwich design (grouped-query attention, latent attention with sinks, state-space
+recurrence, gated feed-forward) beside the depth-averaged design of the same width, its closest model as a whole; single
+kernels also stand beside the post-norm design's grouped-query attention and recurrence and the sandwich design's convolution.
 """
 from __future__ import annotations
 
@@ -40,7 +44,25 @@ from typing import Any, Callable, Dict, List
 import torch
 
 __all__ = ["run_family_compare", "hybrid_bench_config", "vudelix_bench_config", "labepel_bench_config", "zudovik_bench_config",
-           "ratesun_bench_config"]
+           "ratesun_bench_config", "dufelix_bench_config"]
+
+
+def dufelix_bench_config(width: int) -> Dict[str, Any]:
+    """4 layers: attention, latent attention, two recurrences (the second with the first one's sizes and its own weights), each
+    with a gated feed-forward whose three matrices have as many weights as a dense ``4 * width`` one.  Attention sizes are
+    those of the other designs' bench models; the recurrence is twice as wide as the stream, heads of 64, state 128."""
+    h = width // 128
+    yarn = {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}
+    att = {"heads": h, "kv_heads": max(1, h // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+           "rot": {"dims": 64, "base": 500000.0, "scaling": yarn}}
+    lat = {"heads": h, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "q_rank": min(1536, width), "scale": 192 ** -0.5,
+           "rot": {"dims": 64, "base": 10000.0, "scaling": yarn}}
+    ssm = {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 8, "conv": 4, "norm_groups": 8}
+    mlp = {"kind": "dense", "ff": (8 * width // 3 + 63) // 64 * 64}
+    layers = [{"type": t, "mixer": dict(m), "mlp": dict(mlp)}
+              for t, m in (("attention", att), ("latent_attention", lat), ("mamba2", ssm), ("mamba2", ssm))]
+    return {"architecture": "Dufelix", "vocab": 32000, "width": width, "layers": layers, "norm": {"eps": 1e-6},
+            "embedding": {"scale": 32.0}}
 
 
 def ratesun_bench_config(width: int, window: int = 1024) -> Dict[str, Any]:
@@ -148,7 +170,7 @@ def _hybrid(width: int, prompt_len: int, batch: int, steps: int, warmup: int, de
 
     dev = torch.device("cuda")
     make = {"hybrid": hybrid_bench_config, "vudelix": vudelix_bench_config, "labepel": labepel_bench_config,
-            "zudovik": zudovik_bench_config, "ratesun": ratesun_bench_config}[design]
+            "zudovik": zudovik_bench_config, "ratesun": ratesun_bench_config, "dufelix": dufelix_bench_config}[design]
     cfg = HybridConfig.from_dict(make(width))
     model = HybridLM(cfg, {}).init_random(dev, torch.bfloat16, seed=1)
     params = sum(p.numel() for p in model.tensor_map().values())
@@ -182,7 +204,7 @@ def _hybrid(width: int, prompt_len: int, batch: int, steps: int, warmup: int, de
         out[f"decode_ms_b{b}"] = round(ms, 4)
         del r
     kernels = {"hybrid": _hybrid_kernels, "vudelix": _vudelix_kernels, "labepel": _labepel_kernels,
-               "zudovik": _zudovik_kernels, "ratesun": _ratesun_kernels}[design]
+               "zudovik": _zudovik_kernels, "ratesun": _ratesun_kernels, "dufelix": _dufelix_kernels}[design]
     out["kernels"] = kernels(model, prompt_len, batch)
     return out
 
@@ -421,6 +443,92 @@ def _ratesun_kernels(model: Any, T: int, batch: int) -> List[Dict[str, Any]]:
             4.0 * N * C * a.size(1))
         zs = H.linear(h, side.gate)
         rec("token_side_gate", "token_side_gate", phase, lambda: H.token_side_gate(zs, model.side_embed, tok, 0), 6.0 * N * side.dim)
+        del pool
+    return rows
+
+
+def _dufelix_kernels(model: Any, T: int, batch: int) -> List[Dict[str, Any]]:
+    """The RMS sandwich design's kernels alone; ``like`` names the row of ``_ratesun_kernels`` (or of ``_zudovik_kernels`` for the
+    grouped-query attention, the recurrence and its norm, of ``_hybrid_kernels`` for the convolution) with the corresponding work."""
+    from ..ops import hybrid as H
+
+    pk = _peaks()
+    dev, dt, cfg = model.device, model.dtype, model.config
+    C = cfg.width
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    rows: List[Dict[str, Any]] = []
+
+    def rec(name: str, like: str, phase: str, fn: Callable[[], Any], nbytes: float, flops: float = 0.0) -> None:
+        ms = _time(fn, 5, 3, flush)
+        rows.append({"kernel": name, "like": like, "phase": phase, "ms": round(ms, 4), "gb_s": round(nbytes / ms / 1e6, 1),
+                     "tflops": round(flops / ms / 1e9, 2),
+                     "frac_of_roofline": round(max(nbytes / ms / 1e6 / pk["hbm_gbs"], flops / ms / 1e9 / pk["bf16_tflops"]), 4),
+                     "peaks": pk["source"]})
+
+    blk, att, lat, ssm = model.blocks[0], model.blocks[0].mix, model.blocks[1].mix, model.blocks[2].mix
+    for phase, lengths, starts in (("prefill", [T], [0]), ("decode", [1] * batch, [T] * batch)):
+        n_seq, N = len(lengths), sum(lengths)
+        pool = model.new_pool(n_seq, T + 8)
+        plan = H.BatchPlan.make(lengths, list(range(n_seq)), starts, dev)
+        pool.runs[0]["cache"].normal_()
+        pool.runs[1]["cache"].normal_()
+        pairs = sum(s + i + 1 for n, s in zip(lengths, starts) for i in range(n))  # visible (query, key) pairs
+        keys = sum(s + n for n, s in zip(lengths, starts))
+        x, y, h = torch.randn(N, C, device=dev), torch.randn(N, C, device=dev).to(dt), torch.randn(N, C, device=dev).to(dt)
+        tok = torch.randint(0, cfg.vocab, (N,), device=dev, dtype=torch.int32)
+        rec("embed_rows[scale]", "embed_rows[scale]", phase, lambda: H.embed_rows(model.embed, tok, None, plan, cfg.embed_scale), N * C * 6.0)
+        rec("row_update[rms, + next norm]", "row_update" if phase == "prefill" else "row_update[+ next norm, convolution]", phase,
+            lambda: H.row_update(x, y, blk.norm1b.w, None, 1e-6, "rms", nxt=blk._input2({}), plan=plan, out_dtype=dt), N * C * 12.0)
+        # grouped-query attention
+        Hh, G, D, V = att.H, att.G, att.D, att.V
+        cache = pool.runs[0]["cache"]
+        p = H.linear(h, att.w_in)
+        q, g = att.col(p, "q"), att.col(p, "g")
+        rec("window_append[halves, no norm]", "full_norm_append", phase,
+            lambda: H.window_append(q, att.col(p, "k"), att.col(p, "v"), att.inv_freq, cache, plan, Hh, G, D, V, att.nrot, 1e-6, norm=False,
+                                    pairing=att.pairing, amp=att.amp), 2.0 * N * (2 * Hh * D + 2 * G * (D + V)))
+        if phase == "prefill":
+            rec("grouped_attn[fused, gate]", "causal_attn(gemm+softmax)", phase, lambda: att._fused(q, g, cache, plan),
+                2.0 * N * (Hh * (D + V) + G * (D + V)), 2.0 * Hh * pairs * (D + V))
+        else:
+            rec("window_attn[causal, gate]", "window_attn[causal, cap, learned sink]", phase,
+                lambda: H.window_attn(q, g, cache, plan, Hh, G, D, V, att.scale, 0),
+                2.0 * G * keys * (D + V) + 2.0 * N * Hh * (D + V), 2.0 * Hh * pairs * (D + V))
+        # latent attention
+        Hh, D, R, V, L = lat.H, lat.D, lat.R, lat.V, lat.L
+        cache = pool.runs[1]["cache"]
+        p = H.linear(h, lat.w_in)
+        rec("latent_prepare", "latent_prepare", phase,
+            lambda: H.latent_prepare(lat.col(p, "dq"), lat.dq_norm, lat.col(p, "dkv"), lat.dkv_norm, lat.inv_freq, cache, plan, R, L,
+                                     lat.nrot, 1e-6, lat.pairing, lat.amp), 4.0 * N * (L + R + lat.QR))
+        q = H.linear(h[:, :lat.QR].contiguous(), lat.uq)
+        if phase == "prefill":
+            rec("rotate_heads", "rotate_heads", phase,
+                lambda: H.rotate_heads(q, lat.inv_freq, plan, Hh, D, R, lat.nrot, lat.pairing, lat.amp), 4.0 * N * Hh * R)
+            rec("latent_attn_expanded[sink]", "latent_attn_expanded[window]", phase, lambda: lat._expanded(q, cache, plan),
+                2.0 * N * Hh * (D + R + V), 2.0 * T * L * Hh * (D + V) + 2.0 * Hh * pairs * (D + R + V))
+        else:
+            qlat = torch.randn(Hh, N, L, device=dev)
+            rec("latent_attn[sink, rotation]", "latent_attn[window, rotation]", phase,
+                lambda: H.latent_attn(qlat, q, cache, plan, Hh, D, R, L, lat.scale, inv_freq=lat.inv_freq, nrot=lat.nrot,
+                                      pairing=lat.pairing, amp=lat.amp, sink=lat.sink32),
+                6.0 * Hh * N * L + 2.0 * Hh * N * R + 2.0 * (L + R) * keys, 2.0 * Hh * pairs * (2 * L + R))
+        # the recurrence
+        Hh, V, S, G, a, b = ssm.H, ssm.V, ssm.N, ssm.G, ssm.inner, ssm.inner + ssm.ch
+        st = pool.runs[2]
+        p = H.linear(h, ssm.w_in)
+        rec("conv_silu[bias]", "conv_silu", phase, lambda: H.conv_silu(p[:, a:b], ssm.conv, st["conv"], plan, ssm.conv_b), 4.0 * N * ssm.ch)
+        xbc = H.conv_silu(p[:, a:b], ssm.conv, st["conv"], plan, ssm.conv_b)
+        rec("ssd_recurrence[chunks]" if phase == "prefill" else "ssd_recurrence[scan]",
+            "lightning_recurrence[chunks]" if phase == "prefill" else "lightning_recurrence[scan]", phase,
+            lambda: H.ssd_recurrence(xbc, p[:, b:b + Hh], ssm.dt_bias32, ssm.A_log32, ssm.skip32, st["state"], plan, Hh, G, S, V),
+            2.0 * N * (ssm.ch + Hh) + 4.0 * N * a + 8.0 * n_seq * Hh * S * V, 4.0 * N * Hh * S * V)
+        o = torch.randn(N, a, device=dev)
+        rec("silu_gate_norm[parts]", "norm_gate_rows", phase, lambda: H.silu_gate_norm(o, p[:, :a], ssm.norm, ssm.parts, 1e-6, dt), N * a * 8.0)
+        ff = blk.mlp
+        gu = H.linear(h, ff.w_in)
+        rec("act_mul[gelu]", "act_mul[clamped]", phase, lambda: H.act_mul(gu, "gelu_tanh"), 6.0 * N * ff.ff)
+        rec("dense_ff(gemm+gelu*up)", "dense_ff(gemm+poly_norm)", phase, lambda: ff(h), 6.0 * C * ff.ff + 4.0 * N * C, 6.0 * N * C * ff.ff)
         del pool
     return rows
 
@@ -701,6 +809,33 @@ def run_family_compare(widths: List[int], prompt_len: int = 2048, batch: int = 8
                     if other and other["frac_of_roofline"] else None
             results.append({"width": w, "ratesun": new, "hybrid": old, "prenorm_side": side_rows})
         return {"metric": "family_compare", "family": "ratesun", "dtype": "bf16", "data": "synthetic", "prompt_len": prompt_len,
+                "decode_batch": batch, "steps": steps, "warmup": warmup, "l2": "flushed between single-kernel timings",
+                "results": results}
+    if family == "dufelix":
+        from ..models.config import HybridConfig
+        from ..models.hybrid import HybridLM
+
+        for w in widths:
+            new = _hybrid(w, prompt_len, batch, steps, warmup, "dufelix")
+            torch.cuda.empty_cache()
+            old = _hybrid(w, prompt_len, batch, steps, warmup, "ratesun")
+            torch.cuda.empty_cache()
+            theirs = {(k["kernel"], k["phase"]): k for k in old["kernels"]}
+            others: List[Dict[str, Any]] = []  # like kernels of designs that are not timed as a whole here
+            for make, rows_of in ((zudovik_bench_config, _zudovik_kernels), (hybrid_bench_config, _hybrid_kernels)):
+                model = HybridLM(HybridConfig.from_dict(make(w)), {}).init_random(torch.device("cuda"), torch.bfloat16, seed=1)
+                wanted = {k["like"] for k in new["kernels"]}
+                others += [k for k in rows_of(model, prompt_len, batch) if k["kernel"] in wanted and (k["kernel"], k["phase"]) not in theirs]
+                theirs.update({(k["kernel"], k["phase"]): k for k in others})
+                del model
+                torch.cuda.empty_cache()
+            for k in new["kernels"]:  # how far from its roofline, relative to the like kernel (above 1: this one is nearer)
+                other = theirs.get((k["like"], k["phase"]))
+                k["like_ms"] = other["ms"] if other else None
+                k["roofline_vs_like"] = round(k["frac_of_roofline"] / other["frac_of_roofline"], 3) \
+                    if other and other["frac_of_roofline"] else None
+            results.append({"width": w, "dufelix": new, "ratesun": old, "like_kernels": others})
+        return {"metric": "family_compare", "family": "dufelix", "dtype": "bf16", "data": "synthetic", "prompt_len": prompt_len,
                 "decode_batch": batch, "steps": steps, "warmup": warmup, "l2": "flushed between single-kernel timings",
                 "results": results}
     if family == "labepel":

@@ -198,16 +198,16 @@ def random_tensors(cfg: Dict[str, Any], seed: int = 0) -> Dict[str, torch.Tensor
             continue
         m, pre = spec["mixer"], f"l{i}.mix."
         for n in ("norm1", "norm1b") + (("norm2", "norm2b") if spec.get("mlp") else ()):
-            W[f"l{i}.{n}"] = vec(C, 1.0, 0.1)
+            W[f"l{i}.{n}"] = vec(C, 0.4 if n.endswith("b") else 1.0, 0.1)
         if spec["type"] == "attention":
             Hh, G, D, V = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-            W[pre + "q"], W[pre + "k"], W[pre + "v"] = mat(Hh * D, C, 1.5), mat(G * D, C, 1.5), mat(G * V, C)
+            W[pre + "q"], W[pre + "k"], W[pre + "v"] = mat(Hh * D, C), mat(G * D, C), mat(G * V, C)
             W[pre + "g"], W[pre + "o"] = mat(Hh, C, 2.0), mat(C, Hh * V)
         elif spec["type"] == "latent_attention":
             Hh, D, R, V, L, Q = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], m["q_rank"]
-            W[pre + "dq"], W[pre + "dq.norm"], W[pre + "uq"] = mat(Q, C), vec(Q, 1.0, 0.2), mat(Hh * (D + R), Q, 2.0)
+            W[pre + "dq"], W[pre + "dq.norm"], W[pre + "uq"] = mat(Q, C), vec(Q, 1.0, 0.2), mat(Hh * (D + R), Q, 1.5)
             W[pre + "dkv"], W[pre + "dkv.norm"] = mat(L + R, C), vec(L, 1.0, 0.2)
-            W[pre + "uk"], W[pre + "uv"], W[pre + "o"] = mat(Hh * D, L, 2.0), mat(Hh * V, L), mat(C, Hh * V)
+            W[pre + "uk"], W[pre + "uv"], W[pre + "o"] = mat(Hh * D, L, 1.5), mat(Hh * V, L), mat(C, Hh * V)
             W[pre + "sink"] = vec(Hh, 1.0, 1.0)
         else:
             Hh, V, N, G = m["heads"], m["vdim"], m["state"], m["groups"]
