@@ -33,7 +33,7 @@ def nvcc_path() -> Optional[str]:
 # such a model compiles these files only, and they are built with IEEE math (no ``--use_fast_math``) because its
 # 32-bit mode is held to 32-bit rounding.
 HYBRID_LIB = HERE / "_mdi_hybrid.so"
-HYBRID_SOURCES = ("hybrid_mixers.cu", "hybrid_rows.cu", "hybrid_latent.cu", "hybrid_ssd.cu")
+HYBRID_SOURCES = ("hybrid_mixers.cu", "hybrid_rows.cu", "hybrid_latent.cu", "hybrid_grouped.cu", "hybrid_ssd.cu")
 HYBRID_HEADERS = ("hybrid_common.cuh", "hybrid_mma.cuh")
 
 

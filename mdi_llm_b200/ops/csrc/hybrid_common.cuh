@@ -73,6 +73,9 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 __device__ __forceinline__ float sigmoidf_(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplusf_(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 __device__ __forceinline__ float siluf_(float x) { return x / (1.f + expf(-x)); }
+// SiLU for results that are rounded to T: with a 16-bit T the approximate exponential and division (a few ulp of fp32) do
+template <typename T> __device__ __forceinline__ float silu_as(float x) { return siluf_(x); }
+template <> __device__ __forceinline__ float silu_as<bf16>(float x) { return __fdividef(x, 1.f + __expf(-x)); }
 __device__ __forceinline__ float gelu_erff_(float x) { return 0.5f * x * (1.f + erff(x * 0.70710678118654752f)); }
 
 }  // namespace hyb

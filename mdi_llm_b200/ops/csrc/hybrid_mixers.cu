@@ -523,49 +523,76 @@ __global__ void conv_silu_kernel(const T* __restrict__ x, long long x_stride, co
     y[(size_t)tok * y_stride + c] = from_f<T>(siluf_(acc));
   }
 }
-// The same for prompts in rows of whole 16-byte groups: a thread owns 8 channels of `tile` consecutive token rows, keeps
-// the taps and the last taps - 1 inputs in registers and reads every input row once (plus taps - 1 rows in front).
+// The same for prompts in rows of whole 16-byte groups: a thread owns 8 channels of CV_ROWS consecutive token rows.  It
+// requests those rows and the TAPS - 1 in front of them at once (rows of earlier steps from the slot) and keeps them in
+// their storage type; rows of another sequence than the token's own count as that sequence's stored inputs.
+#define CV_ROWS 8
+template <typename T> struct Pack8;  // 8 values as they are stored
+template <> struct Pack8<bf16> {
+  uint4 v;
+  __device__ __forceinline__ void load(const bf16* p) { v = *reinterpret_cast<const uint4*>(p); }
+  __device__ __forceinline__ void get(float* f) const {
+    const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { f[2 * i] = __uint_as_float(w[i] << 16); f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u); }
+  }
+};
+template <> struct Pack8<float> {
+  float4 a, b;
+  __device__ __forceinline__ void load(const float* p) { a = *reinterpret_cast<const float4*>(p); b = *reinterpret_cast<const float4*>(p + 4); }
+  __device__ __forceinline__ void get(float* f) const { f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w; }
+};
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128) conv_silu_rows_kernel(const T* __restrict__ x, long long x_stride,
                                                              const T* __restrict__ w, const T* __restrict__ b,
                                                              const T* __restrict__ state, T* __restrict__ y,
                                                              long long y_stride, const int* __restrict__ meta,
-                                                             const int* __restrict__ tok_seq, int N, int C, int tile) {
+                                                             const int* __restrict__ tok_seq, int N, int C) {
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
   if (c >= C) return;
-  float wt[TAPS][8], bias[8], past[TAPS][8];
+  const int first = blockIdx.x * CV_ROWS;
+  Pack8<T> in[CV_ROWS + TAPS - 1];
 #pragma unroll
-  for (int e = 0; e < 8; ++e) {
-    bias[e] = b ? to_f(b[c + e]) : 0.f;
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) wt[j][e] = to_f(w[(size_t)(c + e) * TAPS + j]);
+  for (int i = 0; i < CV_ROWS + TAPS - 1; ++i) {
+    const int tok = first + i - (TAPS - 1);
+    in[i].load(x + (size_t)min(max(tok, 0), N - 1) * x_stride + c);
   }
-  const int first = blockIdx.x * tile, last = min(N, first + tile);
-  int seq = -1, start = 0;
-  for (int tok = first; tok < last; ++tok) {
-    if (tok_seq[tok] != seq) {  // a sequence begins, or the tile begins inside one: its last TAPS - 1 inputs
-      seq = tok_seq[tok];
-      const int* m = meta + 4 * seq;
-      start = m[0];
-      const T* st = state + (size_t)m[2] * (TAPS - 1) * C + c;
+  float wt[TAPS][8], bias[8];
+  {
+    Pack8<T> pw[TAPS];  // 8 channels x TAPS weights are 8 * TAPS consecutive values
+    float f[TAPS * 8];
 #pragma unroll
-      for (int j = 0; j < TAPS - 1; ++j) {
-        int src = tok - start - (TAPS - 1 - j);
-        load8(src >= 0 ? x + (size_t)(start + src) * x_stride + c : st + (size_t)(TAPS - 1 + src) * C, past[j]);
-      }
+    for (int j = 0; j < TAPS; ++j) {
+      pw[j].load(w + (size_t)c * TAPS + j * 8);
+      pw[j].get(f + 8 * j);
     }
-    load8(x + (size_t)tok * x_stride + c, past[TAPS - 1]);
-    float o[8];
 #pragma unroll
-    for (int e = 0; e < 8; ++e) {
-      float acc = bias[e];
+    for (int e = 0; e < 8; ++e)
 #pragma unroll
-      for (int j = 0; j < TAPS; ++j) acc += wt[j][e] * past[j][e];
-      o[e] = siluf_(acc);
+      for (int j = 0; j < TAPS; ++j) wt[j][e] = f[e * TAPS + j];
 #pragma unroll
-      for (int j = 0; j < TAPS - 1; ++j) past[j][e] = past[j + 1][e];
+    for (int e = 0; e < 8; ++e) bias[e] = 0.f;
+    if (b) load8(b + c, bias);
+  }
+#pragma unroll
+  for (int i = 0; i < CV_ROWS; ++i) {
+    const int tok = first + i;
+    if (tok >= N) return;
+    const int* m = meta + 4 * tok_seq[tok];
+    const int local = tok - m[0];
+    float acc[8], f[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) acc[e] = bias[e];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+      if (local - (TAPS - 1 - j) >= 0) in[i + j].get(f);
+      else load8(state + ((size_t)m[2] * (TAPS - 1) + (j + local)) * C + c, f);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) acc[e] += wt[j][e] * f[e];
     }
-    store8(y + (size_t)tok * y_stride + c, o);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) acc[e] = silu_as<T>(acc[e]);
+    store8(y + (size_t)tok * y_stride + c, acc);
   }
 }
 // Steps of one token per sequence: the convolution and the shift of its stored inputs in one pass, a thread per channel.
@@ -1093,12 +1120,11 @@ int hyb_conv_silu(const void* x, long long x_stride, const void* w, const void* 
                  (conv_silu_step_kernel<float><<<grid, 256, 0, st>>>((const float*)x, x_stride, (const float*)w, (const float*)b, (float*)state, (float*)y, y_stride, meta, tok_seq, C, taps)));
     return (int)cudaGetLastError();
   }
-  uintptr_t bits = (uintptr_t)x | (uintptr_t)y | (uintptr_t)state;
+  uintptr_t bits = (uintptr_t)x | (uintptr_t)y | (uintptr_t)state | (uintptr_t)w | (uintptr_t)b;
   const bool vec = taps >= 2 && taps <= 4 && (bits & 15) == 0 && ((C | x_stride | y_stride) & 7) == 0;
   if (vec) {
-    const int cb = (C / 8 + 127) / 128, tile = max(1, min(16, (int)((long long)N * cb / 592)));
-    dim3 vgrid((N + tile - 1) / tile, cb);
-#define CR(T, TP) conv_silu_rows_kernel<T, TP><<<vgrid, 128, 0, st>>>((const T*)x, x_stride, (const T*)w, (const T*)b, (const T*)state, (T*)y, y_stride, meta, tok_seq, N, C, tile)
+    dim3 vgrid((N + CV_ROWS - 1) / CV_ROWS, (C / 8 + 127) / 128);
+#define CR(T, TP) conv_silu_rows_kernel<T, TP><<<vgrid, 128, 0, st>>>((const T*)x, x_stride, (const T*)w, (const T*)b, (const T*)state, (T*)y, y_stride, meta, tok_seq, N, C)
     if (dt == 0) { if (taps == 2) CR(bf16, 2); else if (taps == 3) CR(bf16, 3); else CR(bf16, 4); }
     else { if (taps == 2) CR(float, 2); else if (taps == 3) CR(float, 3); else CR(float, 4); }
 #undef CR
@@ -1209,6 +1235,16 @@ __device__ __forceinline__ float gelu_tanhf_(float z) {
   return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 
+// VEC values as they are stored; VEC = 4 is one 8-byte (bf16) or 16-byte (fp32) access
+template <int VEC> __device__ __forceinline__ void copy_vec(bf16* dst, const bf16* src) {
+  if (VEC == 4) *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<const uint2*>(src);
+  else dst[0] = src[0];
+}
+template <int VEC> __device__ __forceinline__ void copy_vec(float* dst, const float* src) {
+  if (VEC == 4) *reinterpret_cast<float4*>(dst) = *reinterpret_cast<const float4*>(src);
+  else dst[0] = src[0];
+}
+
 // One block per token.  Warps walk the H query heads and then the G key heads: rotate the first `nrot` entries
 // (entry 2i with 2i+1, or with interleaved == 0 entry i with i + nrot/2; angle pos * inv_freq[i], cosine and sine times
 // amp), with norm != 0 divide the head by its root mean square over D, store queries
@@ -1228,7 +1264,13 @@ __global__ void window_append_kernel(T* __restrict__ q, long long q_stride, cons
   int pos = m[3] + (t - m[0]);
   T* row = cache + (size_t)m[2] * slot_stride + (size_t)pos * (G * (D + V));
   int lane = threadIdx.x & 31, w = threadIdx.x >> 5, nw = blockDim.x >> 5;
-  float fpos = (float)pos;
+  __shared__ float2 turn[16 * WA_MAXD];  // cosine and sine of every pair: the heads of a token share their angles
+  for (int i = threadIdx.x; i < nrot >> 1; i += blockDim.x) {
+    float sn, cs;
+    sincosf((float)pos * inv_freq[i], &sn, &cs);
+    turn[i] = make_float2(cs * amp, sn * amp);
+  }
+  __syncthreads();
   for (int hv = w; hv < H + G; hv += nw) {
     const T* src = hv < H ? q + (size_t)t * q_stride + (size_t)hv * D : k + (size_t)t * k_stride + (size_t)(hv - H) * D;
     T* dst = hv < H ? q + (size_t)t * q_stride + (size_t)hv * D : row + (size_t)(hv - H) * D;
@@ -1244,11 +1286,9 @@ __global__ void window_append_kernel(T* __restrict__ q, long long q_stride, cons
         if (d < nrot) {
           const int half = nrot >> 1;
           const bool second = interleaved ? d & 1 : d >= half;
-          float o = to_f(src[interleaved ? d ^ 1 : (second ? d - half : d + half)]), sn, cs;
-          sincosf(fpos * inv_freq[interleaved ? d >> 1 : (second ? d - half : d)], &sn, &cs);
-          sn *= amp;
-          cs *= amp;
-          x = second ? x * cs + o * sn : x * cs - o * sn;
+          float o = to_f(src[interleaved ? d ^ 1 : (second ? d - half : d + half)]);
+          float2 r = turn[interleaved ? d >> 1 : (second ? d - half : d)];
+          x = second ? x * r.x + o * r.y : x * r.x - o * r.y;
         }
         y[c] = x;
         ss += x * x;
@@ -1272,6 +1312,68 @@ __global__ void window_append_kernel(T* __restrict__ q, long long q_stride, cons
     return;
   }
   for (int i = threadIdx.x; i < G * V; i += blockDim.x) vd[i] = vs[i];
+}
+
+// The same without a norm: one block per token, a thread owns VEC rotated pairs of a head (both members, so queries turn in
+// place), VEC entries a key keeps as they are, or VEC values.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) rotate_append_kernel(T* __restrict__ q, long long q_stride, const T* __restrict__ k,
+                                                            long long k_stride, const T* __restrict__ v, long long v_stride,
+                                                            const float* __restrict__ inv_freq, T* __restrict__ cache,
+                                                            long long slot_stride, const int* __restrict__ meta,
+                                                            const int* __restrict__ tok_seq, int H, int G, int D, int V, int nrot,
+                                                            int interleaved, float amp) {
+  __shared__ float2 turn[16 * WA_MAXD];
+  const int t = blockIdx.x, half = nrot >> 1;
+  const int* m = meta + 4 * tok_seq[t];
+  const int pos = m[3] + (t - m[0]);
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float sn, cs;
+    sincosf((float)pos * inv_freq[i], &sn, &cs);
+    turn[i] = make_float2(cs * amp, sn * amp);
+  }
+  q += (size_t)t * q_stride;
+  k += (size_t)t * k_stride;
+  v += (size_t)t * v_stride;
+  T* row = cache + (size_t)m[2] * slot_stride + (size_t)pos * (G * (D + V));
+  const int per = half / VEC, rest = (D - nrot) / VEC, vals = V / VEC;
+  const int n1 = (H + G) * per, n2 = n1 + G * rest, n3 = n2 + G * vals;
+  __syncthreads();
+  for (int idx = threadIdx.x; idx < n3; idx += blockDim.x) {
+    if (idx < n1) {
+      const int h = idx / per, i = (idx - h * per) * VEC;
+      const T* src = h < H ? q + (size_t)h * D : k + (size_t)(h - H) * D;
+      T* dst = h < H ? q + (size_t)h * D : row + (size_t)(h - H) * D;
+      alignas(16) T a[VEC], b[VEC];
+      if (interleaved) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) { a[e] = src[2 * (i + e)]; b[e] = src[2 * (i + e) + 1]; }
+      } else {
+        copy_vec<VEC>(a, src + i);
+        copy_vec<VEC>(b, src + half + i);
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        const float x = to_f(a[e]), y = to_f(b[e]);
+        const float2 r = turn[i + e];
+        a[e] = from_f<T>(x * r.x - y * r.y);
+        b[e] = from_f<T>(y * r.x + x * r.y);
+      }
+      if (interleaved) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) { dst[2 * (i + e)] = a[e]; dst[2 * (i + e) + 1] = b[e]; }
+      } else {
+        copy_vec<VEC>(dst + i, a);
+        copy_vec<VEC>(dst + half + i, b);
+      }
+    } else if (idx < n2) {
+      const int h = (idx - n1) / rest, i = nrot + (idx - n1 - h * rest) * VEC;
+      copy_vec<VEC>(row + (size_t)h * D + i, k + (size_t)h * D + i);
+    } else {
+      const int i = (idx - n2) * VEC;
+      copy_vec<VEC>(row + (size_t)G * D + i, v + i);
+    }
+  }
 }
 
 // One block per (token, key/value head); warp w is query head g * rep + w.  A tile of 32 cached keys and values is
@@ -1939,6 +2041,16 @@ int hyb_window_append(void* q, long long q_stride, const void* k, long long k_st
   if (N == 0) return 0;
   if (D > 32 * WA_MAXD || nrot > D || (nrot & 1) || (nrot > 0 && !inv_freq)) return -3;
   if (lam && !v_first) return -2;
+  if (!norm && !lam && !qw && !kw) {
+    uintptr_t bits = (uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)cache;
+    const bool vec = (bits & 15) == 0 && ((q_stride | k_stride | v_stride | slot_stride) & 3) == 0 && ((D | V | (nrot >> 1)) & 3) == 0;
+    const int work = ((H + G) * (nrot >> 1) + G * (D - nrot + V)) / (vec ? 4 : 1), th = work >= 256 ? 256 : work > 128 ? 192 : 128;
+#define RA(T, VC) rotate_append_kernel<T, VC><<<N, th, 0, st>>>((T*)q, q_stride, (const T*)k, k_stride, (const T*)v, v_stride, inv_freq, (T*)cache, slot_stride, meta, tok_seq, H, G, D, V, nrot, interleaved, amp)
+    if (dt == 0) { if (vec) RA(bf16, 4); else RA(bf16, 1); }
+    else { if (vec) RA(float, 4); else RA(float, 1); }
+#undef RA
+    return (int)cudaGetLastError();
+  }
   HYB_DISPATCH(dt,
                (window_append_kernel<bf16><<<N, 128, 0, st>>>((bf16*)q, q_stride, (const bf16*)k, k_stride, (const bf16*)v,
                                                               v_stride, inv_freq, (bf16*)cache, slot_stride, meta, tok_seq,
@@ -1985,6 +2097,14 @@ int hyb_window_attn(const void* q, long long q_stride, const void* gate, long lo
     if (nsplit > 1)
       window_combine_kernel<float><<<cgrid, 128, 0, st>>>(part_acc, part_ml, (const float*)gate, g_stride, (float*)out, N, H, V, nsplit, sink, gate_mode, sink_vals);
   }
+  return (int)cudaGetLastError();
+}
+
+int hyb_window_combine(const float* part_acc, const float* part_ml, const void* gate, long long g_stride, void* out, int N, int H, int V,
+                       int nsplit, int sink, int gate_mode, const float* sink_vals, int dt, cudaStream_t st) {
+  dim3 cgrid(N, (H + 3) / 4);
+  HYB_DISPATCH(dt, (window_combine_kernel<bf16><<<cgrid, 128, 0, st>>>(part_acc, part_ml, (const bf16*)gate, g_stride, (bf16*)out, N, H, V, nsplit, sink, gate_mode, sink_vals)),
+               (window_combine_kernel<float><<<cgrid, 128, 0, st>>>(part_acc, part_ml, (const float*)gate, g_stride, (float*)out, N, H, V, nsplit, sink, gate_mode, sink_vals)));
   return (int)cudaGetLastError();
 }
 

@@ -8,13 +8,15 @@
 // slot, position of the first token}.  Two forms:
 //
 //  * ssd_scan_kernel: token by token, state in registers; one-token steps, short portions, and the 32-bit mode.
-//  * ssd_chunk_state / ssd_chunk_scan / ssd_chunk_out: prompts with 16-bit activations, parallel over chunks of CL tokens.
-//    With c_t the running sum of log a inside a chunk and S0 the state before it,
-//      y_t = exp(c_t) S0^T C_t + sum_{s <= t} exp(c_t - c_s) dt_s (C_t . B_s) x_s + D x_t
+//  * ssd_decay_kernel, ssd_walk_kernel, ssd_out_kernel: prompts with 16-bit activations, in chunks.  With c_t the running sum of log a
+//    inside a chunk and S0 the state before it,
 //      S'  = exp(c_last) S0 + sum_s exp(c_last - c_s) dt_s B_s x_s^T
-//    so a chunk is four small matrix products.  They run on the tensor cores: x, B, C are bf16 as they come, everything
-//    fp32 that meets them (weights, states) enters as a bf16 number plus its bf16 remainder, sums are fp32.  Running
-//    sums of log a are kept as a pair of floats: only differences of them are exponentiated, and those are never positive.
+//      y_t = exp(c_t) S0^T C_t + sum_{s <= t} exp(c_t - c_s) dt_s (C_t . B_s) x_s + D x_t
+//    Only the first line chains the chunks: the walk follows it through a sequence with the state in registers and leaves
+//    the state before every chunk; the second line then runs for all chunks at once.  Both are small matrix products on
+//    the tensor cores: x, B, C are bf16 as they come, everything fp32 that meets them (weights, states) enters as a bf16
+//    number plus its bf16 remainder, sums are fp32.  Running sums of log a are kept as a pair of floats: only differences
+//    of them are exponentiated, and those are never positive.
 #include "hybrid_mma.cuh"
 
 namespace hyb {
@@ -24,12 +26,11 @@ struct SsdArgs {
   const float *dt_bias, *a_log, *d;  // [H]
   float* state;                      // [slots][H][N][V]
   float* y;                          // [tokens][H * V]
-  const int *meta, *ctab, *stab;     // chunk c: {first token row, tokens, sequence, 0}; sequence: {first chunk, chunks}
-  float* u;                          // [chunks][H][N][V]: what a chunk adds to the state
-  float* decay;                      // [chunks][H]: exp(c_last)
+  const int *meta, *ctab, *stab;     // chunk of SSD_CL tokens: {first token row, tokens, sequence, 0}; sequence: {first chunk, chunks}
   void* before;                      // [chunks][H][2][N][V] bf16: the state before a chunk, rounded, and the remainder
+  float4* dec;                       // [H][tokens]: {running sum of log a in its 64 tokens (two floats), dt, exp(c_last - c) dt}
   long long xbc_stride, dt_stride;
-  int H, G, N, V, nseq, nchunks;
+  int H, G, N, V, nseq, nchunks, tokens;
 };
 
 // Block = (sequence, head, 32 value columns): lane = column, warp w owns the state rows w, w + 8, ..
@@ -96,25 +97,37 @@ __device__ __forceinline__ float2 pair_add(float2 a, float2 b) {
 }
 __device__ __forceinline__ float pair_diff(float2 a, float2 b) { return (a.x - b.x) + (a.y - b.y); }
 
-// dts[s] = dt of the chunk's token s, cum[s] = log a_0 + .. + log a_s; tokens from len on: dt 0, log a 0.  One warp.
-template <int CL>
-__device__ __forceinline__ void chunk_decays(const SsdArgs& a, int row0, int len, int h, int lane, float* dts, float2* cum) {
+// Step sizes and decays of 64 tokens at a time (the steps of the walk), one warp per 64 tokens and head: dt, the running sum
+// c of log a, and what weighs a token in the state after the 64: exp(c_last - c) dt.
+#define SW_L 64
+#define SSD_CL 128  // tokens per chunk of the outputs: the state before every second step of the walk is written out
+__global__ void __launch_bounds__(256) ssd_decay_kernel(SsdArgs a) {
+  const int* ch = a.ctab + 4 * blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, piece = warp & 1, h = blockIdx.y * 4 + (warp >> 1);
+  const int row0 = ch[0] + piece * SW_L, len = min(SW_L, ch[1] - piece * SW_L);
+  if (h >= a.H || len <= 0) return;
   const float bias = a.dt_bias[h], rate = expf(a.a_log[h]);
-  float2 carry = make_float2(0.f, 0.f);
-  for (int s0 = 0; s0 < CL; s0 += 32) {
-    const int s = s0 + lane;
-    float dt = 0.f;
-    if (s < len) dt = softplusf_(to_f(((const bf16*)a.dt)[(size_t)(row0 + s) * a.dt_stride + h]) + bias);
-    float2 c = make_float2(-rate * dt, 0.f);
+  float dt[2];
+  float2 c[2];
 #pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-      float2 p = make_float2(__shfl_up_sync(0xffffffffu, c.x, o), __shfl_up_sync(0xffffffffu, c.y, o));
-      if (lane >= o) c = pair_add(c, p);
+  for (int i = 0; i < 2; ++i) {
+    const int s = lane + 32 * i;
+    dt[i] = s < len ? softplusf_(to_f(((const bf16*)a.dt)[(size_t)(row0 + s) * a.dt_stride + h]) + bias) : 0.f;
+    c[i] = make_float2(-rate * dt[i], 0.f);
+  }
+#pragma unroll
+  for (int k = 1; k < 32; k <<= 1)
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      float2 p = make_float2(__shfl_up_sync(0xffffffffu, c[i].x, k), __shfl_up_sync(0xffffffffu, c[i].y, k));
+      if (lane >= k) c[i] = pair_add(c[i], p);
     }
-    c = pair_add(carry, c);
-    dts[s] = dt;
-    cum[s] = c;
-    carry = make_float2(__shfl_sync(0xffffffffu, c.x, 31), __shfl_sync(0xffffffffu, c.y, 31));
+  c[1] = pair_add(make_float2(__shfl_sync(0xffffffffu, c[0].x, 31), __shfl_sync(0xffffffffu, c[0].y, 31)), c[1]);
+  const float2 last = make_float2(__shfl_sync(0xffffffffu, c[1].x, 31), __shfl_sync(0xffffffffu, c[1].y, 31));
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int s = lane + 32 * i;
+    if (s < len) a.dec[(size_t)h * a.tokens + row0 + s] = make_float4(c[i].x, c[i].y, dt[i], dt[i] * expf(pair_diff(last, c[i])));
   }
 }
 
@@ -137,188 +150,195 @@ __device__ __forceinline__ void stage(bf16* dst, int ld, const bf16* src, long l
   }
 }
 
-// U = sum_s B_s (w_s x_s)^T, w_s = exp(c_last - c_s) dt_s.  Block = (chunk, head), 4 warps; warp w owns the state rows of
-// the 16-row tiles w, w + 4, ..; value columns in tiles of 64, the weighted x as number plus remainder.
-template <int CL>
-__global__ void __launch_bounds__(128) ssd_chunk_state_kernel(SsdArgs a, int vec) {
+// Block = (sequence, head, 32 value columns), 8 warps: warp w owns the state rows of the 16-row tiles w, w + 8, .. as
+// accumulators in registers.  A step takes in 64 tokens; its rows arrive by asynchronous copies two steps ahead.
+#define SW_TH 256
+#define SW_VT 32
+#define SW_STAGES 3
+template <int MT>
+__global__ void __launch_bounds__(SW_TH) ssd_walk_kernel(SsdArgs a, int vec) {
   extern __shared__ __align__(16) unsigned char raw[];
-  __shared__ float dts[CL];
-  __shared__ float2 cum[CL];
-  const int N = a.N, V = a.V, Np = (N + 15) & ~15, ldn = Np + 8, ldv = 64 + 8;
-  bf16* bs = reinterpret_cast<bf16*>(raw);  // [CL][ldn]
-  bf16* xh = bs + CL * ldn;                 // [CL][ldv]
-  bf16* xl = xh + CL * ldv;                 // [CL][ldv]
-  const int* c = a.ctab + 4 * blockIdx.x;
-  const int row0 = c[0], len = c[1], h = blockIdx.y, g = h / (a.H / a.G);
+  __shared__ __align__(16) float4 dec[SW_STAGES][SW_L];
+  const int N = a.N, V = a.V, Np = (N + 15) & ~15, ldn = Np + 8;
+  constexpr int ldv = SW_VT + 8;
+  bf16* bs = reinterpret_cast<bf16*>(raw);       // [SW_STAGES][SW_L][ldn]
+  bf16* xs = bs + SW_STAGES * SW_L * ldn;        // [SW_STAGES][SW_L][ldv]
+  const int* m = a.meta + 4 * blockIdx.x;
+  const int first = m[0], n = m[1], h = blockIdx.y, g = h / (a.H / a.G), v0 = blockIdx.z * SW_VT;
+  const int cols = min(SW_VT, V - v0);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gr = lane >> 2, t2 = (lane & 3) * 2;
-  const bf16* base = (const bf16*)a.xbc + (size_t)row0 * a.xbc_stride;
-  stage<128>(bs, ldn, base + (size_t)a.H * V + (size_t)g * N, a.xbc_stride, CL, len, N, Np, vec);
-  cp_commit();
-  if (warp == 0) chunk_decays<CL>(a, row0, len, h, lane, dts, cum);
-  __syncthreads();
-  if (tid == 0) a.decay[(size_t)blockIdx.x * a.H + h] = expf(cum[CL - 1].x + cum[CL - 1].y);
-  for (int s = tid; s < CL; s += 128) dts[s] *= expf(pair_diff(cum[CL - 1], cum[s]));
-  float* up = a.u + ((size_t)blockIdx.x * a.H + h) * N * V;
-  for (int v0 = 0; v0 < V; v0 += 64) {
-    const int cols = min(64, V - v0), colsp = (cols + 15) & ~15;
-    __syncthreads();  // weights are final; the tile before is done with xh, xl
-    if (vec) {
-      const int per = colsp >> 3;
-      for (int i = tid; i < CL * per; i += 128) {
-        int s = i / per, cc = (i - s * per) * 8;
-        float f[8], lo[8];
-        if (s < len && cc < cols) {
-          load8(base + (size_t)s * a.xbc_stride + (size_t)h * V + v0 + cc, f);
-        } else {
-#pragma unroll
-          for (int e = 0; e < 8; ++e) f[e] = 0.f;
-        }
-        const float w = dts[s];
-#pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          f[e] *= w;
-          lo[e] = f[e] - __bfloat162float(__float2bfloat16_rn(f[e]));
-        }
-        store8(xh + s * ldv + cc, f);
-        store8(xl + s * ldv + cc, lo);
-      }
-    } else {
-      for (int i = tid; i < CL * colsp; i += 128) {
-        int s = i / colsp, cc = i - s * colsp;
-        float f = s < len && cc < cols ? dts[s] * to_f(base[(size_t)s * a.xbc_stride + (size_t)h * V + v0 + cc]) : 0.f;
-        bf16 hi = __float2bfloat16_rn(f);
-        xh[s * ldv + cc] = hi;
-        xl[s * ldv + cc] = __float2bfloat16_rn(f - __bfloat162float(hi));
+  float* sp = a.state + ((size_t)m[2] * a.H + h) * N * V + v0;
+  bf16* out = (bf16*)a.before + ((size_t)a.stab[2 * blockIdx.x] * a.H + h) * 2 * N * V + v0;
+  auto fetch = [&](int c, int buf) {
+    if (c < n) {
+      const bf16* base = (const bf16*)a.xbc + (size_t)(first + c) * a.xbc_stride;
+      const int len = min(SW_L, n - c);
+      stage<SW_TH>(bs + buf * SW_L * ldn, ldn, base + (size_t)a.H * V + (size_t)g * N, a.xbc_stride, SW_L, len, N, Np, vec);
+      stage<SW_TH>(xs + buf * SW_L * ldv, ldv, base + (size_t)h * V + v0, a.xbc_stride, SW_L, len, cols, SW_VT, vec);
+      if (tid < SW_L) {
+        const float4* src = a.dec + (size_t)h * a.tokens + first + c;
+        cp16(reinterpret_cast<bf16*>(&dec[buf][tid]), reinterpret_cast<const bf16*>(src + (tid < len ? tid : 0)), tid < len);
       }
     }
-    cp_wait<0>();
+    cp_commit();  // possibly an empty group: the wait below counts groups
+  };
+  float S[MT][SW_VT / 8][4];
+  fetch(0, 0);
+  fetch(SW_L, 1);
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int j = 0; j < SW_VT / 8; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int d = (warp + 8 * i) * 16 + gr + 8 * (e >> 1), c = j * 8 + t2 + (e & 1);
+        S[i][j][e] = d < N && c < cols ? sp[(size_t)d * V + c] : 0.f;
+      }
+  int buf = 0;
+  for (int c0 = 0; c0 < n; c0 += SW_L, buf = buf == SW_STAGES - 1 ? 0 : buf + 1) {
+    const int len = min(SW_L, n - c0);
+    cp_wait<1>();
     __syncthreads();
-    const int nv = colsp >> 4;
-    for (int d0 = warp * 16; d0 < Np; d0 += 64) {
-      float acc[8][4];
+    fetch(c0 + 2 * SW_L, buf == 0 ? SW_STAGES - 1 : buf - 1);
+    const float4* dk = dec[buf];
+    const bf16* bb = bs + buf * SW_L * ldn;
+    const bf16* xb = xs + buf * SW_L * ldv;
+    if (c0 % SSD_CL == 0) {  // the state before this chunk of the outputs
+      bf16* hi = out + (size_t)(c0 / SSD_CL) * a.H * 2 * N * V;
 #pragma unroll
-      for (int i = 0; i < 8; ++i)
+      for (int i = 0; i < MT; ++i)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
+        for (int j = 0; j < SW_VT / 8; ++j)
 #pragma unroll
-      for (int k = 0; k < CL; k += 16) {
-        uint32_t A[4];  // A[d][s] = B[s][d]: transposed 8x8 blocks (d 0-7 | 8-15) x (s 0-7 | 8-15)
-        ldm4t(A, bs + (k + (lane & 7) + (lane >> 4) * 8) * ldn + d0 + ((lane >> 3) & 1) * 8);
-#pragma unroll
-        for (int i = 0; i < 4; ++i)
-          if (i < nv) {
-            uint32_t b[4];
-            ldm4t(b, xh + (k + (lane & 15)) * ldv + i * 16 + (lane >> 4) * 8);
-            mma(acc[2 * i], A, b);
-            mma(acc[2 * i + 1], A, b + 2);
-            ldm4t(b, xl + (k + (lane & 15)) * ldv + i * 16 + (lane >> 4) * 8);
-            mma(acc[2 * i], A, b);
-            mma(acc[2 * i + 1], A, b + 2);
+          for (int r = 0; r < 2; ++r) {
+            const int d = (warp + 8 * i) * 16 + gr + 8 * r, c = j * 8 + t2;
+            if (d >= N || c >= cols) continue;
+            uint32_t x, y;
+            split2(S[i][j][2 * r], S[i][j][2 * r + 1], x, y);
+            bf16* p = hi + (size_t)d * V + c;
+            if (vec) {
+              *reinterpret_cast<uint32_t*>(p) = x;
+              *reinterpret_cast<uint32_t*>(p + (size_t)N * V) = y;
+            } else {
+              const __nv_bfloat162 px = *reinterpret_cast<__nv_bfloat162*>(&x), py = *reinterpret_cast<__nv_bfloat162*>(&y);
+              p[0] = px.x;
+              p[(size_t)N * V] = py.x;
+              if (c + 1 < cols) { p[1] = px.y; p[(size_t)N * V + 1] = py.y; }
+            }
           }
-      }
-#pragma unroll
-      for (int i = 0; i < 8; ++i)
-#pragma unroll
-        for (int r = 0; r < 2; ++r) {
-          int d = d0 + gr + 8 * r, cc = i * 8 + t2;
-          if (d >= N || cc >= cols) continue;
-          float* p = up + (size_t)d * V + v0 + cc;
-          if (vec) {
-            *reinterpret_cast<float2*>(p) = make_float2(acc[i][2 * r], acc[i][2 * r + 1]);
-          } else {
-            p[0] = acc[i][2 * r];
-            if (cc + 1 < cols) p[1] = acc[i][2 * r + 1];
-          }
-        }
     }
-  }
-}
-
-// Walks a sequence's chunks: before[c] = S (number and remainder), S = decay_c S + U_c; the slot keeps the final S.
-// VEC neighbouring elements of the [N, V] state per thread, the U of eight chunks in flight.
-template <int VEC>
-__global__ void __launch_bounds__(256) ssd_chunk_scan_kernel(SsdArgs a) {
-  const int seq = blockIdx.x, h = blockIdx.y, NV = a.N * a.V;
-  const int slot = a.meta[4 * seq + 2], c0 = a.stab[2 * seq], nc = a.stab[2 * seq + 1];
-  const int e = (blockIdx.z * 256 + threadIdx.x) * VEC;
-  if (e >= NV) return;
-  float* sp = a.state + ((size_t)slot * a.H + h) * NV + e;
-  const float* u = a.u + ((size_t)c0 * a.H + h) * NV + e;
-  bf16* bf = (bf16*)a.before + ((size_t)c0 * a.H + h) * 2 * NV + e;
-  const float* dc = a.decay + (size_t)c0 * a.H + h;
-  const size_t cs = (size_t)a.H * NV;
-  float S[VEC];
+    const float all = expf(dk[len - 1].x + dk[len - 1].y);
 #pragma unroll
-  for (int k = 0; k < VEC; ++k) S[k] = sp[k];
-  for (int c = 0; c < nc; c += 8) {
-    float U[8][VEC], D[8];
+    for (int i = 0; i < MT; ++i)
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      const bool ok = c + i < nc;
-      D[i] = ok ? dc[(size_t)(c + i) * a.H] : 0.f;
-      if (VEC == 4) {
-        float4 f = ok ? *reinterpret_cast<const float4*>(u + (size_t)(c + i) * cs) : make_float4(0.f, 0.f, 0.f, 0.f);
-        U[i][0] = f.x; U[i][1] = f.y; U[i][2] = f.z; U[i][3] = f.w;
-      } else {
-        U[i][0] = ok ? u[(size_t)(c + i) * cs] : 0.f;
-      }
-    }
+      for (int j = 0; j < SW_VT / 8; ++j)
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      if (c + i < nc) {
-        bf16* b = bf + (size_t)(c + i) * 2 * cs;
-        if (VEC == 4) {
-          uint32_t h0, l0, h1, l1;
-          split2(S[0], S[1], h0, l0);
-          split2(S[2], S[3], h1, l1);
-          *reinterpret_cast<uint2*>(b) = make_uint2(h0, h1);
-          *reinterpret_cast<uint2*>(b + NV) = make_uint2(l0, l1);
-        } else {
-          bf16 hi = __float2bfloat16_rn(S[0]);
-          b[0] = hi;
-          b[NV] = __float2bfloat16_rn(S[0] - __bfloat162float(hi));
+        for (int e = 0; e < 4; ++e) S[i][j][e] *= all;
+#pragma unroll
+    for (int k = 0; k < SW_L; k += 16) {
+      if (k >= len) break;
+      const float w[4] = {dk[k + t2].w, dk[k + t2 + 1].w, dk[k + 8 + t2].w, dk[k + 8 + t2 + 1].w};
+      uint32_t b[SW_VT / 16][4];
+#pragma unroll
+      for (int j = 0; j < SW_VT / 16; ++j) ldm4t(b[j], xb + (k + (lane & 15)) * ldv + (lane >> 4) * 8 + j * 16);
+#pragma unroll
+      for (int i = 0; i < MT; ++i) {
+        const int d0 = (warp + 8 * i) * 16;
+        if (d0 >= Np) continue;
+        uint32_t A[4], ah[4], al[4];  // A[d][s] = B[s][d]: transposed 8x8 blocks (d 0-7 | 8-15) x (s 0-7 | 8-15)
+        ldm4t(A, bb + (k + (lane & 7) + (lane >> 4) * 8) * ldn + d0 + ((lane >> 3) & 1) * 8);
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          split2(__uint_as_float(A[e] << 16) * w[(e >> 1) * 2], __uint_as_float(A[e] & 0xffff0000u) * w[(e >> 1) * 2 + 1], ah[e], al[e]);
+#pragma unroll
+        for (int j = 0; j < SW_VT / 16; ++j) {
+          mma(S[i][2 * j], ah, b[j]);
+          mma(S[i][2 * j + 1], ah, b[j] + 2);
         }
 #pragma unroll
-        for (int k = 0; k < VEC; ++k) S[k] = D[i] * S[k] + U[i][k];
+        for (int j = 0; j < SW_VT / 16; ++j) {
+          mma(S[i][2 * j], al, b[j]);
+          mma(S[i][2 * j + 1], al, b[j] + 2);
+        }
       }
     }
   }
 #pragma unroll
-  for (int k = 0; k < VEC; ++k) sp[k] = S[k];
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int j = 0; j < SW_VT / 8; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int d = (warp + 8 * i) * 16 + gr + 8 * (e >> 1), c = j * 8 + t2 + (e & 1);
+        if (d < N && c < cols) sp[(size_t)d * V + c] = S[i][j][e];
+      }
 }
 
-// y of a chunk.  Block = (chunk, head), CL / 16 warps of 16 token rows; value columns in tiles of 64.  Per row: first the
-// read-out of the state before the chunk, scaled by exp(c_t), then tile by tile of 16 earlier tokens the products C.B,
-// weighed in registers and multiplied into x.
-template <int CL>
-__global__ void __launch_bounds__(2 * CL) ssd_chunk_out_kernel(SsdArgs a, int vec) {
-  constexpr int TH = 2 * CL;
+// y of a chunk.  Block = (chunk, head), 8 warps of 16 token rows; value columns in tiles of 64.  C stays in registers as
+// left operand (NK: 16-wide steps of the state size).  Per row: the read-out of the state before the chunk, scaled by exp(c_t), then
+// by 16 earlier tokens the products C.B, weighed in registers and multiplied into x.
+template <int NK>
+__global__ void __launch_bounds__(2 * SSD_CL) ssd_out_kernel(SsdArgs a, int vec) {
+  constexpr int TH = 2 * SSD_CL, ldv = 64 + 8;
   extern __shared__ __align__(16) unsigned char raw[];
-  __shared__ float dts[CL];
-  __shared__ float2 cum[CL];
-  const int N = a.N, V = a.V, Np = (N + 15) & ~15, ldn = Np + 8, ldv = 64 + 8;
-  bf16* cm = reinterpret_cast<bf16*>(raw);  // [CL][ldn]
-  bf16* bs = cm + CL * ldn;                 // [CL][ldn]
-  bf16* xs = bs + CL * ldn;                 // [CL][ldv]
-  bf16* sh = xs + CL * ldv;                 // [Np][ldv]
+  __shared__ float2 cum[SSD_CL];
+  __shared__ float dts[SSD_CL];
+  const int N = a.N, V = a.V, Np = (N + 15) & ~15, ldn = Np + 8;
+  bf16* bs = reinterpret_cast<bf16*>(raw);  // [CL][ldn]
+  bf16* xs = bs + SSD_CL * ldn;             // [CL][ldv]
+  bf16* sh = xs + SSD_CL * ldv;             // [Np][ldv]
   bf16* sl = sh + Np * ldv;                 // [Np][ldv]
   const int* c = a.ctab + 4 * blockIdx.x;
   const int row0 = c[0], len = c[1], h = blockIdx.y, g = h / (a.H / a.G);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gr = lane >> 2, t2 = (lane & 3) * 2;
   const bf16* base = (const bf16*)a.xbc + (size_t)row0 * a.xbc_stride;
   const bf16* before = (const bf16*)a.before + ((size_t)blockIdx.x * a.H + h) * 2 * N * V;
-  stage<TH>(cm, ldn, base + (size_t)a.H * V + (size_t)(a.G + g) * N, a.xbc_stride, CL, len, N, Np, vec);
-  stage<TH>(bs, ldn, base + (size_t)a.H * V + (size_t)g * N, a.xbc_stride, CL, len, N, Np, vec);
+  stage<TH>(bs, ldn, base + (size_t)a.H * V + (size_t)g * N, a.xbc_stride, SSD_CL, len, N, Np, vec);
   const int r0 = warp * 16;  // this lane's rows: r0 + gr and r0 + gr + 8
+  uint32_t C[NK][4];
+  {
+    const bf16* cp = base + (size_t)a.H * V + (size_t)(a.G + g) * N;
+#pragma unroll
+    for (int k = 0; k < NK; ++k)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int row = r0 + gr + (e & 1) * 8, col = k * 16 + t2 + (e >> 1) * 8;
+        C[k][e] = 0;
+        if (row < len && col < N) {
+          const bf16* p = cp + (size_t)row * a.xbc_stride + col;
+          if (vec) {
+            C[k][e] = *reinterpret_cast<const uint32_t*>(p);
+          } else {
+            __nv_bfloat162 v = __halves2bfloat162(p[0], col + 1 < N ? p[1] : __float2bfloat16_rn(0.f));
+            C[k][e] = *reinterpret_cast<uint32_t*>(&v);
+          }
+        }
+      }
+  }
+  for (int s = tid; s < SSD_CL; s += TH) {
+    float4 d = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (s < len) {
+      const float4* dp = a.dec + (size_t)h * a.tokens + row0;
+      d = dp[s];
+      if (s >= SW_L) {  // the sums start over after 64 tokens
+        float4 o = dp[SW_L - 1];
+        float2 t = pair_add(make_float2(o.x, o.y), make_float2(d.x, d.y));
+        d.x = t.x;
+        d.y = t.y;
+      }
+    }
+    cum[s] = make_float2(d.x, d.y);
+    dts[s] = d.z;
+  }
   const float skip = a.d[h];
+  const int sv = (lane & 15) * ldv + (lane >> 4) * 8;
   for (int v0 = 0; v0 < V; v0 += 64) {
     const int cols = min(64, V - v0), colsp = (cols + 15) & ~15, nv = colsp >> 4;
-    __syncthreads();  // the tile before is done with xs, sh, sl
-    stage<TH>(xs, ldv, base + (size_t)h * V + v0, a.xbc_stride, CL, len, cols, colsp, vec);
+    if (v0) __syncthreads();  // the tile before is done with xs, sh, sl
+    stage<TH>(xs, ldv, base + (size_t)h * V + v0, a.xbc_stride, SSD_CL, len, cols, colsp, vec);
     stage<TH>(sh, ldv, before + v0, V, Np, N, cols, colsp, vec);
     stage<TH>(sl, ldv, before + (size_t)N * V + v0, V, Np, N, cols, colsp, vec);
     cp_commit();
-    if (v0 == 0 && warp == 0) chunk_decays<CL>(a, row0, len, h, lane, dts, cum);
     cp_wait<0>();
     __syncthreads();
     if (r0 < len) {
@@ -327,19 +347,19 @@ __global__ void __launch_bounds__(2 * CL) ssd_chunk_out_kernel(SsdArgs a, int ve
       for (int i = 0; i < 8; ++i)
 #pragma unroll
         for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
-      const bf16* ap = cm + (r0 + (lane & 15)) * ldn + (lane >> 4) * 8;
-      for (int k = 0; k < Np; k += 16) {
-        uint32_t A[4], b[4];
-        ldm4(A, ap + k);
+#pragma unroll
+      for (int k = 0; k < NK; ++k) {
+        if (k * 16 >= Np) break;
 #pragma unroll
         for (int i = 0; i < 4; ++i)
           if (i < nv) {
-            ldm4t(b, sh + (k + (lane & 15)) * ldv + i * 16 + (lane >> 4) * 8);
-            mma(acc[2 * i], A, b);
-            mma(acc[2 * i + 1], A, b + 2);
-            ldm4t(b, sl + (k + (lane & 15)) * ldv + i * 16 + (lane >> 4) * 8);
-            mma(acc[2 * i], A, b);
-            mma(acc[2 * i + 1], A, b + 2);
+            uint32_t b[4], d[4];
+            ldm4t(b, sh + k * 16 * ldv + sv + i * 16);
+            ldm4t(d, sl + k * 16 * ldv + sv + i * 16);
+            mma(acc[2 * i], C[k], b);
+            mma(acc[2 * i + 1], C[k], b + 2);
+            mma(acc[2 * i], C[k], d);
+            mma(acc[2 * i + 1], C[k], d + 2);
           }
       }
       const float2 ct[2] = {cum[r0 + gr], cum[r0 + gr + 8]};
@@ -353,31 +373,31 @@ __global__ void __launch_bounds__(2 * CL) ssd_chunk_out_kernel(SsdArgs a, int ve
 #pragma unroll
           for (int e = 0; e < 4; ++e) s[i][e] = 0.f;
         const bf16* bp = bs + (s0 + (lane & 7) + (lane >> 4) * 8) * ldn + ((lane >> 3) & 1) * 8;
-#pragma unroll 4
-        for (int k = 0; k < Np; k += 16) {
-          uint32_t A[4], b[4];
-          ldm4(A, ap + k);
-          ldm4(b, bp + k);
-          mma(s[0], A, b);
-          mma(s[1], A, b + 2);
+#pragma unroll
+        for (int k = 0; k < NK; ++k) {
+          if (k * 16 >= Np) break;
+          uint32_t b[4];
+          ldm4(b, bp + k * 16);
+          mma(s[0], C[k], b);
+          mma(s[1], C[k], b + 2);
         }
         uint32_t hi[4], lo[4];
 #pragma unroll
         for (int u = 0; u < 2; ++u) {
+          const int src = s0 + u * 8 + t2;
+          const float2 cs[2] = {cum[src], cum[src + 1]};
+          const float w[2] = {dts[src], dts[src + 1]};
 #pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const int src = s0 + u * 8 + t2 + (e & 1), row = r0 + gr + (e >> 1) * 8;
-            s[u][e] = src <= row ? s[u][e] * (dts[src] * expf(pair_diff(ct[e >> 1], cum[src]))) : 0.f;
-          }
+          for (int e = 0; e < 4; ++e)
+            s[u][e] = src + (e & 1) <= r0 + gr + (e >> 1) * 8 ? s[u][e] * (w[e & 1] * expf(pair_diff(ct[e >> 1], cs[e & 1]))) : 0.f;
           split2(s[u][0], s[u][1], hi[2 * u], lo[2 * u]);
           split2(s[u][2], s[u][3], hi[2 * u + 1], lo[2 * u + 1]);
         }
-        const bf16* xp = xs + (s0 + (lane & 15)) * ldv + (lane >> 4) * 8;
 #pragma unroll
         for (int i = 0; i < 4; ++i)
           if (i < nv) {
             uint32_t b[4];
-            ldm4t(b, xp + i * 16);
+            ldm4t(b, xs + s0 * ldv + sv + i * 16);
             mma(acc[2 * i], hi, b);
             mma(acc[2 * i + 1], hi, b + 2);
             mma(acc[2 * i], lo, b);
@@ -424,7 +444,7 @@ __global__ void silu_gate_norm_kernel(const float* __restrict__ y, const T* __re
     else { f[0] = yr[i]; g[0] = to_f(zr[i]); }
 #pragma unroll
     for (int e = 0; e < VEC; ++e) {
-      f[e] *= siluf_(g[e]);
+      f[e] *= silu_as<T>(g[e]);
       ss += f[e] * f[e];
     }
     if (VEC == 8) store8(buf + i, f);
@@ -462,32 +482,27 @@ int hyb_ssd_scan(const SsdArgs* args, int dt, cudaStream_t st) {
   return (int)cudaGetLastError();
 }
 
-// Shared memory of the output kernel for chunks of `cl` tokens (the largest of the three); 0: no such kernel.
-static size_t ssd_out_smem(int cl, int N) {
-  size_t Np = (size_t)((N + 15) & ~15);
-  return (2 * cl * (Np + 8) + (size_t)cl * 72 + 2 * Np * 72) * sizeof(bf16);
-}
-
-// The chunked form (bf16): -3 when the shared memory of a block does not hold the shape.
-int hyb_ssd_chunked(const SsdArgs* args, int cl, cudaStream_t st) {
+// The chunked form (bf16), three launches.  -3: more than 256 state rows.
+int hyb_ssd_chunked(const SsdArgs* args, cudaStream_t st) {
   const SsdArgs& a = *args;
   if (a.nseq == 0) return 0;
-  if (a.G < 1 || a.H % a.G || a.N < 1 || a.V < 1 || (cl != 64 && cl != 128)) return -2;
-  const size_t so = ssd_out_smem(cl, a.N), ss = ((size_t)cl * (((a.N + 15) & ~15) + 8) + 2 * (size_t)cl * 72) * sizeof(bf16);
-  if (so > 200 * 1024 || ss > 200 * 1024 || a.H > 65535) return -3;
-  const uintptr_t bits = (uintptr_t)a.xbc | (uintptr_t)a.u | (uintptr_t)a.before | (uintptr_t)a.y | (uintptr_t)a.state;
+  if (a.G < 1 || a.H % a.G || a.N < 1 || a.V < 1) return -2;
+  if (a.N > 256 || a.H > 65535) return -3;
+  const size_t Np = (size_t)((a.N + 15) & ~15);
+  const size_t sw = SW_STAGES * SW_L * (Np + 8 + SW_VT + 8) * sizeof(bf16);
+  const size_t so = (SSD_CL * (Np + 8) + SSD_CL * 72 + 2 * Np * 72) * sizeof(bf16);
+  const uintptr_t bits = (uintptr_t)a.xbc | (uintptr_t)a.y | (uintptr_t)a.before | (uintptr_t)a.dec;
   const int vec = (bits & 15) == 0 && ((a.N | a.V) & 7) == 0 && (a.xbc_stride & 7) == 0;
-  dim3 grid(a.nchunks, a.H);
-#define CK(CL)                                                                                                        \
-  do {                                                                                                                \
-    cudaFuncSetAttribute(ssd_chunk_state_kernel<CL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ss);           \
-    cudaFuncSetAttribute(ssd_chunk_out_kernel<CL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)so);             \
-    ssd_chunk_state_kernel<CL><<<grid, 128, ss, st>>>(a, vec);                                                        \
-    if (vec) ssd_chunk_scan_kernel<4><<<dim3(a.nseq, a.H, (a.N * a.V + 1023) / 1024), 256, 0, st>>>(a);               \
-    else ssd_chunk_scan_kernel<1><<<dim3(a.nseq, a.H, (a.N * a.V + 255) / 256), 256, 0, st>>>(a);                     \
-    ssd_chunk_out_kernel<CL><<<grid, 2 * CL, so, st>>>(a, vec);                                                       \
+  dim3 wgrid(a.nseq, a.H, (a.V + SW_VT - 1) / SW_VT), ogrid(a.nchunks, a.H);
+#define CK(MT, NK)                                                                                          \
+  do {                                                                                                      \
+    cudaFuncSetAttribute(ssd_walk_kernel<MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sw);        \
+    cudaFuncSetAttribute(ssd_out_kernel<NK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)so);         \
+    ssd_decay_kernel<<<dim3(a.nchunks, (a.H + 3) / 4), 256, 0, st>>>(a);                                    \
+    ssd_walk_kernel<MT><<<wgrid, SW_TH, sw, st>>>(a, vec);                                                  \
+    ssd_out_kernel<NK><<<ogrid, 2 * SSD_CL, so, st>>>(a, vec);                                              \
   } while (0)
-  if (cl == 64) CK(64); else CK(128);
+  if (a.N <= 64) CK(1, 4); else if (a.N <= 128) CK(1, 8); else CK(2, 16);
 #undef CK
   return (int)cudaGetLastError();
 }

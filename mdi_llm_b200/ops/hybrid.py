@@ -57,9 +57,9 @@ class _RowUpdateArgs(ctypes.Structure):
 
 
 class _SsdArgs(ctypes.Structure):
-    _fields_ = ([(n, c_void_p) for n in ("xbc", "dt", "dt_bias", "a_log", "d", "state", "y", "meta", "ctab", "stab", "u", "decay", "before")]
+    _fields_ = ([(n, c_void_p) for n in ("xbc", "dt", "dt_bias", "a_log", "d", "state", "y", "meta", "ctab", "stab", "before", "dec")]
                 + [(n, c_longlong) for n in ("xbc_stride", "dt_stride")]
-                + [(n, c_int) for n in ("H", "G", "N", "V", "nseq", "nchunks")])
+                + [(n, c_int) for n in ("H", "G", "N", "V", "nseq", "nchunks", "tokens")])
 
 
 def lib() -> ctypes.CDLL:
@@ -81,6 +81,7 @@ def lib() -> ctypes.CDLL:
     h.hyb_gelu_rows.argtypes = [vp, i64, i32, i32, vp]
     h.hyb_window_append.argtypes = [vp, i64, vp, i64, vp, i64, vp, vp, i64, vp, vp, i32, i32, i32, i32, i32, i32, f32, vp, vp, vp, i64, vp, i32, i32, f32, i32, vp]
     h.hyb_window_attn.argtypes = [vp, i64, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, i32, vp, vp, i32, i32, i32, f32, vp, i32, vp]
+    h.hyb_grouped_decode_mma.argtypes = [vp, i64, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, i32, vp, vp, i32, i32, i32, f32, vp, vp]
     h.hyb_head_gate.argtypes = [vp, vp, i64, vp, i32, i32, i32, i32, vp]
     h.hyb_token_side_gate.argtypes = [vp, i64, vp, i64, i32, vp, vp, i32, i32, i32, vp]
     h.hyb_router_topk.argtypes = [vp, vp, vp, i32, i32, i32, i32, vp, vp]
@@ -98,7 +99,7 @@ def lib() -> ctypes.CDLL:
     h.hyb_latent_decode_mma.argtypes = [vp, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, vp, vp, i32, vp, i32, i32, f32, vp, vp]
     h.hyb_prompt_attn_mma.argtypes = [vp, i64, vp, i64, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, i32, i32, vp, vp, i64, vp]
     h.hyb_ssd_scan.argtypes = [ctypes.POINTER(_SsdArgs), i32, vp]
-    h.hyb_ssd_chunked.argtypes = [ctypes.POINTER(_SsdArgs), i32, vp]
+    h.hyb_ssd_chunked.argtypes = [ctypes.POINTER(_SsdArgs), vp]
     h.hyb_silu_gate_norm.argtypes = [vp, vp, i64, vp, vp, i32, i32, i32, f32, i32, vp]
     h.hyb_row_update.argtypes = [ctypes.POINTER(_RowUpdateArgs), i32, vp]
     h.hyb_norm_conv.argtypes = [vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, i32, i32, vp]
@@ -695,7 +696,7 @@ def visible_from(pos: torch.Tensor, window: int, mask: str) -> torch.Tensor:
 
 def window_attn(q: torch.Tensor, g: Optional[torch.Tensor], cache: torch.Tensor, plan: BatchPlan, H: int, G: int, D: int,
                 V: int, scale: float, window: int, split: int = 0, mask: str = "window", sink: bool = False,
-                cap: float = 0.0, sink_vals: Optional[torch.Tensor] = None) -> torch.Tensor:
+                cap: float = 0.0, sink_vals: Optional[torch.Tensor] = None, mma: bool = True) -> torch.Tensor:
     """Softmax attention of every token over the cached keys of its slot that are not later than it and (``window > 0``)
     fewer than ``window`` positions back; query head ``h`` reads key/value head ``h // (H/G)``.  Each head's output is
     multiplied by ``sigmoid(g[token, h])`` when ``g [N, H]`` is given, or channel by channel by ``sigmoid(g)`` for
@@ -705,7 +706,8 @@ def window_attn(q: torch.Tensor, g: Optional[torch.Tensor], cache: torch.Tensor,
     ``s`` becomes ``cap * tanh(s / cap)``.  Returns ``[N, H*V]``.  The form for one-token steps and
     short portions: one block per token and key/value head, the cache tile shared by the group's query heads.
     ``split`` (CUDA): key shares per token, 0 = chosen from the batch shape and the window alone, so that a captured
-    step stays valid while contexts grow."""
+    step stays valid while contexts grow.  With bf16 activations and ``D``, ``V`` multiples of 16 (at most 256) the products run
+    on the tensor cores (weights as a bf16 number plus its bf16 remainder); else, or with ``mma=False``, on fp32 values."""
     N = q.size(0)
     if not q.is_cuda:
         out = torch.empty(N, H * V, dtype=q.dtype)
@@ -738,6 +740,23 @@ def window_attn(q: torch.Tensor, g: Optional[torch.Tensor], cache: torch.Tensor,
         raise HybridOpsError("sink scores are dense fp32, one per head")
     gate_mode = 0 if g is None else (1 if g.size(1) == H else 2)
     out = torch.empty(N, H * V, device=q.device, dtype=q.dtype)
+    mma = mma and q.dtype == torch.bfloat16 and D % 16 == 0 and V % 16 == 0 and max(D, V) <= 256 and q.stride(0) % 8 == 0 \
+        and cache.stride(0) % 8 == 0 and (q.data_ptr() | cache.data_ptr()) % 16 == 0
+    if mma:
+        blocks = N * G * ((H // G + 15) // 16)
+        most = min(32, (window + 63) // 64 if window > 0 else 32)
+        nsplit = min(32, split) or max(1, min(most, 2 * _SM_TARGET // blocks))
+        pa = pm = None
+        if nsplit > 1:
+            pa = torch.empty(nsplit, N, H, V, device=q.device, dtype=torch.float32)
+            pm = torch.empty(nsplit, N, H, 2, device=q.device, dtype=torch.float32)
+        _check(lib().hyb_grouped_decode_mma(q.data_ptr(), _rows(q)[0], None if g is None else g.data_ptr(), 0 if g is None else _rows(g)[0],
+                                            cache.data_ptr(), cache.stride(0), plan.meta.data_ptr(), plan.tok_seq.data_ptr(), out.data_ptr(),
+                                            N, H, G, D, V, float(scale), int(window), nsplit, None if pa is None else pa.data_ptr(),
+                                            None if pm is None else pm.data_ptr(), _MASK_KINDS[mask if window > 0 else "window"],
+                                            int(bool(sink)), gate_mode, float(cap), None if sink_vals is None else sink_vals.data_ptr(), _st()),
+               "grouped_decode_mma")
+        return out
     blocks = N * G
     tiles = (window + 31) // 32 if window > 0 else 16
     nsplit = min(32, split) or (1 if blocks >= 4 * _SM_TARGET else max(1, min(32, tiles, (4 * _SM_TARGET + blocks - 1) // blocks)))
@@ -1148,18 +1167,11 @@ def norm_gate_rows(o: torch.Tensor, w: torch.Tensor, g: torch.Tensor, eps: float
 
 
 ssd_chunk_from = 16  # as above, for the state-space recurrence with 16-bit activations
-ssd_chunk_len = 64   # tokens per chunk: 64 or 128
-
-
-def _ssd_chunk_smem(length: int, dim: int) -> int:
-    """Bytes of shared memory the chunked form's largest kernel needs."""
-    d = -(-dim // 16) * 16
-    return 2 * (2 * length * (d + 8) + 72 * length + 2 * 72 * d)
 
 
 def ssd_recurrence(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, d: torch.Tensor,
-                   state: torch.Tensor, plan: BatchPlan, heads: int, groups: int, dim: int, vdim: int, variant: int = 0,
-                   chunk: int = 0) -> torch.Tensor:
+                   state: torch.Tensor, plan: BatchPlan, heads: int, groups: int, dim: int, vdim: int,
+                   variant: int = 0) -> torch.Tensor:
     """State-space recurrence with one decay per head and token.  ``xbc [N, heads*vdim + 2*groups*dim]`` holds ``x | B | C``
     (already activated), ``dt [N, heads]`` the raw step sizes (a column slice), ``dt_bias``, ``a_log``, ``d`` fp32 ``[heads]``:
 
@@ -1167,8 +1179,8 @@ def ssd_recurrence(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a
 
     with ``S [dim, vdim]`` fp32 in ``state[slot, head]`` (read at the start of the step, written back at its end) and head
     ``h`` on the ``B``, ``C`` of group ``h // (heads / groups)``.  Returns fp32 ``[N, heads * vdim]``.  ``variant`` (CUDA): 1 the
-    token scan; 2 chunks of ``chunk`` (64 or 128) tokens as tensor-core products, all chunks of the step in parallel (bf16);
-    0 chooses by the longest sequence and the type."""
+    token scan; 2 chunks as tensor-core products (bf16, ``dim`` at most 256): a walk along each sequence leaves the state before
+    every chunk, the outputs of all chunks follow at once; 0 chooses by the longest sequence and the type."""
     N, H, G, D, V = xbc.size(0), heads, groups, dim, vdim
     if state.dtype != torch.float32 or dt_bias.dtype != torch.float32 or a_log.dtype != torch.float32 or d.dtype != torch.float32:
         raise HybridOpsError("recurrent state, decays and skip factors are fp32")
@@ -1188,12 +1200,8 @@ def ssd_recurrence(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a
                 out[t] = (torch.einsum("hdv,hd->hv", S, C[t]) + d[:, None] * x[t]).reshape(-1)
             state[slot] = S
         return out
-    length = int(chunk) or ssd_chunk_len
     if not variant:
-        long = max(n for _, n, _, _ in plan.seqs) >= ssd_chunk_from
-        if long and not chunk and _ssd_chunk_smem(length, D) > 200 * 1024:
-            length = 64
-        variant = 2 if long and xbc.dtype == torch.bfloat16 and _ssd_chunk_smem(length, D) <= 200 * 1024 else 1
+        variant = 2 if max(n for _, n, _, _ in plan.seqs) >= ssd_chunk_from and xbc.dtype == torch.bfloat16 and D <= 256 else 1
     if dt.dtype != xbc.dtype or not (state.is_contiguous() and dt_bias.is_contiguous() and a_log.is_contiguous() and d.is_contiguous()) \
             or dt_bias.numel() != H or a_log.numel() != H or d.numel() != H or tuple(state.shape[1:]) != (H, D, V):
         raise HybridOpsError("dt has the activation type; state and per-head numbers are dense")
@@ -1207,13 +1215,12 @@ def ssd_recurrence(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a
         return out
     if xbc.dtype != torch.bfloat16:
         raise HybridOpsError("the chunked form takes 16-bit activations")
-    ctab, stab, nchunks = _chunk_tables(plan, length, xbc.device)
-    u = torch.empty(nchunks, H, D, V, device=xbc.device, dtype=torch.float32)
+    ctab, stab, nchunks = _chunk_tables(plan, 128, xbc.device)
     before = torch.empty(nchunks, H, 2, D, V, device=xbc.device, dtype=torch.bfloat16)
-    decay = torch.empty(nchunks, H, device=xbc.device, dtype=torch.float32)
-    a.ctab, a.stab, a.nchunks = ctab.data_ptr(), stab.data_ptr(), nchunks
-    a.u, a.before, a.decay = u.data_ptr(), before.data_ptr(), decay.data_ptr()
-    _check(lib().hyb_ssd_chunked(ctypes.byref(a), length, _st()), "ssd_chunked")
+    dec = torch.empty(H, N, 4, device=xbc.device, dtype=torch.float32)
+    a.ctab, a.stab, a.nchunks, a.tokens = ctab.data_ptr(), stab.data_ptr(), nchunks, N
+    a.before, a.dec = before.data_ptr(), dec.data_ptr()
+    _check(lib().hyb_ssd_chunked(ctypes.byref(a), _st()), "ssd_chunked")
     return out
 
 

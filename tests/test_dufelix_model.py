@@ -316,11 +316,11 @@ SSD_SHAPES = [(2, 1, 5, 3), (4, 2, 16, 16), (3, 3, 24, 40), (2, 2, 128, 64), (2,
 @pytest.mark.parametrize("shape", SSD_SHAPES, ids=str)
 @pytest.mark.parametrize("speed", ["slow", "mixed", "fast"])
 def test_state_space_recurrence_in_every_form(where, dtype, shape, speed):
-    """Unequal sequences in scattered slots, the first with a state from before; the token scan, chunks of 64 and of 128.
+    """Unequal sequences in scattered slots, the first with a state from before; the token scan and the chunked form.
     ``fast``: the decay of a few tokens underflows; ``slow``: a chunk hardly decays at all."""
     Hh, G, N, V = shape
     dt_mean, a_mean = {"slow": (-3.0, -3.0), "mixed": (-1.0, 0.0), "fast": (3.0, 4.0)}[speed]
-    lengths, slots = [131, 1, 64, 17], [3, 0, 2, 4]
+    lengths, slots = [291, 1, 64, 17], [3, 0, 2, 4]
     xbc, dt, bias, a_log, d = _ssd_case(dtype, Hh, G, N, V, lengths, 5, dt_mean, a_mean)
     start = torch.zeros(6, Hh, N, V)
     start[3] = torch.randn(Hh, N, V, generator=torch.Generator().manual_seed(8))
@@ -333,14 +333,12 @@ def test_state_space_recurrence_in_every_form(where, dtype, shape, speed):
     want = torch.cat(want)
     plan = BatchPlan.make(lengths, slots, [9, 0, 0, 0], torch.device(where))
     wide = torch.cat((xbc.new_zeros(xbc.size(0), 8), dt, xbc.new_zeros(xbc.size(0), 5)), 1).to(where)
-    forms = [(0, 0)] if where == "cpu" else [(0, 0), (1, 0)] + ([(2, 64), (2, 128)] if dtype == torch.bfloat16 else [])
-    for variant, chunk in forms:
-        if variant == 2 and H._ssd_chunk_smem(chunk, N) > 200 * 1024:
-            continue
+    forms = [0] if where == "cpu" else ([0, 1, 2] if dtype == torch.bfloat16 else [0, 1])
+    for variant in forms:
         state = start.clone().to(where)
         plan.shared.clear()
         got = H.ssd_recurrence(xbc.to(where), wide[:, 8:8 + Hh], bias.to(where), a_log.to(where), d.to(where), state, plan, Hh, G, N, V,
-                               variant, chunk)
+                               variant)
         scale = max(1.0, want.abs().max().item())
         torch.testing.assert_close(got.cpu(), want, rtol=1e-4, atol=5e-5 * scale)  # whatever the activation type: the state is fp32
         torch.testing.assert_close(state[slots].cpu(), torch.stack(finals), rtol=1e-4, atol=5e-5 * max(1.0, start[3].abs().max().item(), scale))
@@ -526,7 +524,7 @@ def _plain_grouped(m, q, gate, cache, pos):
     return torch.cat(outs)
 
 
-GQA_SHAPES = [(4, 2, 10, 7), (6, 3, 32, 16), (8, 1, 64, 48), (5, 5, 16, 128), (9, 3, 128, 64)]
+GQA_SHAPES = [(4, 2, 10, 7), (6, 3, 32, 16), (20, 1, 64, 48), (5, 5, 16, 128), (9, 3, 128, 64), (2, 1, 48, 256)]
 
 
 @pytest.mark.parametrize("where", WHERE)
@@ -556,8 +554,9 @@ def test_grouped_attention_forms_on_unequal_sequences(where, dtype, shape, windo
         rows = [r0 + i for (r0, n, _, _) in plan.seqs for i in ({n - 1} if case else {0, 1, 30, 63, n - 1})]
         where_of = {r0 + i: (slot, p0 + i) for (r0, n, slot, p0) in plan.seqs for i in range(n)}
         want = torch.stack([_plain_grouped(m, q[r], gate[r], cache[where_of[r][0]], where_of[r][1]) for r in rows]).float()
-        got = H.window_attn(q, gate, cache, plan, Hh, G, D, V, m.scale, window, sink=sink is not None, sink_vals=m.sink32)
-        torch.testing.assert_close(got[rows].float().cpu(), want, **tol)
+        for split, mma in (((0, True), (1, True), (2, True), (7, True), (32, True), (0, False), (5, False)) if where == "cuda" else ((0, True),)):
+            got = H.window_attn(q, gate, cache, plan, Hh, G, D, V, m.scale, window, split, sink=sink is not None, sink_vals=m.sink32, mma=mma)
+            torch.testing.assert_close(got[rows].float().cpu(), want, **tol)
         got = H.head_gate(m._banded(q, cache, plan), gate)
         torch.testing.assert_close(got[rows].float().cpu(), want, **tol)
         if m._takes_fused(q):
@@ -565,6 +564,27 @@ def test_grouped_attention_forms_on_unequal_sequences(where, dtype, shape, windo
             torch.testing.assert_close(m._fused(q, gate, cache, plan)[rows].float().cpu(), want, **tol)
     if where == "cuda":
         assert m._takes_fused(q) == (dtype == torch.bfloat16 and shape != GQA_SHAPES[0])
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("mask,window,sink,cap,gate", [("chunk", 48, True, 0.0, "channel"), ("window", 0, "learned", 15.0, "head"),
+                                                       ("chunk", 64, "learned", 0.0, None), ("window", 20, False, 5.0, "channel")])
+def test_single_token_attention_variants_agree_with_the_fp32_form(mask, window, sink, cap, gate):
+    """The tensor-core form and the form on fp32 values, on one-token steps of unequal contexts with every mask, sink, gate and cap."""
+    Hh, G, D, V = 6, 2, 32, 48
+    g = torch.Generator().manual_seed(3)
+    starts = [0, 1, 15, 16, 47, 48, 63, 64, 127, 150]
+    n = len(starts)
+    plan = BatchPlan.make([1] * n, list(range(n)), starts, torch.device("cuda"))
+    bf = dict(device="cuda", dtype=torch.bfloat16)
+    q, cache = torch.randn(n, Hh * D, generator=g).to(**bf), torch.randn(n, 160, G * (D + V), generator=g).to(**bf)
+    gt = None if gate is None else torch.randn(n, Hh * (V if gate == "channel" else 1), generator=g).to(**bf)
+    sv = torch.randn(Hh, generator=g).cuda() if sink == "learned" else None
+    kw = dict(mask=mask, sink=bool(sink), cap=cap, sink_vals=sv)
+    for split in (0, 1, 3):
+        a = H.window_attn(q, gt, cache, plan, Hh, G, D, V, 0.3, window, split, **kw)
+        b = H.window_attn(q, gt, cache, plan, Hh, G, D, V, 0.3, window, split, mma=False, **kw)
+        torch.testing.assert_close(a.float(), b.float(), rtol=1e-2, atol=1e-2)
 
 
 # ---- whole models: prompts, decoding, portions, batches, slots ------------------------------------------------
