@@ -39,23 +39,17 @@ __global__ void __launch_bounds__(128) grouped_decode_mma_kernel(GroupedArgs a) 
   const int kb = lo + blockIdx.z * share, ke = min(pos + 1, kb + share);
   const size_t rowlen = (size_t)a.G * (D + V);
   const bf16* base = a.cache + (size_t)m[2] * a.slot_stride;
-  const int dk8 = D >> 3, v8 = V >> 3;
+  const int dk8 = D >> 3;
+  const RowCopy rk(dk8, lane, 32), rv(V >> 3, lane, 32);
   const int nt = kb < ke ? max(0, ((ke - kb + GD_KEYS - 1) / GD_KEYS - warp + 3) / 4) : 0;
   auto fetch = [&](int it) {
     if (it < nt) {
       bf16* k = ring + (it % GD_STAGES) * GD_KEYS * (ldk + ldv);
       bf16* v = k + GD_KEYS * ldk;
       const int j0 = kb + (warp + 4 * it) * GD_KEYS;
-      for (int i = lane; i < GD_KEYS * dk8; i += 32) {
-        int j = i / dk8, c = (i - j * dk8) * 8;
-        bool ok = j0 + j < ke;
-        cp16(k + j * ldk + c, base + (size_t)(ok ? j0 + j : kb) * rowlen + (size_t)g * D + c, ok);
-      }
-      for (int i = lane; i < GD_KEYS * v8; i += 32) {
-        int j = i / v8, c = (i - j * v8) * 8;
-        bool ok = j0 + j < ke;
-        cp16(v + j * ldv + c, base + (size_t)(ok ? j0 + j : kb) * rowlen + (size_t)a.G * D + (size_t)g * V + c, ok);
-      }
+      const bf16* row = base + (size_t)j0 * rowlen;
+      rk.run(k, ldk, row + (size_t)g * D, rowlen, GD_KEYS, ke - j0, D);
+      rv.run(v, ldv, row + (size_t)a.G * D + (size_t)g * V, rowlen, GD_KEYS, ke - j0, V);
     }
     cp_commit();  // possibly an empty group: the wait counts groups
   };

@@ -44,12 +44,9 @@ __global__ void __launch_bounds__(128) latent_decode_mma_kernel(const float* __r
   const int chunk = ((nkeys + nsplit - 1) / nsplit + LD_TILE - 1) / LD_TILE * LD_TILE;
   const int k_begin = blockIdx.z * chunk, k_end = min(nkeys, k_begin + chunk);
   const int per = Dk >> 3;
+  const RowCopy rc(per, tid, 128);
   auto fetch = [&](int t0, bf16* dst) {
-    for (int i = tid; i < LD_TILE * per; i += 128) {
-      int j = i / per, c = (i - j * per) * 8;
-      bool ok = t0 + j < k_end;
-      cp16(dst + j * ld + c, rows + (size_t)(ok ? t0 + j : k_begin) * Dk + c, ok);
-    }
+    rc.run(dst, ld, rows + (size_t)t0 * Dk, Dk, LD_TILE, k_end - t0, Dk);
     cp_commit();
   };
   const bool any = k_begin < k_end;
@@ -266,24 +263,13 @@ __global__ void __launch_bounds__(128) prompt_attn_mma_kernel(const bf16* __rest
   const int hk = h / (H / G);
   const bf16* kbase = kv + (size_t)hk * DK;
   const bf16* vbase = kv + (size_t)G * DK + (size_t)hk * V;
+  const RowCopy rk(dk8, tid, 128), rv(v8, tid, 128);
   auto fetch = [&](int j0, int buf) {
-    for (int i = tid; i < PA_KEYS * dk8; i += 128) {
-      int j = i / dk8, c = (i - j * dk8) * 8;
-      bool ok = j0 + j < ke;
-      cp16(ks + (buf * PA_KEYS + j) * ldk + c, kbase + (size_t)(ok ? j0 + j : kb) * kv_stride + c, ok);
-    }
-    for (int i = tid; i < PA_KEYS * v8; i += 128) {
-      int j = i / v8, c = (i - j * v8) * 8;
-      bool ok = j0 + j < ke;
-      cp16(vs + (buf * PA_KEYS + j) * ldv + c, vbase + (size_t)(ok ? j0 + j : kb) * kv_stride + c, ok);
-    }
+    rk.run(ks + buf * PA_KEYS * ldk, ldk, kbase + (size_t)j0 * kv_stride, kv_stride, PA_KEYS, ke - j0, DK);
+    rv.run(vs + buf * PA_KEYS * ldv, ldv, vbase + (size_t)j0 * kv_stride, kv_stride, PA_KEYS, ke - j0, V);
     cp_commit();
   };
-  for (int i = tid; i < PA_ROWS * dk8; i += 128) {
-    int j = i / dk8, c = (i - j * dk8) * 8;
-    bool ok = i0 + j < n;
-    cp16(qs + j * ldk + c, q + (size_t)(ok ? i0 + j : 0) * q_stride + (size_t)h * DK + c, ok);
-  }
+  rk.run(qs, ldk, q + (size_t)i0 * q_stride + (size_t)h * DK, q_stride, PA_ROWS, n - i0, DK);
   fetch(kb, 0);  // kb < ke: row i0 sees at least itself
   float o[NV][4], mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
 #pragma unroll

@@ -10,6 +10,32 @@ __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)_
 __device__ __forceinline__ void cp16(bf16* dst, const bf16* src, bool valid) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(valid ? 16 : 0));
 }
+// How `threads` threads share the 16-byte groups of rows that are `per` groups wide: a thread keeps its group and walks rows
+// r, r + step, ..; worked out once, so that a copy inside a loop costs an addition.  Needs per <= threads.
+struct RowCopy {
+  int r, c, step;
+  bool on;
+  __device__ __forceinline__ RowCopy(int per, int tid, int threads) {
+    step = threads / per;
+    r = tid / per;
+    c = (tid - r * per) * 8;
+    on = r < step;
+  }
+  // rows [0, rows) of src (row length `stride`) to dst (row length ld); rows from `live` on, and groups from column `cols` on, become zero
+  __device__ __forceinline__ void run(bf16* dst, int ld, const bf16* src, long long stride, int rows, int live, int cols) const {
+    if (!on) return;
+    const bool in = c < cols;
+    const bf16* p = src + (size_t)r * stride + c;
+    bf16* d = dst + r * ld + c;
+    const size_t ps = (size_t)step * stride;
+    const int ds = step * ld;
+#pragma unroll 4
+    for (int j = r; j < rows; j += step, p += ps, d += ds) {
+      const bool ok = in && j < live;
+      cp16(d, ok ? p : src, ok);
+    }
+  }
+};
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;"); }
 template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N)); }
 __device__ __forceinline__ void ldm4(uint32_t* r, const bf16* p) {

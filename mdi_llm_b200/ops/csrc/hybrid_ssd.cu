@@ -132,16 +132,12 @@ __global__ void __launch_bounds__(256) ssd_decay_kernel(SsdArgs a) {
 }
 
 // rows [0, rows) x columns [0, cols) of a bf16 matrix into shared memory with row length ld; columns up to `colsp` and
-// rows from `live` on become zero.  vec: 16-byte asynchronous copies (cols a multiple of 8, sources 16-byte aligned).
+// rows from `live` on become zero.  vec: 16-byte asynchronous copies by `rc` (cols a multiple of 8, sources 16-byte aligned).
 template <int TH>
-__device__ __forceinline__ void stage(bf16* dst, int ld, const bf16* src, long long stride, int rows, int live, int cols, int colsp, int vec) {
+__device__ __forceinline__ void stage(const RowCopy& rc, bf16* dst, int ld, const bf16* src, long long stride, int rows, int live, int cols,
+                                      int colsp, int vec) {
   if (vec) {
-    const int per = colsp >> 3;
-    for (int i = threadIdx.x; i < rows * per; i += TH) {
-      int r = i / per, c = (i - r * per) * 8;
-      bool ok = r < live && c < cols;
-      cp16(dst + r * ld + c, ok ? src + (size_t)r * stride + c : src, ok);
-    }
+    rc.run(dst, ld, src, stride, rows, live, cols);
     return;
   }
   for (int i = threadIdx.x; i < rows * colsp; i += TH) {
@@ -151,10 +147,11 @@ __device__ __forceinline__ void stage(bf16* dst, int ld, const bf16* src, long l
 }
 
 // Block = (sequence, head, 32 value columns), 8 warps: warp w owns the state rows of the 16-row tiles w, w + 8, .. as
-// accumulators in registers.  A step takes in 64 tokens; its rows arrive by asynchronous copies two steps ahead.
+// accumulators in registers.  A step takes in 64 tokens.  Its rows arrive by asynchronous copies ahead of time; one step
+// ahead, x is multiplied by the tokens' weights and split into a bf16 number and its remainder, the right operands.
 #define SW_TH 256
 #define SW_VT 32
-#define SW_STAGES 3
+#define SW_STAGES 4
 template <int MT>
 __global__ void __launch_bounds__(SW_TH) ssd_walk_kernel(SsdArgs a, int vec) {
   extern __shared__ __align__(16) unsigned char raw[];
@@ -163,28 +160,43 @@ __global__ void __launch_bounds__(SW_TH) ssd_walk_kernel(SsdArgs a, int vec) {
   constexpr int ldv = SW_VT + 8;
   bf16* bs = reinterpret_cast<bf16*>(raw);       // [SW_STAGES][SW_L][ldn]
   bf16* xs = bs + SW_STAGES * SW_L * ldn;        // [SW_STAGES][SW_L][ldv]
+  bf16* wx = xs + SW_STAGES * SW_L * ldv;        // [2][number, remainder][SW_L][ldv]
   const int* m = a.meta + 4 * blockIdx.x;
   const int first = m[0], n = m[1], h = blockIdx.y, g = h / (a.H / a.G), v0 = blockIdx.z * SW_VT;
   const int cols = min(SW_VT, V - v0);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gr = lane >> 2, t2 = (lane & 3) * 2;
   float* sp = a.state + ((size_t)m[2] * a.H + h) * N * V + v0;
   bf16* out = (bf16*)a.before + ((size_t)a.stab[2 * blockIdx.x] * a.H + h) * 2 * N * V + v0;
-  auto fetch = [&](int c, int buf) {
+  const RowCopy rb(Np >> 3, tid, SW_TH), rx(SW_VT >> 3, tid, SW_TH);
+  const bf16* bsrc = (const bf16*)a.xbc + (size_t)first * a.xbc_stride + (size_t)a.H * V + (size_t)g * N;
+  const bf16* xsrc = (const bf16*)a.xbc + (size_t)first * a.xbc_stride + (size_t)h * V + v0;
+  const float4* dsrc = a.dec + (size_t)h * a.tokens + first;
+  auto fetch = [&](int c) {
     if (c < n) {
-      const bf16* base = (const bf16*)a.xbc + (size_t)(first + c) * a.xbc_stride;
-      const int len = min(SW_L, n - c);
-      stage<SW_TH>(bs + buf * SW_L * ldn, ldn, base + (size_t)a.H * V + (size_t)g * N, a.xbc_stride, SW_L, len, N, Np, vec);
-      stage<SW_TH>(xs + buf * SW_L * ldv, ldv, base + (size_t)h * V + v0, a.xbc_stride, SW_L, len, cols, SW_VT, vec);
-      if (tid < SW_L) {
-        const float4* src = a.dec + (size_t)h * a.tokens + first + c;
-        cp16(reinterpret_cast<bf16*>(&dec[buf][tid]), reinterpret_cast<const bf16*>(src + (tid < len ? tid : 0)), tid < len);
-      }
+      const int len = min(SW_L, n - c), buf = (c / SW_L) % SW_STAGES;
+      stage<SW_TH>(rb, bs + buf * SW_L * ldn, ldn, bsrc + (size_t)c * a.xbc_stride, a.xbc_stride, SW_L, len, N, Np, vec);
+      stage<SW_TH>(rx, xs + buf * SW_L * ldv, ldv, xsrc + (size_t)c * a.xbc_stride, a.xbc_stride, SW_L, len, cols, SW_VT, vec);
+      if (tid < SW_L) cp16(reinterpret_cast<bf16*>(&dec[buf][tid]), reinterpret_cast<const bf16*>(dsrc + c + (tid < len ? tid : 0)), tid < len);
     }
-    cp_commit();  // possibly an empty group: the wait below counts groups
+    cp_commit();  // possibly an empty group: the waits count groups
+  };
+  auto weigh = [&](int c) {  // 8 channels of one token per thread
+    if (c >= n) return;
+    const int buf = (c / SW_L) % SW_STAGES, s = tid >> 2, cc = (tid & 3) * 8;
+    bf16* o = wx + ((c / SW_L) & 1) * 2 * SW_L * ldv + s * ldv + cc;
+    const float w = dec[buf][s].w;
+    float f[8];
+    load8(xs + (buf * SW_L + s) * ldv + cc, f);
+    uint32_t hi[4], lo[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) split2(f[2 * e] * w, f[2 * e + 1] * w, hi[e], lo[e]);
+    *reinterpret_cast<uint4*>(o) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+    *reinterpret_cast<uint4*>(o + SW_L * ldv) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
   };
   float S[MT][SW_VT / 8][4];
-  fetch(0, 0);
-  fetch(SW_L, 1);
+  fetch(0);
+  fetch(SW_L);
+  fetch(2 * SW_L);
 #pragma unroll
   for (int i = 0; i < MT; ++i)
 #pragma unroll
@@ -194,40 +206,45 @@ __global__ void __launch_bounds__(SW_TH) ssd_walk_kernel(SsdArgs a, int vec) {
         const int d = (warp + 8 * i) * 16 + gr + 8 * (e >> 1), c = j * 8 + t2 + (e & 1);
         S[i][j][e] = d < N && c < cols ? sp[(size_t)d * V + c] : 0.f;
       }
-  int buf = 0;
-  for (int c0 = 0; c0 < n; c0 += SW_L, buf = buf == SW_STAGES - 1 ? 0 : buf + 1) {
-    const int len = min(SW_L, n - c0);
-    cp_wait<1>();
-    __syncthreads();
-    fetch(c0 + 2 * SW_L, buf == 0 ? SW_STAGES - 1 : buf - 1);
-    const float4* dk = dec[buf];
+  cp_wait<2>();
+  __syncthreads();
+  weigh(0);
+  for (int c0 = 0; c0 < n; c0 += SW_L) {
+    const int len = min(SW_L, n - c0), buf = (c0 / SW_L) % SW_STAGES;
+    cp_wait<1>();     // this thread's copies of the next step
+    __syncthreads();  // everybody's; and everybody is done with the step before
+    fetch(c0 + 3 * SW_L);
     const bf16* bb = bs + buf * SW_L * ldn;
-    const bf16* xb = xs + buf * SW_L * ldv;
+    const bf16* wh = wx + ((c0 / SW_L) & 1) * 2 * SW_L * ldv;
     if (c0 % SSD_CL == 0) {  // the state before this chunk of the outputs
       bf16* hi = out + (size_t)(c0 / SSD_CL) * a.H * 2 * N * V;
 #pragma unroll
       for (int i = 0; i < MT; ++i)
 #pragma unroll
-        for (int j = 0; j < SW_VT / 8; ++j)
+        for (int r = 0; r < 2; ++r) {
+          const int d = (warp + 8 * i) * 16 + gr + 8 * r;
+          if (d >= N) continue;
+          bf16* p = hi + (size_t)d * V + t2;
 #pragma unroll
-          for (int r = 0; r < 2; ++r) {
-            const int d = (warp + 8 * i) * 16 + gr + 8 * r, c = j * 8 + t2;
-            if (d >= N || c >= cols) continue;
+          for (int j = 0; j < SW_VT / 8; ++j) {
+            const int c = j * 8 + t2;
+            if (c >= cols) continue;
             uint32_t x, y;
             split2(S[i][j][2 * r], S[i][j][2 * r + 1], x, y);
-            bf16* p = hi + (size_t)d * V + c;
             if (vec) {
-              *reinterpret_cast<uint32_t*>(p) = x;
-              *reinterpret_cast<uint32_t*>(p + (size_t)N * V) = y;
+              *reinterpret_cast<uint32_t*>(p + j * 8) = x;
+              *reinterpret_cast<uint32_t*>(p + (size_t)N * V + j * 8) = y;
             } else {
               const __nv_bfloat162 px = *reinterpret_cast<__nv_bfloat162*>(&x), py = *reinterpret_cast<__nv_bfloat162*>(&y);
-              p[0] = px.x;
-              p[(size_t)N * V] = py.x;
-              if (c + 1 < cols) { p[1] = px.y; p[(size_t)N * V + 1] = py.y; }
+              p[j * 8] = px.x;
+              p[(size_t)N * V + j * 8] = py.x;
+              if (c + 1 < cols) { p[j * 8 + 1] = px.y; p[(size_t)N * V + j * 8 + 1] = py.y; }
             }
           }
+        }
     }
-    const float all = expf(dk[len - 1].x + dk[len - 1].y);
+    const float4 end = dec[buf][len - 1];
+    const float all = expf(end.x + end.y);
 #pragma unroll
     for (int i = 0; i < MT; ++i)
 #pragma unroll
@@ -235,33 +252,32 @@ __global__ void __launch_bounds__(SW_TH) ssd_walk_kernel(SsdArgs a, int vec) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) S[i][j][e] *= all;
 #pragma unroll
-    for (int k = 0; k < SW_L; k += 16) {
-      if (k >= len) break;
-      const float w[4] = {dk[k + t2].w, dk[k + t2 + 1].w, dk[k + 8 + t2].w, dk[k + 8 + t2 + 1].w};
-      uint32_t b[SW_VT / 16][4];
+    for (int k = 0; k < SW_L; k += 16) {  // rows from len on are zero
+      uint32_t b[SW_VT / 16][4], d[SW_VT / 16][4];
 #pragma unroll
-      for (int j = 0; j < SW_VT / 16; ++j) ldm4t(b[j], xb + (k + (lane & 15)) * ldv + (lane >> 4) * 8 + j * 16);
+      for (int j = 0; j < SW_VT / 16; ++j) {
+        ldm4t(b[j], wh + (k + (lane & 15)) * ldv + (lane >> 4) * 8 + j * 16);
+        ldm4t(d[j], wh + (SW_L + k + (lane & 15)) * ldv + (lane >> 4) * 8 + j * 16);
+      }
 #pragma unroll
       for (int i = 0; i < MT; ++i) {
         const int d0 = (warp + 8 * i) * 16;
         if (d0 >= Np) continue;
-        uint32_t A[4], ah[4], al[4];  // A[d][s] = B[s][d]: transposed 8x8 blocks (d 0-7 | 8-15) x (s 0-7 | 8-15)
+        uint32_t A[4];  // A[d][s] = B[s][d]: transposed 8x8 blocks (d 0-7 | 8-15) x (s 0-7 | 8-15)
         ldm4t(A, bb + (k + (lane & 7) + (lane >> 4) * 8) * ldn + d0 + ((lane >> 3) & 1) * 8);
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
-          split2(__uint_as_float(A[e] << 16) * w[(e >> 1) * 2], __uint_as_float(A[e] & 0xffff0000u) * w[(e >> 1) * 2 + 1], ah[e], al[e]);
-#pragma unroll
         for (int j = 0; j < SW_VT / 16; ++j) {
-          mma(S[i][2 * j], ah, b[j]);
-          mma(S[i][2 * j + 1], ah, b[j] + 2);
+          mma(S[i][2 * j], A, b[j]);
+          mma(S[i][2 * j + 1], A, b[j] + 2);
         }
 #pragma unroll
         for (int j = 0; j < SW_VT / 16; ++j) {
-          mma(S[i][2 * j], al, b[j]);
-          mma(S[i][2 * j + 1], al, b[j] + 2);
+          mma(S[i][2 * j], A, d[j]);
+          mma(S[i][2 * j + 1], A, d[j] + 2);
         }
       }
     }
+    weigh(c0 + SW_L);
   }
 #pragma unroll
   for (int i = 0; i < MT; ++i)
@@ -275,14 +291,16 @@ __global__ void __launch_bounds__(SW_TH) ssd_walk_kernel(SsdArgs a, int vec) {
 }
 
 // y of a chunk.  Block = (chunk, head), 8 warps of 16 token rows; value columns in tiles of 64.  C stays in registers as
-// left operand (NK: 16-wide steps of the state size).  Per row: the read-out of the state before the chunk, scaled by exp(c_t), then
-// by 16 earlier tokens the products C.B, weighed in registers and multiplied into x.
+// left operand (NK: 16-wide steps of the state size).  With r the last token before a warp's 16 rows,
+//   y_t = exp(c_t - c_r) [exp(c_r) S0^T C_t + sum_{s <= r} f(r, s) (C_t . B_s) x_s] + (the same 16 tokens, weighed one by one)
+// where f(r, s) = exp(c_r - c_s) dt_s is shared by the warp's rows: a table of them is made once per block.
 template <int NK>
-__global__ void __launch_bounds__(2 * SSD_CL) ssd_out_kernel(SsdArgs a, int vec) {
+__global__ void __launch_bounds__(2 * SSD_CL, NK <= 8 ? 2 : 1) ssd_out_kernel(SsdArgs a, int vec) {
   constexpr int TH = 2 * SSD_CL, ldv = 64 + 8;
   extern __shared__ __align__(16) unsigned char raw[];
   __shared__ float2 cum[SSD_CL];
   __shared__ float dts[SSD_CL];
+  __shared__ __align__(8) float tab[SSD_CL / 16][SSD_CL];  // tab[w][s] = f(16 w - 1, s), s < 16 w
   const int N = a.N, V = a.V, Np = (N + 15) & ~15, ldn = Np + 8;
   bf16* bs = reinterpret_cast<bf16*>(raw);  // [CL][ldn]
   bf16* xs = bs + SSD_CL * ldn;             // [CL][ldv]
@@ -293,7 +311,8 @@ __global__ void __launch_bounds__(2 * SSD_CL) ssd_out_kernel(SsdArgs a, int vec)
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gr = lane >> 2, t2 = (lane & 3) * 2;
   const bf16* base = (const bf16*)a.xbc + (size_t)row0 * a.xbc_stride;
   const bf16* before = (const bf16*)a.before + ((size_t)blockIdx.x * a.H + h) * 2 * N * V;
-  stage<TH>(bs, ldn, base + (size_t)a.H * V + (size_t)g * N, a.xbc_stride, SSD_CL, len, N, Np, vec);
+  const RowCopy rb(Np >> 3, tid, TH), rv((min(64, V) + 15) / 16 * 2, tid, TH);
+  stage<TH>(rb, bs, ldn, base + (size_t)a.H * V + (size_t)g * N, a.xbc_stride, SSD_CL, len, N, Np, vec);
   const int r0 = warp * 16;  // this lane's rows: r0 + gr and r0 + gr + 8
   uint32_t C[NK][4];
   {
@@ -335,10 +354,17 @@ __global__ void __launch_bounds__(2 * SSD_CL) ssd_out_kernel(SsdArgs a, int vec)
   for (int v0 = 0; v0 < V; v0 += 64) {
     const int cols = min(64, V - v0), colsp = (cols + 15) & ~15, nv = colsp >> 4;
     if (v0) __syncthreads();  // the tile before is done with xs, sh, sl
-    stage<TH>(xs, ldv, base + (size_t)h * V + v0, a.xbc_stride, SSD_CL, len, cols, colsp, vec);
-    stage<TH>(sh, ldv, before + v0, V, Np, N, cols, colsp, vec);
-    stage<TH>(sl, ldv, before + (size_t)N * V + v0, V, Np, N, cols, colsp, vec);
+    stage<TH>(rv, xs, ldv, base + (size_t)h * V + v0, a.xbc_stride, SSD_CL, len, cols, colsp, vec);
+    stage<TH>(rv, sh, ldv, before + v0, V, Np, N, cols, colsp, vec);
+    stage<TH>(rv, sl, ldv, before + (size_t)N * V + v0, V, Np, N, cols, colsp, vec);
     cp_commit();
+    if (v0 == 0) {
+      __syncthreads();  // cum and dts are written
+      for (int i = tid; i < SSD_CL / 16 * SSD_CL; i += TH) {
+        const int w = i / SSD_CL, s = i % SSD_CL;
+        if (s < 16 * w) tab[w][s] = dts[s] * expf(pair_diff(cum[16 * w - 1], cum[s]));
+      }
+    }
     cp_wait<0>();
     __syncthreads();
     if (r0 < len) {
@@ -363,9 +389,13 @@ __global__ void __launch_bounds__(2 * SSD_CL) ssd_out_kernel(SsdArgs a, int vec)
           }
       }
       const float2 ct[2] = {cum[r0 + gr], cum[r0 + gr + 8]};
-      const float e0 = expf(ct[0].x + ct[0].y), e1 = expf(ct[1].x + ct[1].y);
+      float2 cr = make_float2(0.f, 0.f);
+      if (warp) cr = cum[r0 - 1];
+      const float er = expf(cr.x + cr.y);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) { acc[i][0] *= e0; acc[i][1] *= e0; acc[i][2] *= e1; acc[i][3] *= e1; }
+      for (int i = 0; i < 8; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[i][e] *= er;
       for (int s0 = 0; s0 <= r0; s0 += 16) {
         float s[2][4];
 #pragma unroll
@@ -381,15 +411,29 @@ __global__ void __launch_bounds__(2 * SSD_CL) ssd_out_kernel(SsdArgs a, int vec)
           mma(s[0], C[k], b);
           mma(s[1], C[k], b + 2);
         }
+        if (s0 < r0) {
+#pragma unroll
+          for (int u = 0; u < 2; ++u) {
+            const float2 f = *reinterpret_cast<const float2*>(&tab[warp][s0 + u * 8 + t2]);
+            s[u][0] *= f.x; s[u][1] *= f.y; s[u][2] *= f.x; s[u][3] *= f.y;
+          }
+        } else {  // the rows' own tokens: everything so far belongs to tokens up to r
+          const float e0 = expf(pair_diff(ct[0], cr)), e1 = expf(pair_diff(ct[1], cr));
+#pragma unroll
+          for (int i = 0; i < 8; ++i) { acc[i][0] *= e0; acc[i][1] *= e0; acc[i][2] *= e1; acc[i][3] *= e1; }
+#pragma unroll
+          for (int u = 0; u < 2; ++u) {
+            const int src = s0 + u * 8 + t2;
+            const float2 cs[2] = {cum[src], cum[src + 1]};
+            const float w[2] = {dts[src], dts[src + 1]};
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+              s[u][e] = src + (e & 1) <= r0 + gr + (e >> 1) * 8 ? s[u][e] * (w[e & 1] * expf(pair_diff(ct[e >> 1], cs[e & 1]))) : 0.f;
+          }
+        }
         uint32_t hi[4], lo[4];
 #pragma unroll
         for (int u = 0; u < 2; ++u) {
-          const int src = s0 + u * 8 + t2;
-          const float2 cs[2] = {cum[src], cum[src + 1]};
-          const float w[2] = {dts[src], dts[src + 1]};
-#pragma unroll
-          for (int e = 0; e < 4; ++e)
-            s[u][e] = src + (e & 1) <= r0 + gr + (e >> 1) * 8 ? s[u][e] * (w[e & 1] * expf(pair_diff(ct[e >> 1], cs[e & 1]))) : 0.f;
           split2(s[u][0], s[u][1], hi[2 * u], lo[2 * u]);
           split2(s[u][2], s[u][3], hi[2 * u + 1], lo[2 * u + 1]);
         }
@@ -489,7 +533,7 @@ int hyb_ssd_chunked(const SsdArgs* args, cudaStream_t st) {
   if (a.G < 1 || a.H % a.G || a.N < 1 || a.V < 1) return -2;
   if (a.N > 256 || a.H > 65535) return -3;
   const size_t Np = (size_t)((a.N + 15) & ~15);
-  const size_t sw = SW_STAGES * SW_L * (Np + 8 + SW_VT + 8) * sizeof(bf16);
+  const size_t sw = (SW_STAGES * SW_L * (Np + 8 + SW_VT + 8) + 4 * SW_L * (SW_VT + 8)) * sizeof(bf16);
   const size_t so = (SSD_CL * (Np + 8) + SSD_CL * 72 + 2 * Np * 72) * sizeof(bf16);
   const uintptr_t bits = (uintptr_t)a.xbc | (uintptr_t)a.y | (uintptr_t)a.before | (uintptr_t)a.dec;
   const int vec = (bits & 15) == 0 && ((a.N | a.V) & 7) == 0 && (a.xbc_stride & 7) == 0;
