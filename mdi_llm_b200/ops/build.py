@@ -3,7 +3,7 @@
 ``nvcc -gencode arch=compute_100a,code=sm_100a -lineinfo`` over ``csrc/*.cu`` into one shared
 object ``mdi_llm_b200/ops/_mdi_ops.so`` (plain C ABI, loaded with ctypes — no torch headers, so a
 full rebuild takes seconds and the binary does not depend on the torch ABI).  The ``.so`` is
-git-ignored but travels with the ``gpurun`` snapshot.  nvcc cross-compiles without a GPU.
+git-ignored.  nvcc cross-compiles without a GPU.
 """
 from __future__ import annotations
 
